@@ -8,13 +8,14 @@ layers only, and `conv_state [n_conv][K-1][D]` zeroed at reset (src/model.zig:14
 * a *slot* is one sequence of a batch: its length, its pages in every group, its row in every
   state tensor.  Slots are handed out by `alloc_slots` and given back by `free_slots`; a freed
   slot's pages return to their pools and are reused by later batches.
-* layers whose mixers ask for the same kind of growing cache (same KV heads, widths and
-  window) form a *group* with storage of its own: two tensors
+* layers whose mixers ask for the same kind of growing cache (same KV heads, widths,
+  window and chunk) form a *group* with storage of its own: two tensors
   [layers of the group, pages, kv heads, page_size, width] (keys and values for attention; a
   mixer may ask for another width of the second, or for one tensor only) and one page table
   [slots, pages per sequence] shared by the group's layers.  A group with a window gives pages
   back as soon as every position in them has left the window; the pages that hold a sequence's first
-  `keep_first` tokens are never given back while the sequence lives.
+  `keep_first` tokens are never given back while the sequence lives.  A group whose tokens see only their own
+  stretch of `chunk` positions gives back the pages of the stretches before the next token's.
 * a mixer that asks for fixed-size state gets a row per slot in a tensor
   [calls with that state shape, slots, *shape], zeroed when the slot is handed out.
 
@@ -104,11 +105,11 @@ class KVGroup:
 
     def trim(self, slot: int, length: int) -> None:
         """Gives back pages whose positions all lie more than `window` behind the next query
-        (position `length`, which sees keys [length + 1 - window, length])."""
-        w = self.request.window
-        if w <= 0:
+        (position `length`, which sees keys [length + 1 - window, length]), or before its chunk."""
+        w, c = self.request.window, self.request.chunk
+        if w <= 0 and c <= 0:
             return
-        first_needed = max(0, length + 1 - w) // self.page_size
+        first_needed = (length // c * c if c > 0 else max(0, length + 1 - w)) // self.page_size
         while self.first_page_of[slot] < min(first_needed, self.n_pages_of[slot]):
             i = int(self.first_page_of[slot])
             if i >= self.kept_pages:
@@ -168,19 +169,22 @@ class CacheManager:
         # storage keeps what the widest of them sees (window 0 = everything), each call masks for itself.
         keep: dict[int, int] = {}
         first: dict[int, int] = {}      # the most first tokens any of them keeps beside its window
+        chunk: dict[int, int] = {}      # the chunk all of them share, or 0
         for c, owner in self._kv_of_call.items():
             if owner != c:
                 if owner not in self._kv_of_call or self._kv_of_call[owner] != owner:
                     raise CacheError(f"call {c} reads the cache of call {owner}, which owns none")
-                if replace(calls[owner].kv, window=0, keep_first=0) != replace(calls[c].kv, window=0, keep_first=0):
+                if (replace(calls[owner].kv, window=0, keep_first=0, chunk=0)
+                        != replace(calls[c].kv, window=0, keep_first=0, chunk=0)):
                     raise CacheError(f"call {c} reads the cache of call {owner} but asks for a different layout")
             w = calls[c].kv.window
             keep[owner] = w if owner not in keep else (0 if w <= 0 or keep[owner] <= 0 else max(keep[owner], w))
             first[owner] = max(first.get(owner, 0), calls[c].kv.keep_first)
+            chunk[owner] = calls[c].kv.chunk if chunk.get(owner, calls[c].kv.chunk) == calls[c].kv.chunk else 0
         for c, owner in self._kv_of_call.items():
             if owner == c:
-                by_request.setdefault(replace(calls[c].kv, window=keep[c], keep_first=first[c] if keep[c] > 0 else 0),
-                                      []).append(c)
+                by_request.setdefault(replace(calls[c].kv, window=keep[c], keep_first=first[c] if keep[c] > 0 else 0,
+                                              chunk=chunk[c]), []).append(c)
         for request, owners in by_request.items():
             g = len(self.groups)
             self.groups.append(KVGroup(request, len(owners), self.num_pages, page_size, max_slots,

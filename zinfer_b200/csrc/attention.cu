@@ -38,7 +38,11 @@ __global__ void qk_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_o
                                   const int* __restrict__ tok_pos, const int* __restrict__ seq_slot,
                                   const int* __restrict__ page_table, int pt_stride, int n_tokens, int H, int Hkv,
                                   int hd, int n_rot, int interleaved, float eps, int page_size, int write_kv,
-                                  int* status, int vd, int unit_norm_after, float qt_coef, int qt_every) {
+                                  int* status, int vd, int unit_norm_after, float qt_coef, int qt_every, int ld,
+                                  const T* __restrict__ v_first, int ld_first, int hs_first, int vd_first, float v_share) {
+  // ld: elements between rows of qkv (what lies behind a row's values is left alone).  v_first: value heads of the same tokens
+  // (rows ld_first, heads hs_first elements apart, vd_first values each) that are mixed in before the value is cached,
+  // v <- (1 - v_share) v + v_share v_first, in float32.
   // vd: width of a value head (a row of qkv is [q H*hd | k Hkv*hd | v Hkv*vd]).  unit_norm_after: q and k
   // heads are divided by their root mean square (no weight) AFTER the rotation; q_w / k_w, if given,
   // weigh an RMS norm BEFORE it.  qt_every > 0: a query at position p is multiplied, last of all, by
@@ -53,10 +57,9 @@ __global__ void qk_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_o
   const int kind = s < H ? 0 : (s < H + Hkv ? 1 : 2);  // 0 q, 1 k, 2 v
   if (kind != 0 && !write_kv && !dense_out) return;
   float* sm = sm_all[warp];
-  const size_t row_w = (size_t)(H + Hkv) * hd + (size_t)Hkv * vd;
   const int wd = kind == 2 ? vd : hd;
   const size_t col0 = kind == 2 ? (size_t)(H + Hkv) * hd + (size_t)(s - H - Hkv) * vd : (size_t)s * hd;
-  const T* src = qkv + (size_t)t * row_w + col0;
+  const T* src = qkv + (size_t)t * ld + col0;
   const float* w = kind == 0 ? q_w : (kind == 1 ? k_w : nullptr);
 
   float ss = 0.f;
@@ -69,6 +72,10 @@ __global__ void qk_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_o
     ss = warp_sum(ss);
     const float scale = 1.0f / sqrtf(ss / (float)hd + eps);
     for (int d = lane; d < hd; d += 32) sm[d] = (sm[d] * scale) * w[d];
+  }
+  if (kind == 2 && v_first) {
+    const T* vf = v_first + (size_t)t * ld_first + (size_t)(s - H - Hkv) * hs_first;
+    for (int d = lane; d < min(wd, vd_first); d += 32) sm[d] = (1.0f - v_share) * sm[d] + v_share * to_f32(vf[d]);
   }
   __syncwarp();
   const int pos = tok_pos[t];
@@ -100,7 +107,7 @@ __global__ void qk_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_o
   }
   T* dst;
   if (dense_out) {
-    dst = dense_out + (size_t)t * row_w + col0;
+    dst = dense_out + (size_t)t * ld + col0;
   } else if (kind == 0) {
     dst = q_out + (size_t)t * H * hd + (size_t)s * hd;
   } else {
@@ -129,7 +136,8 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
                             const float* __restrict__ inv_freq, const int* __restrict__ tok_seq,
                             const int* __restrict__ tok_pos, const int* __restrict__ seq_slot,
                             const int* __restrict__ page_table, int pt_stride, int H, int Hkv, float eps, int page_size,
-                            int write_kv, int* status, float qt_coef, int qt_every) {
+                            int write_kv, int* status, float qt_coef, int qt_every, int ld,
+                            const T* __restrict__ v_first, int ld_first, int hs_first, int vd_first, float v_share) {
   constexpr int E = HD / 64, HALF = HD / 2;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t = blockIdx.x;
@@ -156,7 +164,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
 #pragma unroll
     for (int u = 0; u < UN; ++u) {
       const int s = s0 + u * ATT_WARPS;
-      const T* src = qkv + (size_t)t * slots * HD + (size_t)min(s, n_slots - 1) * HD;
+      const T* src = qkv + (size_t)t * ld + (size_t)min(s, n_slots - 1) * HD;
 #pragma unroll
       for (int e = 0; e < E; ++e) {
         av[u][e] = to_f32(src[lane + 32 * e]);
@@ -195,6 +203,15 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
           const float x = a[e], y = b[e];
           a[e] = x * cs[e] - y * sn[e];
           b[e] = x * sn[e] + y * cs[e];
+        }
+      }
+      if (kind == 2 && v_first) {
+        const T* vf = v_first + (size_t)t * ld_first + (size_t)(s - H - Hkv) * hs_first;
+#pragma unroll
+        for (int e = 0; e < E; ++e) {
+          const int d = lane + 32 * e;
+          if (d < vd_first) a[e] = (1.0f - v_share) * a[e] + v_share * to_f32(vf[d]);
+          if (d + HALF < vd_first) b[e] = (1.0f - v_share) * b[e] + v_share * to_f32(vf[d + HALF]);
         }
       }
       T* dst;
@@ -359,7 +376,12 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
                     const int* __restrict__ page_table, int pt_stride, int n_tokens, int H, int Hkv, int hd,
                     int page_size, int window, float scale, int bq, int gc, int num_splits, int split_keys, int vd,
                     const float* __restrict__ bias_r1, const float* __restrict__ bias_r2, int cross, int keep,
-                    const float* __restrict__ sink, int v_from_k, float softcap) {
+                    const float* __restrict__ sink, int v_from_k, float softcap, const float* __restrict__ dist,
+                    int dist_len, int mask_chunk, const T* __restrict__ gate, int ld_gate) {
+  // dist [H, dist_len]: dist[h, min(i - j, dist_len - 1)] is added to the scaled score of query i and key j.
+  // mask_chunk > 0: a query sees only keys of its own stretch of mask_chunk positions, counted from position 0; the cuts
+  // of the keys between blocks then lie at multiples of split_keys from the start of the first query's stretch.
+  // gate: logits, rows ld_gate apart; head h's output of token t is multiplied by sigmoid(gate[t, h]) where it is normalised.
   // softcap > 0: a scaled score s becomes softcap * tanh(s / softcap) before anything else is done with it.
   // keep: with a window, the first `keep` positions of a sequence stay visible to every later query.
   // sink [H]: exp(sink_h) is one more term of head h's softmax denominator (no key, no value, unscaled).
@@ -403,6 +425,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
     row_h[i] = kvh * g + chunk * gc + hl;
     row_hi[i] = start + q0 + tq + 1;
     row_lo[i] = (window > 0 && row_hi[i] > window) ? row_hi[i] - window : 0;
+    if (mask_chunk > 0) row_lo[i] = (row_hi[i] - 1) / mask_chunk * mask_chunk;
   }
   float r1[4], r2[4];
 #pragma unroll
@@ -428,11 +451,13 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
     const int first_hi = start + q0 + 1;
     k_begin = first_hi > window ? first_hi - window : 0;
   }
+  const int cut0 = mask_chunk > 0 ? (start + q0) / mask_chunk * mask_chunk : 0;
+  if (mask_chunk > 0) k_begin = cut0;
   // the kept first tokens that lie below the window's reach: tiles [a_lo, a_hi), walked before the window's
   int a_lo = 0, a_hi = (keep > 0 && k_begin > 0) ? min(keep, k_begin) : 0;
   if (num_splits > 1) {
-    k_begin = max(k_begin, split * split_keys);
-    k_end = min(k_end, (split + 1) * split_keys);
+    k_begin = max(k_begin, cut0 + split * split_keys);
+    k_end = min(k_end, cut0 + (split + 1) * split_keys);
     a_lo = split * split_keys;
     a_hi = min(a_hi, (split + 1) * split_keys);
   }
@@ -447,7 +472,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
 #pragma unroll
     for (int c = 0; c < NPL; ++c) o[i][c] = 0.f;
   }
-  const int split_lo = num_splits > 1 ? split * split_keys : 0;
+  const int split_lo = num_splits > 1 ? cut0 + split * split_keys : 0;
 
   for (int phase = 0; phase < 2; ++phase)
   for (int kb = phase ? k_begin : a_lo; kb < (phase ? k_end : a_hi); kb += ATT_TK) {
@@ -493,6 +518,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
         sc = s[i] * scale;
         if (softcap > 0.f) sc = softcap * tanhf(sc / softcap);
         if (biased) sc -= r1[i] * log1pf(r2[i] * (float)(row_hi[i] - 1 - kp));
+        if (dist) sc += dist[(size_t)row_h[i] * dist_len + min(row_hi[i] - 1 - kp, dist_len - 1)];
       }
       const float mt = warp_max(sc);
       if (mt == -INFINITY) {  // no key of this tile is visible to this row
@@ -535,7 +561,8 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
 #pragma unroll
         for (int c = 0; c < NPL; ++c) o[i][c] *= alpha;
       }
-      const float inv = l[i] > 0.f ? 1.0f / l[i] : 0.f;
+      float inv = l[i] > 0.f ? 1.0f / l[i] : 0.f;
+      if (gate) inv /= 1.0f + expf(-to_f32(gate[(size_t)row_t[i] * ld_gate + row_h[i]]));
       T* dst = out + (size_t)row_t[i] * H * vd + (size_t)row_h[i] * vd;
 #pragma unroll
       for (int c = 0; c < NPL; ++c) {
@@ -561,12 +588,13 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
 // (3) merge: out = sum_s e^{m_s - M} o_s / sum_s e^{m_s - M} l_s.  One warp per (token, head).
 // A lane holds the (m, l) of one chunk (32 chunks at a time), so that the loads of all chunks are
 // under way together; the sums run over the chunks in ascending order whatever the timing.
-// With `sink` [H] (rows ordered (token, head)): exp(sink_h) is one more term of the denominator.  Rows wider than
+// With `sink` [H] (rows ordered (token, head)): exp(sink_h) is one more term of the denominator; with `gate` (logits, a
+// token's rows ld_gate apart) head h's result is multiplied by sigmoid(gate[t, h]).  Rows wider than
 // 256 values are merged 256 columns at a time.
 template <typename T>
 __global__ void attn_merge_kernel(const float* __restrict__ part_o_all, const float* __restrict__ part_ml,
                                   T* __restrict__ out_all, int n_rows, int hd_all, int num_splits,
-                                  const float* __restrict__ sink, int H) {
+                                  const float* __restrict__ sink, int H, const T* __restrict__ gate, int ld_gate) {
   zk_let_next_start();
   zk_wait_prior();   // nothing of the kernels before is read, and nothing written, above this line
   const int lane = threadIdx.x & 31;
@@ -613,7 +641,8 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o_all, const fl
         for (int i = 0; i < 8; ++i) acc[i] = fmaf(w[u], v[u][i], acc[i]);
     }
   }
-  const float inv = L > 0.f ? 1.0f / L : 0.f;
+  float inv = L > 0.f ? 1.0f / L : 0.f;
+  if (gate) inv /= 1.0f + expf(-to_f32(gate[(size_t)(row / H) * ld_gate + row % H]));
 #pragma unroll
   for (int i = 0; i < 8; ++i)
     if (lane + 32 * i < hd) out[(size_t)row * hd_all + lane + 32 * i] = from_f32<T>(acc[i] * inv);
@@ -727,7 +756,8 @@ int launch_attn(const void* q, const void* k_cache, const void* v_cache, void* o
                 const int* tile_seq, const int* tile_q0, const int* cu_q, const int* seq_start, const int* seq_slot,
                 const int* page_table, int pt_stride, int n_tiles, int n_tokens, int H, int Hkv, int hd, int page_size,
                 int window, float scale, int bq, int gc, int num_splits, int split_keys, int vd, const float* r1,
-                const float* r2, int cross, int keep, const float* sink, int v_from_k, float softcap, cudaStream_t stream) {
+                const float* r2, int cross, int keep, const float* sink, int v_from_k, float softcap, const float* dist,
+                int dist_len, int mask_chunk, const void* gate, int ld_gate, cudaStream_t stream) {
   const size_t smem = attn_smem_bytes(hd, v_from_k ? 0 : vd);
   if (smem > 227 * 1024) return ZK_EINVAL;
   auto kern = attn_fwd_kernel<T, NPL>;
@@ -741,7 +771,8 @@ int launch_attn(const void* q, const void* k_cache, const void* v_cache, void* o
   kern<<<grid, ATT_WARPS * 32, smem, stream>>>((const T*)q, (const T*)k_cache, (const T*)v_cache, (T*)out, part_o,
                                                part_ml, tile_seq, tile_q0, cu_q, seq_start, seq_slot, page_table,
                                                pt_stride, n_tokens, H, Hkv, hd, page_size, window, scale, bq, gc,
-                                               num_splits, split_keys, vd, r1, r2, cross, keep, sink, v_from_k, softcap);
+                                               num_splits, split_keys, vd, r1, r2, cross, keep, sink, v_from_k, softcap, dist,
+                                               dist_len, mask_chunk, (const T*)gate, ld_gate);
   return ZK_LAUNCH_STATUS();
 }
 
@@ -751,12 +782,13 @@ int dispatch_attn(int hd, const void* q, const void* k_cache, const void* v_cach
                   const int* seq_slot, const int* page_table, int pt_stride, int n_tiles, int n_tokens, int H, int Hkv,
                   int page_size, int window, float scale, int bq, int gc, int num_splits, int split_keys, int vd,
                   const float* r1, const float* r2, int cross, int keep, const float* sink, int v_from_k, float softcap,
-                  cudaStream_t stream) {
+                  const float* dist, int dist_len, int mask_chunk, const void* gate, int ld_gate, cudaStream_t stream) {
 #define ZK_ATT_CASE(N)                                                                                               \
   case N:                                                                                                            \
     return launch_attn<T, N>(q, k_cache, v_cache, out, part_o, part_ml, tile_seq, tile_q0, cu_q, seq_start, seq_slot, \
                              page_table, pt_stride, n_tiles, n_tokens, H, Hkv, hd, page_size, window, scale, bq, gc,  \
-                             num_splits, split_keys, vd, r1, r2, cross, keep, sink, v_from_k, softcap, stream);
+                             num_splits, split_keys, vd, r1, r2, cross, keep, sink, v_from_k, softcap, dist, dist_len,   \
+                             mask_chunk, gate, ld_gate, stream);
   int npl = (vd + 31) / 32;                 // value columns per lane: every count up to 8, then 12, 16, 20
   if (npl > 8) npl = npl <= 12 ? 12 : (npl <= 16 ? 16 : 20);
   switch (npl) {
@@ -780,11 +812,14 @@ int zk_qk_prepare(const void* qkv, void* q_out, void* dense_out, void* k_cache, 
                   const float* inv_freq, const int* tok_seq, const int* tok_pos, const int* seq_slot,
                   const int* page_table, int pt_stride, int n_tokens, int H, int Hkv, int hd, int n_rot,
                   int interleaved, float eps, int page_size, int write_kv, int dtype, int* status, int vd,
-                  int unit_norm_after, float qt_coef, int qt_every, cudaStream_t stream) {
+                  int unit_norm_after, float qt_coef, int qt_every, int ld, const void* v_first, int ld_first, int hs_first,
+                  int vd_first, float v_share, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (hd <= 0 || hd > ATT_MAX_HD || H <= 0 || Hkv <= 0 || n_rot > hd || (n_rot & 1) || page_size <= 0) return ZK_EINVAL;
   if (vd <= 0) vd = hd;
   if (vd > ATT_MAX_HD) return ZK_EINVAL;
+  if (ld < (H + Hkv) * hd + Hkv * vd) return ZK_EINVAL;
+  if (v_first && (vd_first <= 0 || vd_first > vd || hs_first < vd_first || ld_first < (Hkv - 1) * hs_first + vd_first)) return ZK_EINVAL;
   // many tokens, whole-head half-split rotation (or none): one block per token
   if (n_tokens >= 256 && !dense_out && (hd == 64 || hd == 128) && vd == hd && !unit_norm_after &&
       (!inv_freq || (n_rot == hd && !interleaved)) &&
@@ -792,7 +827,8 @@ int zk_qk_prepare(const void* qkv, void* q_out, void* dense_out, void* k_cache, 
 #define ZK_QKP(T, HDV)                                                                                               \
   zk_launch_dependent(qk_prepare_token_kernel<T, HDV>, dim3(n_tokens), dim3(ATT_WARPS * 32), 0, stream,             \
       (const T*)qkv, (T*)q_out, (T*)k_cache, (T*)v_cache, q_w, k_w, inv_freq, tok_seq, tok_pos, seq_slot, page_table, \
-      pt_stride, H, Hkv, eps, page_size, write_kv, status, qt_coef, qt_every)
+      pt_stride, H, Hkv, eps, page_size, write_kv, status, qt_coef, qt_every, ld, (const T*)v_first, ld_first, hs_first,     \
+      vd_first, v_share)
     if (dtype == ZK_F32 && hd == 64) ZK_QKP(float, 64);
     else if (dtype == ZK_F32) ZK_QKP(float, 128);
     else if (hd == 64) ZK_QKP(bf16, 64);
@@ -806,12 +842,12 @@ int zk_qk_prepare(const void* qkv, void* q_out, void* dense_out, void* k_cache, 
     return zk_launch_dependent(qk_prepare_kernel<float>, dim3(blocks), dim3(ATT_WARPS * 32), 0, stream,
         (const float*)qkv, (float*)q_out, (float*)dense_out, (float*)k_cache, (float*)v_cache, q_w, k_w, inv_freq, tok_seq, tok_pos,
         seq_slot, page_table, pt_stride, n_tokens, H, Hkv, hd, n_rot, interleaved, eps, page_size, write_kv, status, vd,
-        unit_norm_after, qt_coef, qt_every);
+        unit_norm_after, qt_coef, qt_every, ld, (const float*)v_first, ld_first, hs_first, vd_first, v_share);
   else if (dtype == ZK_BF16)
     return zk_launch_dependent(qk_prepare_kernel<bf16>, dim3(blocks), dim3(ATT_WARPS * 32), 0, stream,
         (const bf16*)qkv, (bf16*)q_out, (bf16*)dense_out, (bf16*)k_cache, (bf16*)v_cache, q_w, k_w, inv_freq, tok_seq, tok_pos, seq_slot,
         page_table, pt_stride, n_tokens, H, Hkv, hd, n_rot, interleaved, eps, page_size, write_kv, status, vd,
-        unit_norm_after, qt_coef, qt_every);
+        unit_norm_after, qt_coef, qt_every, ld, (const bf16*)v_first, ld_first, hs_first, vd_first, v_share);
   else
     return ZK_EINVAL;
   return ZK_LAUNCH_STATUS();
@@ -860,8 +896,12 @@ int zk_attn_fwd(const void* q, const void* k_cache, const void* v_cache, void* o
                 const int* page_table, int pt_stride, int n_tiles, int n_tokens, int H, int Hkv, int hd, int page_size,
                 int window, float scale, int bq, int gc, int num_splits, int split_keys, int dtype, int vd,
                 const float* bias_r1, const float* bias_r2, int cross, int keep, const float* sink, int v_from_k,
-                float softcap, cudaStream_t stream) {
+                float softcap, const float* dist, int dist_len, int mask_chunk, const void* gate, int ld_gate, cudaStream_t stream) {
   if (n_tiles <= 0 || n_tokens <= 0) return 0;
+  if ((dist && dist_len <= 0) || mask_chunk < 0 || (mask_chunk > 0 && (window > 0 || cross)) || (cross && (dist || gate)) ||
+      (gate && ld_gate < H))
+    return ZK_EINVAL;
+  if (mask_chunk > 0 && num_splits > 1 && bq != 1 && n_tiles != n_tokens) return ZK_EINVAL;   // the cuts follow ONE query's stretch
   if (keep < 0 || (v_from_k && (vd > hd || cross))) return ZK_EINVAL;
   if (cross && (!part_o || !part_ml)) return ZK_EINVAL;
   if (hd <= 0 || hd > ATT_MAX_HD || H <= 0 || Hkv <= 0 || H % Hkv || page_size <= 0) return ZK_EINVAL;
@@ -871,11 +911,11 @@ int zk_attn_fwd(const void* q, const void* k_cache, const void* v_cache, void* o
   if (dtype == ZK_F32)
     return dispatch_attn<float>(hd, q, k_cache, v_cache, out, part_o, part_ml, tile_seq, tile_q0, cu_q, seq_start,
                                 seq_slot, page_table, pt_stride, n_tiles, n_tokens, H, Hkv, page_size, window, scale,
-                                bq, gc, num_splits, split_keys, vd, bias_r1, bias_r2, cross, keep, sink, v_from_k, softcap, stream);
+                                bq, gc, num_splits, split_keys, vd, bias_r1, bias_r2, cross, keep, sink, v_from_k, softcap, dist, dist_len, mask_chunk, gate, ld_gate, stream);
   if (dtype == ZK_BF16)
     return dispatch_attn<bf16>(hd, q, k_cache, v_cache, out, part_o, part_ml, tile_seq, tile_q0, cu_q, seq_start,
                                seq_slot, page_table, pt_stride, n_tiles, n_tokens, H, Hkv, page_size, window, scale, bq,
-                               gc, num_splits, split_keys, vd, bias_r1, bias_r2, cross, keep, sink, v_from_k, softcap, stream);
+                               gc, num_splits, split_keys, vd, bias_r1, bias_r2, cross, keep, sink, v_from_k, softcap, dist, dist_len, mask_chunk, gate, ld_gate, stream);
   return ZK_EINVAL;
 }
 
@@ -917,15 +957,16 @@ int zk_attn_merge_talk(const float* part_o, const float* part_ml, const float* t
 }
 
 int zk_attn_merge(const float* part_o, const float* part_ml, void* out, int n_rows, int hd, int num_splits, int dtype,
-                  const float* sink, int H, cudaStream_t stream) {
+                  const float* sink, int H, const void* gate, int ld_gate, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
-  if (sink && (H <= 0 || n_rows % H)) return ZK_EINVAL;
+  if ((sink || gate) && (H <= 0 || n_rows % H)) return ZK_EINVAL;
+  if (gate && ld_gate < H) return ZK_EINVAL;
   const int warps = 4;
   const int blocks = (n_rows + warps - 1) / warps;
   if (dtype == ZK_F32)
-    return zk_launch_dependent(attn_merge_kernel<float>, dim3(blocks), dim3(warps * 32), 0, stream, part_o, part_ml, (float*)out, n_rows, hd, num_splits, sink, H);
+    return zk_launch_dependent(attn_merge_kernel<float>, dim3(blocks), dim3(warps * 32), 0, stream, part_o, part_ml, (float*)out, n_rows, hd, num_splits, sink, H, (const float*)gate, ld_gate);
   else if (dtype == ZK_BF16)
-    return zk_launch_dependent(attn_merge_kernel<bf16>, dim3(blocks), dim3(warps * 32), 0, stream, part_o, part_ml, (bf16*)out, n_rows, hd, num_splits, sink, H);
+    return zk_launch_dependent(attn_merge_kernel<bf16>, dim3(blocks), dim3(warps * 32), 0, stream, part_o, part_ml, (bf16*)out, n_rows, hd, num_splits, sink, H, (const bf16*)gate, ld_gate);
   else
     return ZK_EINVAL;
   return ZK_LAUNCH_STATUS();

@@ -73,7 +73,12 @@ __global__ void __launch_bounds__(DT_WARPS * 32)
                           const int* __restrict__ page_table, int pt_stride, int n_seqs, int H, int Hkv, int page_size,
                           int window, float scale, int num_splits, int split_keys, const float* __restrict__ bias_r1,
                           const float* __restrict__ bias_r2, int cross, int keep, const float* __restrict__ sink,
-                          float softcap) {
+                          float softcap, const float* __restrict__ dist, int dist_len, int mask_chunk,
+                          const bf16* __restrict__ gate, int ld_gate) {
+  // dist [H, dist_len]: dist[h, min(distance, dist_len - 1)] is added to the scaled score of the key `distance` tokens
+  // behind the query.  mask_chunk > 0: only keys of the query's own stretch of mask_chunk positions (counted from position
+  // 0) are visible, and the cuts between blocks lie at multiples of split_keys from the stretch's start.
+  // gate: logits, rows ld_gate apart; head h's output is multiplied by sigmoid(gate[b, h]) where it is normalised.
   // softcap > 0: a scaled score s becomes softcap * tanh(s / softcap) (then carried to base 2 like every score).
   // keep: with a window, the first `keep` keys of a sequence stay visible; the block whose chunk starts at the
   // window's lower edge also walks the tiles that hold them, before its own.
@@ -101,11 +106,12 @@ __global__ void __launch_bounds__(DT_WARPS * 32)
   // (vh - kvh) * page_size rows further on in the same page
   const bf16* v_rows = v_cache + (ptrdiff_t)(vh - kvh) * page_size * HD;
   const int L = seq_start[b] + 1;  // keys 0 .. L-1; the new token's own key is the last
-  const int lo = (window > 0 && L > window) ? L - window : 0;
+  const int lo = mask_chunk > 0 ? (L - 1) / mask_chunk * mask_chunk : (window > 0 && L > window) ? L - window : 0;
+  const int cut0 = mask_chunk > 0 ? lo : 0;
   int c0 = lo, c1 = L;             // this block's keys [c0, c1)
   if (num_splits > 1) {
-    c0 = max(lo, split * split_keys);
-    c1 = min(L, (split + 1) * split_keys);
+    c0 = max(lo, cut0 + split * split_keys);
+    c1 = min(L, cut0 + (split + 1) * split_keys);
   }
   const int* pt = page_table + (size_t)seq_slot[b] * pt_stride;
 
@@ -191,6 +197,11 @@ __global__ void __launch_bounds__(DT_WARPS * 32)
       r2[h] = bias_r2[head];
     }
   }
+  const float* dist_row[2] = {nullptr, nullptr};
+  if (dist) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h) dist_row[h] = dist + (size_t)(kvh * G + min(g + 8 * h, G - 1)) * dist_len;
+  }
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   float o[HD / 8][4];
 #pragma unroll
@@ -241,6 +252,7 @@ __global__ void __launch_bounds__(DT_WARPS * 32)
         float sc = s[j][i] * scale2;
         if (softcap > 0.f) sc = cap2 * fast_tanh(s[j][i] * scale_cap);
         if (biased) sc -= r1_2[i >> 1] * log1pf(r2[i >> 1] * (float)max(L - 1 - kp, 0));
+        if (dist) sc = fmaf(dist_row[i >> 1][min(max(L - 1 - kp, 0), dist_len - 1)], 1.4426950408889634f, sc);
         if (edge_tile) {
           const bool vis = (kp >= c0 || kp < keep_here) && kp < c1;
           s[j][i] = vis ? sc : -INFINITY;
@@ -340,6 +352,7 @@ __global__ void __launch_bounds__(DT_WARPS * 32)
         Lsum = Lsum * back + expf(sk - m_fin);
         O *= back;
       }
+      if (gate) O /= 1.0f + expf(-to_f32(gate[(size_t)b * ld_gate + head]));
       out[(size_t)b * H * HD + (size_t)head * HD + d] = __float2bfloat16_rn(Lsum > 0.f ? O / Lsum : 0.f);
     } else {
       const size_t row = cross ? (((size_t)split * n_seqs + b) * H + head) * Hkv + vh : ((size_t)split * n_seqs + b) * H + head;
@@ -356,7 +369,8 @@ template <int HD, int NST>
 int launch(const void* q, const void* k_cache, const void* v_cache, void* out, float* part_o, float* part_ml,
            const int* seq_start, const int* seq_slot, const int* page_table, int pt_stride, int n_seqs, int H, int Hkv,
            int page_size, int window, float scale, int num_splits, int split_keys, const float* r1, const float* r2,
-           int cross, int keep, const float* sink, float softcap, cudaStream_t stream) {
+           int cross, int keep, const float* sink, float softcap, const float* dist, int dist_len, int mask_chunk,
+           const void* gate, int ld_gate, cudaStream_t stream) {
   auto kern = attn_decode_tc_kernel<HD, NST>;
   const size_t smem = 2 * NST * (size_t)DT_TK * HD * 2;
   static_assert(2 * NST * DT_TK * HD * 2 >= (2 * DT_WARPS * 16 + DT_WARPS * 16 * HD) * 4, "the merge fits in the tile buffers");
@@ -367,8 +381,8 @@ int launch(const void* q, const void* k_cache, const void* v_cache, void* out, f
   dim3 grid(n_seqs, Hkv * (cross ? Hkv : 1), num_splits);
   return zk_launch_dependent(kern, grid, dim3(DT_WARPS * 32), smem, stream, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out,
                                               part_o, part_ml, seq_start, seq_slot, page_table, pt_stride, n_seqs, H, Hkv,
-                                              page_size, window, scale, num_splits, split_keys, r1, r2, cross, keep, sink, softcap);
-  return ZK_LAUNCH_STATUS();
+                                              page_size, window, scale, num_splits, split_keys, r1, r2, cross, keep, sink, softcap, dist, dist_len, mask_chunk,
+                                              (const bf16*)gate, ld_gate);
 }
 
 }  // namespace
@@ -386,12 +400,17 @@ int zk_attn_decode_tc_takes(int H, int Hkv, int hd, int page_size) {
 
 // q, out [n_seqs, H*hd] bfloat16; partials as for zk_attn_fwd when num_splits > 1 (the merge then adds the sink).
 // keep > 0 (with a window) and sink [H] float32 as the kernel describes them; neither goes with the cross mode.
+// dist [H, dist_len] float32, mask_chunk (not with a window) and gate [n_seqs, >= H] bfloat16 as the kernel describes them, each
+// absent as null or 0; none goes with the cross mode.  With num_splits > 1 the merge applies the gate.
 int zk_attn_decode_tc(const void* q, const void* k_cache, const void* v_cache, void* out, float* part_o, float* part_ml,
                       const int* seq_start, const int* seq_slot, const int* page_table, int pt_stride, int n_seqs, int H,
                       int Hkv, int hd, int page_size, int window, float scale, int num_splits, int split_keys,
                       const float* bias_r1, const float* bias_r2, int cross, int keep, const float* sink, float softcap,
-                      cudaStream_t stream) {
+                      const float* dist, int dist_len, int mask_chunk, const void* gate, int ld_gate, cudaStream_t stream) {
   if (n_seqs <= 0) return 0;
+  if ((dist && dist_len <= 0) || mask_chunk < 0 || (mask_chunk > 0 && (window > 0 || cross)) || (cross && (dist || gate)) ||
+      (gate && ld_gate < H))
+    return ZK_EINVAL;
   if (keep < 0 || (keep > 0 && window <= 0) || (cross && (keep > 0 || sink))) return ZK_EINVAL;
   if (cross && (!part_o || !part_ml)) return ZK_EINVAL;
   if (!zk_attn_decode_tc_takes(H, Hkv, hd, page_size) || num_splits < 1) return ZK_EINVAL;
@@ -406,12 +425,12 @@ int zk_attn_decode_tc(const void* q, const void* k_cache, const void* v_cache, v
   const bool short_chunks = num_splits > 1 && split_keys <= 4 * DT_TK;
   if (hd == 64 && short_chunks)
     return launch<64, 4>(q, k_cache, v_cache, out, part_o, part_ml, seq_start, seq_slot, page_table, pt_stride, n_seqs, H,
-                         Hkv, page_size, window, scale, num_splits, split_keys, bias_r1, bias_r2, cross, keep, sink, softcap, stream);
+                         Hkv, page_size, window, scale, num_splits, split_keys, bias_r1, bias_r2, cross, keep, sink, softcap, dist, dist_len, mask_chunk, gate, ld_gate, stream);
   if (hd == 64)
     return launch<64, 2>(q, k_cache, v_cache, out, part_o, part_ml, seq_start, seq_slot, page_table, pt_stride, n_seqs, H,
-                         Hkv, page_size, window, scale, num_splits, split_keys, bias_r1, bias_r2, cross, keep, sink, softcap, stream);
+                         Hkv, page_size, window, scale, num_splits, split_keys, bias_r1, bias_r2, cross, keep, sink, softcap, dist, dist_len, mask_chunk, gate, ld_gate, stream);
   return launch<128, 2>(q, k_cache, v_cache, out, part_o, part_ml, seq_start, seq_slot, page_table, pt_stride, n_seqs, H,
-                     Hkv, page_size, window, scale, num_splits, split_keys, bias_r1, bias_r2, cross, keep, sink, softcap, stream);
+                     Hkv, page_size, window, scale, num_splits, split_keys, bias_r1, bias_r2, cross, keep, sink, softcap, dist, dist_len, mask_chunk, gate, ld_gate, stream);
 }
 
 }  // extern "C"

@@ -63,7 +63,12 @@ __global__ void __launch_bounds__(PF_WARPS * 32)
                         const int* __restrict__ seq_slot, const int* __restrict__ page_table, int pt_stride, int H,
                         int Hkv, int page_size, int window, float scale, const float* __restrict__ bias_r1,
                         const float* __restrict__ bias_r2, float* __restrict__ part_o, float* __restrict__ part_ml,
-                        int keep, const float* __restrict__ sink, float softcap) {
+                        int keep, const float* __restrict__ sink, float softcap, const float* __restrict__ dist,
+                        int dist_len, int mask_chunk, const bf16* __restrict__ gate, int ld_gate) {
+  // dist [H, dist_len]: dist[h, min(i - j, dist_len - 1)] is added to the scaled score of query position i and key
+  // position j; the stretch of it that a key tile needs is staged in shared memory.
+  // mask_chunk > 0: a query sees only keys of its own stretch of mask_chunk positions, counted from position 0.
+  // gate: logits, rows ld_gate apart; head h's output of token t is multiplied by sigmoid(gate[t, h]).
   // keep: with a window, the first `keep` positions of a sequence stay visible to every later query; the tiles
   // that hold them and lie below the window's reach are walked before the window's.
   // sink [H]: exp(sink_h) is one more term of head h's softmax denominator (no key, no value, unscaled).
@@ -81,6 +86,7 @@ __global__ void __launch_bounds__(PF_WARPS * 32)
   constexpr int CHV = HDV / 8;
   constexpr int TILE_BYTES = PF_TK * HD * 2, VTILE_BYTES = PF_TK * HDV * 2;
   extern __shared__ __align__(128) unsigned char smem[];
+  __shared__ float dist_sm[GP][PF_TK + BQ];
   unsigned char* Ksm[2] = {smem, smem + TILE_BYTES};
   unsigned char* Vsm[2] = {smem + 2 * TILE_BYTES, smem + 2 * TILE_BYTES + VTILE_BYTES};
 
@@ -100,7 +106,7 @@ __global__ void __launch_bounds__(PF_WARPS * 32)
   const int page0 = seq_slot[b];
 
   // this thread's two rows: r0 = warp*16 + g and r0 + 8
-  int row_tok[2], row_head[2], row_hi[2], row_lo[2];
+  int row_tok[2], row_head[2], row_hi[2], row_lo[2], row_dist[2];   // row_dist: where key 0 of a tile meets the row in dist_sm
   bool row_ok[2];
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
@@ -111,6 +117,8 @@ __global__ void __launch_bounds__(PF_WARPS * 32)
     row_head[h] = kvh * G + chunk * GP + hl;
     row_hi[h] = start + q0 + tq + 1;
     row_lo[h] = (window > 0 && row_hi[h] > window) ? row_hi[h] - window : 0;
+    if (mask_chunk > 0) row_lo[h] = (row_hi[h] - 1) / mask_chunk * mask_chunk;
+    row_dist[h] = hl * (PF_TK + BQ) + tq + PF_TK - 1;
   }
   const bool biased = bias_r1 != nullptr;
   float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};
@@ -140,6 +148,7 @@ __global__ void __launch_bounds__(PF_WARPS * 32)
     const int first_hi = start + q0 + 1;
     k_begin = first_hi > window ? first_hi - window : 0;
   }
+  if (mask_chunk > 0) k_begin = (start + q0) / mask_chunk * mask_chunk;
   k_begin = (k_begin / PF_TK) * PF_TK;
   // kept first tokens below the window's first tile: keys [0, a_hi) in a_tiles tiles, which end at or before k_begin
   const int a_hi = (keep > 0 && k_begin > 0) ? min(keep, k_begin) : 0;
@@ -181,8 +190,15 @@ __global__ void __launch_bounds__(PF_WARPS * 32)
     } else {
       cp_async_wait<0>();
     }
-    __syncthreads();
     const int kb = t < a_tiles ? t * PF_TK : k_begin + (t - a_tiles) * PF_TK;
+    if (dist) {      // distances start + q0 - kb - (PF_TK - 1) .. + BQ - 1 of this block's heads (the last tile is consumed)
+      const int d0 = start + q0 - kb - (PF_TK - 1);
+      for (int i = tid; i < GP * (PF_TK + BQ); i += PF_WARPS * 32) {
+        const int hl = i / (PF_TK + BQ), n = d0 + i % (PF_TK + BQ);
+        (&dist_sm[0][0])[i] = dist[(size_t)(kvh * G + chunk * GP + hl) * dist_len + min(max(n, 0), dist_len - 1)];
+      }
+    }
+    __syncthreads();
 
     // S = Q K^T: 8 key groups of 8, KS k steps
     float s[8][4];
@@ -216,6 +232,7 @@ __global__ void __launch_bounds__(PF_WARPS * 32)
         float sc = s[j][i] * scale;
         if (softcap > 0.f) sc = softcap * fast_tanh(sc * inv_cap);     // capped scores
         if (biased && vis) sc -= r1[h] * log1pf(r2[h] * (float)(row_hi[h] - 1 - kp));
+        if (dist) sc += (&dist_sm[0][0])[row_dist[h] - (kp - kb)];
         s[j][i] = vis ? sc : -INFINITY;
         m_new[h] = fmaxf(m_new[h], s[j][i]);
       }
@@ -289,7 +306,8 @@ __global__ void __launch_bounds__(PF_WARPS * 32)
       back = m_run[h] == -INFINITY ? 0.f : expf(m_run[h] - m_fin);
       l_run[h] = l_run[h] * back + expf(sk - m_fin);
     }
-    const float inv = l_run[h] > 0.f ? back / l_run[h] : 0.f;
+    float inv = l_run[h] > 0.f ? back / l_run[h] : 0.f;
+    if (gate) inv /= 1.0f + expf(-to_f32(gate[(size_t)row_tok[h] * ld_gate + row_head[h]]));
     bf16* dst = out + (size_t)row_tok[h] * H * HDV + (size_t)row_head[h] * HDV;
 #pragma unroll
     for (int j = 0; j < HDV / 8; ++j)
@@ -301,7 +319,8 @@ template <int HD, int HDV, int GP>
 int launch(const void* q, const void* k_cache, const void* v_cache, void* out, const int* tile_seq, const int* tile_q0,
            const int* cu_q, const int* seq_start, const int* seq_slot, const int* page_table, int pt_stride, int n_tiles,
            int H, int Hkv, int page_size, int window, float scale, const float* r1, const float* r2, float* part_o,
-           float* part_ml, int keep, const float* sink, float softcap, cudaStream_t stream) {
+           float* part_ml, int keep, const float* sink, float softcap, const float* dist, int dist_len, int mask_chunk,
+           const void* gate, int ld_gate, cudaStream_t stream) {
   auto kern = attn_prefill_kernel<HD, HDV, GP>;
   const size_t smem = 2 * (size_t)PF_TK * (HD + HDV) * 2;
   if (smem > 48 * 1024) {
@@ -311,7 +330,8 @@ int launch(const void* q, const void* k_cache, const void* v_cache, void* out, c
   dim3 grid(n_tiles, Hkv * ((H / Hkv) / GP), part_o ? Hkv : 1);
   kern<<<grid, PF_WARPS * 32, smem, stream>>>((const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out,
                                               tile_seq, tile_q0, cu_q, seq_start, seq_slot, page_table, pt_stride, H,
-                                              Hkv, page_size, window, scale, r1, r2, part_o, part_ml, keep, sink, softcap);
+                                              Hkv, page_size, window, scale, r1, r2, part_o, part_ml, keep, sink, softcap, dist,
+                                              dist_len, mask_chunk, (const bf16*)gate, ld_gate);
   return ZK_LAUNCH_STATUS();
 }
 
@@ -337,12 +357,18 @@ int zk_attn_prefill_tile_tokens(int H, int Hkv) { return PF_ROWS / packed_heads(
 // part_ml [n_tokens*H*Hkv, 2] float32 (both or neither) switch the cross mode on: `out` is then not written.
 // keep > 0 (with a window) and sink [H] float32 as the kernel describes them; neither goes with the cross mode.
 // page_table null: keys and values laid out for this step alone, as the kernel describes (seq_slot = first pages).
+// dist [H, dist_len] float32, mask_chunk, gate [n_tokens, >= H] bfloat16 (rows ld_gate apart) as the kernel describes them, each
+// absent as null or 0; none goes with the cross mode, mask_chunk not with a window.
 int zk_attn_prefill(const void* q, const void* k_cache, const void* v_cache, void* out, const int* tile_seq,
                     const int* tile_q0, const int* cu_q, const int* seq_start, const int* seq_slot,
                     const int* page_table, int pt_stride, int n_tiles, int H, int Hkv, int hd, int vd,
                     int page_size, int window, float scale, const float* bias_r1, const float* bias_r2, float* part_o, float* part_ml,
-                    int keep, const float* sink, float softcap, cudaStream_t stream) {
+                    int keep, const float* sink, float softcap, const float* dist, int dist_len, int mask_chunk,
+                    const void* gate, int ld_gate, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
+  if ((dist && dist_len <= 0) || mask_chunk < 0 || (mask_chunk > 0 && window > 0) || (part_o && (mask_chunk > 0 || dist || gate)) ||
+      (gate && ld_gate < H))
+    return ZK_EINVAL;
   if (!zk_attn_prefill_takes(H, Hkv, hd, page_size) || ((bias_r1 == nullptr) != (bias_r2 == nullptr))) return ZK_EINVAL;
   if ((part_o == nullptr) != (part_ml == nullptr) || (part_o && Hkv > 65535)) return ZK_EINVAL;
   if (keep < 0 || (keep > 0 && window <= 0) || (part_o && (keep > 0 || sink))) return ZK_EINVAL;
@@ -352,14 +378,14 @@ int zk_attn_prefill(const void* q, const void* k_cache, const void* v_cache, voi
   if (hd == HDK && vd == HDK && gp == GPV)                                                                       \
     return launch<HDK, HDK, GPV>(q, k_cache, v_cache, out, tile_seq, tile_q0, cu_q, seq_start, seq_slot, page_table,  \
                             pt_stride, n_tiles, H, Hkv, page_size, window, scale, bias_r1, bias_r2, part_o, part_ml,  \
-                            keep, sink, softcap, stream);
+                            keep, sink, softcap, dist, dist_len, mask_chunk, gate, ld_gate, stream);
   ZK_PF(64, 1) ZK_PF(64, 2) ZK_PF(64, 4) ZK_PF(64, 8)
   ZK_PF(128, 1) ZK_PF(128, 2) ZK_PF(128, 4) ZK_PF(128, 8)
 #undef ZK_PF
   if (hd == 128 && vd == 64 && gp == 1)      // narrow values: attention whose heads each have keys and values of their own
     return launch<128, 64, 1>(q, k_cache, v_cache, out, tile_seq, tile_q0, cu_q, seq_start, seq_slot, page_table,
                               pt_stride, n_tiles, H, Hkv, page_size, window, scale, bias_r1, bias_r2, part_o, part_ml,
-                              keep, sink, softcap, stream);
+                              keep, sink, softcap, dist, dist_len, mask_chunk, gate, ld_gate, stream);
   return ZK_EINVAL;
 }
 

@@ -7,10 +7,25 @@
 // yields a zero row (reference: row lookup of token_embd, src/model.zig:2352-2358).
 // With `pos_table` [max_pos, dim] a learned position vector is added, unscaled, in float32:
 // x[t, :] += float(pos_table[tok_pos[t], :]); a position outside the table sets *status = 3.
+// With `bg.rows` [buckets + 1, dim] the row (token before * mul_prev + token * mul_cur) mod buckets of that table is added,
+// unscaled; the last row for a sequence's first token.  The token before a step's first one is the sequence's state
+// prev[slot * prev_stride]; `single` (one token per sequence) also writes the token there, other steps leave that to
+// last_token_kernel, since another block may still have to read it.
+// The row goes to `copies` planes of [n, dim], one behind the other.
+struct Bigram {
+  const void* rows;
+  int buckets;
+  long long mul_prev, mul_cur;
+  int* prev;
+  long long prev_stride;
+  const int *tok_seq, *cu_q, *seq_slot;
+  int single;
+};
+
 template <typename T>
 __global__ void embed_kernel(const int* __restrict__ tokens, const T* __restrict__ table, float* __restrict__ x,
                              int dim, int vocab, float scale, int* status, const T* __restrict__ pos_table,
-                             const int* __restrict__ tok_pos, int max_pos) {
+                             const int* __restrict__ tok_pos, int max_pos, Bigram bg, int copies) {
   zk_let_next_start();
   zk_wait_prior();   // nothing of the kernels before is read, and nothing written, above this line
   const int t = blockIdx.x;
@@ -25,11 +40,38 @@ __global__ void embed_kernel(const int* __restrict__ tokens, const T* __restrict
     if (p >= 0 && p < max_pos) prow = pos_table + (size_t)p * dim;
     else if (threadIdx.x == 0) atomicExch(status, 3);
   }
+  const T* brow = nullptr;
+  if (bg.rows) {
+    const int b = bg.tok_seq[t];
+    int* st = bg.prev + (size_t)bg.seq_slot[b] * bg.prev_stride;
+    long long r = bg.buckets;
+    if (tok_pos[t] > 0) {
+      const int before = t > bg.cu_q[b] ? tokens[t - 1] : *st;
+      r = ((long long)before * bg.mul_prev + (long long)tok * bg.mul_cur) % bg.buckets;
+      if (r < 0) r += bg.buckets;
+    }
+    brow = (const T*)bg.rows + (size_t)r * dim;
+    if (bg.single) {
+      __syncthreads();                   // every thread has read the token before
+      if (threadIdx.x == 0) *st = tok;
+    }
+  }
+  const size_t plane = (size_t)gridDim.x * dim;
   for (int d = threadIdx.x; d < dim; d += blockDim.x) {
     float v = ok ? to_f32(row[d]) * scale : 0.f;
     if (prow) v += to_f32(prow[d]);
-    out[d] = v;
+    if (brow) v += to_f32(brow[d]);
+    for (int c = 0; c < copies; ++c) out[c * plane + d] = v;
   }
+}
+
+// prev[slot] <- the last token each sequence brought.
+__global__ void last_token_kernel(const int* __restrict__ tokens, const int* __restrict__ cu_q, const int* __restrict__ seq_slot,
+                                  int* __restrict__ prev, long long prev_stride, int n_seqs) {
+  zk_let_next_start();
+  zk_wait_prior();
+  const int b = blockIdx.x * blockDim.x + threadIdx.x;
+  if (b < n_seqs && cu_q[b + 1] > cu_q[b]) prev[(size_t)seq_slot[b] * prev_stride] = tokens[cu_q[b + 1] - 1];
 }
 
 // y[r, :] = (x[src(r), :] * rsqrt(mean(x^2) + eps)) * w   (src/model.zig:1166-1181: scale
@@ -486,6 +528,81 @@ __device__ __forceinline__ float zk_activate(float z, int kind) {
   }
 }
 
+// h[t, f] = act(gate_f) * up_f, act as numbered above (float32 arithmetic).  Rows of gu as in silu_mul_kernel.
+template <typename T>
+__global__ void gated_act_kernel(const T* __restrict__ gu, T* __restrict__ h, int n, int F, int il, int kind) {
+  zk_let_next_start();
+  zk_wait_prior();
+  const size_t total = (size_t)n * F;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = i / F, f = i - t * F;
+    const size_t gi = il ? (f / il) * 2 * il + f % il : f;
+    const size_t ui = il ? gi + il : F + f;
+    h[i] = from_f32<T>(zk_activate(to_f32(gu[t * 2 * F + gi]), kind) * to_f32(gu[t * 2 * F + ui]));
+  }
+}
+
+// u = y * silu(z) (float32 rows, z rows ld_z apart); every one of `parts` equal stretches of u is divided by its own root
+// mean square and multiplied by w: block (t, part) writes out[t, part's stretch] in the run dtype.  With W a multiple of 4,
+// at most 16 values a thread and aligned rows (VEC) u stays in registers; else it is computed twice.
+template <typename TO, bool VEC>
+__global__ void gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ z, int ld_z,
+                                        const float* __restrict__ w, TO* __restrict__ out, int inner, int W, float eps) {
+  __shared__ float scratch[32];
+  zk_let_next_start();
+  zk_wait_prior();
+  const int t = blockIdx.x, c0 = blockIdx.y * W;
+  const float* yr = y + (size_t)t * inner + c0;
+  const float* zr = z + (size_t)t * ld_z + c0;
+  TO* dst = out + (size_t)t * inner + c0;
+  float ss = 0.f;
+  if constexpr (VEC) {
+    float4 u[4];
+    const int n4 = W >> 2;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int d = threadIdx.x + i * blockDim.x;
+      u[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (d < n4) {
+        const float4 a = reinterpret_cast<const float4*>(yr)[d], g = reinterpret_cast<const float4*>(zr)[d];
+        u[i] = make_float4(a.x * (g.x / (1.0f + expf(-g.x))), a.y * (g.y / (1.0f + expf(-g.y))),
+                           a.z * (g.z / (1.0f + expf(-g.z))), a.w * (g.w / (1.0f + expf(-g.w))));
+      }
+      ss = fmaf(u[i].x, u[i].x, ss);
+      ss = fmaf(u[i].y, u[i].y, ss);
+      ss = fmaf(u[i].z, u[i].z, ss);
+      ss = fmaf(u[i].w, u[i].w, ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float scale = 1.0f / sqrtf(ss / (float)W + eps);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int d = threadIdx.x + i * blockDim.x;
+      if (d >= n4) continue;
+      const float4 wv = reinterpret_cast<const float4*>(w + c0)[d];
+      const float o0 = (u[i].x * scale) * wv.x, o1 = (u[i].y * scale) * wv.y, o2 = (u[i].z * scale) * wv.z,
+                  o3 = (u[i].w * scale) * wv.w;
+      if constexpr (sizeof(TO) == 4) {
+        reinterpret_cast<float4*>(dst)[d] = make_float4(o0, o1, o2, o3);
+      } else {
+        __nv_bfloat162 p[2] = {__floats2bfloat162_rn(o0, o1), __floats2bfloat162_rn(o2, o3)};
+        reinterpret_cast<uint2*>(dst)[d] = *reinterpret_cast<const uint2*>(p);
+      }
+    }
+  } else {
+    for (int d = threadIdx.x; d < W; d += blockDim.x) {
+      const float g = zr[d], u = yr[d] * (g / (1.0f + expf(-g)));
+      ss = fmaf(u, u, ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float scale = 1.0f / sqrtf(ss / (float)W + eps);
+    for (int d = threadIdx.x; d < W; d += blockDim.x) {
+      const float g = zr[d], u = yr[d] * (g / (1.0f + expf(-g)));
+      dst[d] = from_f32<TO>((u * scale) * w[c0 + d]);
+    }
+  }
+}
+
 template <typename T>
 __global__ void activation_kernel(const T* __restrict__ in, T* __restrict__ out, size_t total, int kind) {
   zk_let_next_start();
@@ -807,18 +924,25 @@ const char* zk_error_name(int code) {
 }
 
 int zk_embed(const int* tokens, const void* table, float* x, int n, int dim, int vocab, float scale, int dtype,
-             int* status, const void* pos_table, const int* tok_pos, int max_pos, cudaStream_t stream) {
+             int* status, const void* pos_table, const int* tok_pos, int max_pos, const void* bigram, int buckets,
+             long long mul_prev, long long mul_cur, int* prev, long long prev_stride, const int* tok_seq, const int* cu_q,
+             const int* seq_slot, int n_seqs, int single, int copies, cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (dim <= 0 || vocab <= 0 || (pos_table && (!tok_pos || max_pos <= 0))) return ZK_EINVAL;
+  if (dim <= 0 || vocab <= 0 || (pos_table && (!tok_pos || max_pos <= 0)) || copies < 1) return ZK_EINVAL;
+  if (bigram && (buckets <= 0 || !tok_pos || !prev || !tok_seq || !cu_q || !seq_slot || n_seqs <= 0)) return ZK_EINVAL;
+  const Bigram bg{bigram, buckets, mul_prev, mul_cur, prev, prev_stride, tok_seq, cu_q, seq_slot, single};
   const int threads = dim >= 1024 ? 256 : 128;
   if (dtype == ZK_F32)
     embed_kernel<float><<<n, threads, 0, stream>>>(tokens, (const float*)table, x, dim, vocab, scale, status,
-                                                   (const float*)pos_table, tok_pos, max_pos);
+                                                   (const float*)pos_table, tok_pos, max_pos, bg, copies);
   else if (dtype == ZK_BF16)
     embed_kernel<bf16><<<n, threads, 0, stream>>>(tokens, (const bf16*)table, x, dim, vocab, scale, status,
-                                                  (const bf16*)pos_table, tok_pos, max_pos);
+                                                  (const bf16*)pos_table, tok_pos, max_pos, bg, copies);
   else
     return ZK_EINVAL;
+  if (bigram && !single)
+    return zk_launch_dependent(last_token_kernel, dim3((n_seqs + 127) / 128), dim3(128), 0, stream, tokens, cu_q, seq_slot, prev,
+                               prev_stride, n_seqs);
   return ZK_LAUNCH_STATUS();
 }
 
@@ -905,6 +1029,38 @@ int zk_cast_rows(const float* in, void* out, long long total, int dtype, cudaStr
     return zk_launch_dependent(cast_rows_kernel<float>, dim3(blocks), dim3(threads), 0, stream, in, (float*)out, (size_t)total);
   if (dtype == ZK_BF16)
     return zk_launch_dependent(cast_rows_kernel<bf16>, dim3(blocks), dim3(threads), 0, stream, in, (bf16*)out, (size_t)total);
+  return ZK_EINVAL;
+}
+
+// gu [n, 2F] (layout `il` as for zk_silu_mul); kind as for zk_activation.
+int zk_gated_act(const void* gu, void* h, int n, int F, int il, int kind, int dtype, cudaStream_t stream) {
+  if (n <= 0 || F <= 0) return 0;
+  if (kind < 0 || kind > 4 || (il && F % il)) return ZK_EINVAL;
+  const size_t want = ((size_t)n * F + 255) / 256;
+  const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
+  if (dtype == ZK_F32)
+    return zk_launch_dependent(gated_act_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, (float*)h, n, F, il, kind);
+  if (dtype == ZK_BF16)
+    return zk_launch_dependent(gated_act_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)gu, (bf16*)h, n, F, il, kind);
+  return ZK_EINVAL;
+}
+
+// y float32 [n, inner], z float32 rows ld_z apart, w float32 [inner]; `parts` equal stretches normalised each on its own.
+int zk_gated_group_norm(const float* y, const float* z, int ld_z, const float* w, void* out, int n, int inner, int parts,
+                        float eps, int out_dtype, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (inner <= 0 || parts <= 0 || parts > 65535 || inner % parts || ld_z < inner) return ZK_EINVAL;
+  const int W = inner / parts;
+  int threads = 32;
+  while (threads < 512 && threads * 8 < W) threads <<= 1;
+  const bool aligned = (reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(w) |
+                        reinterpret_cast<uintptr_t>(out)) % 16 == 0;
+  const bool vec = W % 4 == 0 && ld_z % 4 == 0 && W <= 16 * threads && aligned;
+  const dim3 grid(n, parts);
+#define ZK_GGN(TO, V) zk_launch_dependent(gated_group_norm_kernel<TO, V>, grid, dim3(threads), 0, stream, y, z, ld_z, w, (TO*)out, inner, W, eps)
+  if (out_dtype == ZK_F32) return vec ? ZK_GGN(float, true) : ZK_GGN(float, false);
+  if (out_dtype == ZK_BF16) return vec ? ZK_GGN(bf16, true) : ZK_GGN(bf16, false);
+#undef ZK_GGN
   return ZK_EINVAL;
 }
 

@@ -41,7 +41,8 @@ struct Args {
   const float* bias;     // per weight row, or null
   const float* col_scale;  // EPI_PLAIN: per output column, applied to the sum (after bias and activation) before it is
                            // stored or added to C; or null
-  int act;               // EPI_PLAIN: 0 none, 1 the square of relu, applied to the sum (after the bias)
+  int act;               // EPI_PLAIN: 0 none, 1 the square of relu, applied to the sum (after the bias); EPI_SWIGLU: the gate's
+                         // activation, 0 silu, 1 relu
   int M, N, K, ldx, ldw, ldc, accumulate;
   // NORM_SCALED: X holds bfloat16(x * norm weight); ssq_in [M, ssq_parts] are partial sums of x^2
   const float* ssq_in;
@@ -394,7 +395,8 @@ __global__ void __launch_bounds__(WARPS * 32, skinny_min_blocks(WARPS, NT, EPI))
       const int n = n0 + i;
       if (m >= M || n >= N) continue;
       const float gate = total(i, m), up = total(16 + i, m);
-      C[(size_t)m * a.ldc + n] = __float2bfloat16_rn(gate / (1.0f + expf(-gate)) * up);
+      const float g = a.act ? fmaxf(gate, 0.f) : gate / (1.0f + expf(-gate));
+      C[(size_t)m * a.ldc + n] = __float2bfloat16_rn(g * up);
     }
   } else {  // EPI_CONV: token m is sequence m
     bf16* C = reinterpret_cast<bf16*>(a.C);
@@ -579,15 +581,15 @@ int zk_gemm_skinny(const void* X, const float* Xf, const float* norm_w, float ep
   return ZK_EINVAL;
 }
 
-// h[M, F] = silu(x W_gate^T) * (x W_up^T); W [2F, K] holds groups of 16 gate rows followed by their
+// h[M, F] = act(x W_gate^T) * (x W_up^T), act 0 silu, 1 relu; W [2F, K] holds groups of 16 gate rows followed by their
 // 16 up rows (F a multiple of 16); M <= 16.
 int zk_gemm_skinny_swiglu(const void* X, const float* Xf, const float* norm_w, float eps, const void* W, void* H,
-                          int M, int F, int K, int ldx, int ldw, int ldh, const float* ssq_in, int ssq_parts,
+                          int M, int F, int K, int ldx, int ldw, int ldh, const float* ssq_in, int ssq_parts, int act,
                           cudaStream_t stream) {
   if (M <= 0 || F <= 0) return 0;
   Args a{};
   a.X = (const bf16*)X; a.Xf = Xf; a.norm_w = norm_w; a.eps = eps; a.W = (const bf16*)W; a.C = H;
-  a.M = M; a.N = F; a.K = K; a.ldx = ldx; a.ldw = ldw; a.ldc = ldh;
+  a.M = M; a.N = F; a.K = K; a.ldx = ldx; a.ldw = ldw; a.ldc = ldh; a.act = act;
   a.ssq_in = Xf ? nullptr : ssq_in; a.ssq_parts = ssq_parts;
   if (ldh < F || F % 16 || check_common(a, 16)) return ZK_EINVAL;
   return dispatch_fused<2, EPI_SWIGLU>(a, stream);

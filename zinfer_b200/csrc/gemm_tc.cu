@@ -41,13 +41,15 @@ constexpr int BK = 64;           // k block: 64 bfloat16 = one 128-byte swizzle 
 constexpr int UMMA_K = 16;
 constexpr int THREADS = 192;     // producer warp, MMA warp, four epilogue warps
 
-// The gated unit of the fused epilogues: silu(g) * u, or with limit > 0 the clamped unit described in Params.
+// The gated unit of the fused epilogues: silu(g) * u, with limit > 0 the clamped unit described in Params, with limit < 0
+// relu(g) * u.
 __device__ __forceinline__ float glu_unit(float g, float u, float limit, float alpha) {
   if (limit > 0.f) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit) + 1.0f;
     return g / (1.0f + expf(-alpha * g)) * u;
   }
+  if (limit < 0.f) return fmaxf(g, 0.f) * u;
   return g / (1.0f + expf(-g)) * u;
 }
 

@@ -17,13 +17,25 @@
 // registers while the current sixteen are worked on, and go into the other half of a double buffer.  The order of every sum is fixed by the layout alone, so a
 // sequence cut into steps gives the same bits as the whole.
 //
-// The same kernel runs the recurrence of a retention layer (its KEYED form): a key projection in place of the gate and
-// one fixed decay per head, S_t = decay_h S_{t-1} + k_t v_t^T; retention_prepare_kernel rotates q and k and scales k first.
+// The same kernel runs two more recurrences.  KEYED: a retention layer's, a key projection in place of the gate and one
+// fixed decay per head, S_t = decay_h S_{t-1} + k_t v_t^T; retention_prepare_kernel rotates q and k and scales k first.
+// STEPPED: a state-space layer's (Mamba-2), whose step size dt_t > 0 per head and token sets both the decay and what enters,
+// S_t = exp(-exp(A_log_h) dt_t) S_{t-1} + dt_t k_t v_t^T, o_t = S_t^T q_t + skip_h v_t, with k and q shared by the heads of
+// a group; lane i of every warp turns the raw step size of a group's token i into dt = softplus(z + bias) and the decay.
 #include "common.cuh"
 #include <math.h>
 
 #define HG_R 8             // warps of a block, each with a stretch of the d channels
 #define HG_MAX_D 512
+
+enum { REC_GATED = 0, REC_KEYED = 1, REC_STEPPED = 2 };
+
+// Where a STEPPED recurrence's operands lie and its numbers per head.  Rows of the float32 input hold the values [H * e] at
+// column 0, the keys [groups * d] at off_k, the queries [groups * d] at off_q; z holds the raw step sizes, rows ld_z apart.
+struct Stepped {
+  const float *z, *dt_bias, *a_log, *skip;
+  int ld_z, off_k, off_q, heads_per_group;
+};
 
 // In place on the rows of qfv: q <- silu(q), f <- lower + (1 - lower) * sigmoid(f + bias); v is left alone.
 __global__ void hgrn2_gates_kernel(float* __restrict__ qfv, int ld, const float* __restrict__ f_bias,
@@ -80,13 +92,13 @@ __global__ void __launch_bounds__(256)
 }
 
 // DPT: channels per warp; TT: tokens staged at once (sixteen, or eight or four where more do not fit shared memory).
-// KEYED: the recurrence of a retention layer instead, S_t = decay_h S_{t-1} + k_t v_t^T with one fixed decay per head
+// REC_KEYED: the recurrence of a retention layer instead, S_t = decay_h S_{t-1} + k_t v_t^T with one fixed decay per head
 // (`decay` [H]); the row's second part then holds the keys k_t in place of the gates.
-template <int DPT, int TT, bool KEYED>
+template <int DPT, int TT, int REC>
 __global__ void __launch_bounds__(HG_R * 32)
     hgrn2_scan_kernel(const float* __restrict__ qfv, int ld, float* __restrict__ state, long long state_stride,
                       float* __restrict__ o, const int* __restrict__ cu_q, const int* __restrict__ seq_slot, int H, int d,
-                      int e, const float* __restrict__ decay) {
+                      int e, const float* __restrict__ decay, Stepped sp) {
   constexpr int DM = HG_R * DPT;                                     // channels the block covers, >= d
   constexpr int NL = (TT * DM + HG_R * 32 - 1) / (HG_R * 32);     // q (and f) values a thread fetches per group of tokens
   __shared__ __align__(16) float qs[2][TT][DM];
@@ -107,21 +119,25 @@ __global__ void __launch_bounds__(HG_R * 32)
   }
   zk_wait_prior();   // qfv is the kernel before's result
   const int t0 = cu_q[b], t1 = cu_q[b + 1];
-  const float dk = KEYED ? decay[h] : 0.f;
+  const float dk = REC == REC_KEYED ? decay[h] : 0.f;
+  const float skip = REC == REC_STEPPED ? sp.skip[h] : 0.f, dt_bias = REC == REC_STEPPED ? sp.dt_bias[h] : 0.f;
+  const float rate = REC == REC_STEPPED ? -expf(sp.a_log[h]) : 0.f;
   float* st = state + (size_t)seq_slot[b] * state_stride + (size_t)h * d * e;
   float S[DPT];
 #pragma unroll
   for (int k = 0; k < DPT; ++k) S[k] = (col && row0 + k < d) ? st[(size_t)(row0 + k) * e + c] : 0.f;
 
-  const int off_f = H * d, off_v = 2 * H * d;
+  const int head_q = REC == REC_STEPPED ? sp.off_q + h / sp.heads_per_group * d : h * d;       // columns of this head's q
+  const int off_f = REC == REC_STEPPED ? sp.off_k - sp.off_q : H * d, off_v = REC == REC_STEPPED ? 0 : 2 * H * d;
   float rq[NL], rf[NL], v_cur[TT], v_next[TT];
+  float rz = 0.f, lane_decay = 0.f, lane_dt = 0.f;      // REC_STEPPED: the raw step size, decay and dt of token `lane` of a group
   // where a thread's n-th value of a group comes from (relative to the group's first row) and goes to
   int src[NL], dst[NL];
 #pragma unroll
   for (int n = 0; n < NL; ++n) {
     const int idx = tid + n * HG_R * 32;
     const int tt = idx / d, i = idx - tt * d;
-    src[n] = tt < TT ? tt * ld + h * d + i : -1;
+    src[n] = tt < TT ? tt * ld + head_q + i : -1;
     dst[n] = tt * DM + i;
   }
   auto fetch = [&](int tb) {
@@ -136,6 +152,7 @@ __global__ void __launch_bounds__(HG_R * 32)
 #pragma unroll
     for (int tt = 0; tt < TT; ++tt)
       v_next[tt] = (col && tt < nt) ? base[(size_t)tt * ld + off_v + h * e + c] : 0.f;
+    if (REC == REC_STEPPED && lane < nt) rz = sp.z[(size_t)(tb + lane) * sp.ld_z + h];
   };
   auto stage = [&](int buf, int tb) {
     const int nt = min(TT, t1 - tb);
@@ -148,6 +165,11 @@ __global__ void __launch_bounds__(HG_R * 32)
     }
 #pragma unroll
     for (int tt = 0; tt < TT; ++tt) v_cur[tt] = v_next[tt];
+    if (REC == REC_STEPPED) {
+      const float z = rz + dt_bias;
+      lane_dt = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));      // softplus
+      lane_decay = expf(rate * lane_dt);
+    }
   };
 
   if (t0 < t1) {
@@ -161,8 +183,13 @@ __global__ void __launch_bounds__(HG_R * 32)
     const bool more = tb + TT < t1;
     if (more) fetch(tb + TT);       // under way while this group is worked on
     auto token = [&](int tt) {
-      const float v = v_cur[tt];
+      float v = v_cur[tt], keep = dk;
       float acc = 0.f;
+      if (REC == REC_STEPPED) {
+        if (warp == 0) acc = skip * v;
+        keep = __shfl_sync(0xffffffffu, lane_decay, tt);
+        v *= __shfl_sync(0xffffffffu, lane_dt, tt);
+      }
       if constexpr (DPT % 4 == 0) {
 #pragma unroll
         for (int k4 = 0; k4 < DPT; k4 += 4) {
@@ -171,7 +198,7 @@ __global__ void __launch_bounds__(HG_R * 32)
           const float ff[4] = {f4.x, f4.y, f4.z, f4.w}, qq[4] = {q4.x, q4.y, q4.z, q4.w};
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
-            if (KEYED) S[k4 + j] = fmaf(dk, S[k4 + j], ff[j] * v);               // decay S + k v
+            if (REC != REC_GATED) S[k4 + j] = fmaf(keep, S[k4 + j], ff[j] * v);   // decay S + k v
             else S[k4 + j] = fmaf(ff[j], S[k4 + j], fmaf(-ff[j], v, v));        // f S + (1 - f) v
             acc = fmaf(S[k4 + j], qq[j], acc);
           }
@@ -180,7 +207,7 @@ __global__ void __launch_bounds__(HG_R * 32)
 #pragma unroll
         for (int k = 0; k < DPT; ++k) {
           const float f = fs[buf][tt][row0 + k];
-          if (KEYED) S[k] = fmaf(dk, S[k], f * v);
+          if (REC != REC_GATED) S[k] = fmaf(keep, S[k], f * v);
           else S[k] = fmaf(f, S[k], fmaf(-f, v, v));
           acc = fmaf(S[k], qs[buf][tt][row0 + k], acc);
         }
@@ -240,8 +267,8 @@ int zk_hgrn2_scan(float* qfv, int ld, const float* f_bias, const float* lower, f
   }
   dim3 grid(n_seqs, H, (e + 31) / 32);
 #define ZK_HG(DP)                                                                                                    \
-  return zk_launch_dependent(hgrn2_scan_kernel<DP, (DP > 32 ? 4 : (DP > 16 ? 8 : 16)), false>, grid, dim3(HG_R * 32), 0, stream, (const float*)qfv, ld, \
-                             state, state_stride, o, cu_q, seq_slot, H, d, e, (const float*)nullptr)
+  return zk_launch_dependent(hgrn2_scan_kernel<DP, (DP > 32 ? 4 : (DP > 16 ? 8 : 16)), REC_GATED>, grid, dim3(HG_R * 32), 0, stream, (const float*)qfv, ld, \
+                             state, state_stride, o, cu_q, seq_slot, H, d, e, (const float*)nullptr, Stepped{})
   const int dpt = (d + HG_R - 1) / HG_R;
   if (dpt <= 1) ZK_HG(1);
   if (dpt <= 2) ZK_HG(2);
@@ -271,8 +298,8 @@ int zk_retention_scan(float* qkv, int ld, const float* decay, const float* inv_f
   }
   dim3 grid(n_seqs, H, (e + 31) / 32);
 #define ZK_RT(DP)                                                                                                    \
-  return zk_launch_dependent(hgrn2_scan_kernel<DP, (DP > 32 ? 4 : (DP > 16 ? 8 : 16)), true>, grid, dim3(HG_R * 32), 0, stream, (const float*)qkv, ld, \
-                             state, state_stride, o, cu_q, seq_slot, H, d, e, decay)
+  return zk_launch_dependent(hgrn2_scan_kernel<DP, (DP > 32 ? 4 : (DP > 16 ? 8 : 16)), REC_KEYED>, grid, dim3(HG_R * 32), 0, stream, (const float*)qkv, ld, \
+                             state, state_stride, o, cu_q, seq_slot, H, d, e, decay, Stepped{})
   const int dpt = (d + HG_R - 1) / HG_R;
   if (dpt <= 1) ZK_RT(1);
   if (dpt <= 2) ZK_RT(2);
@@ -282,6 +309,31 @@ int zk_retention_scan(float* qkv, int ld, const float* decay, const float* inv_f
   if (dpt <= 32) ZK_RT(32);
   ZK_RT(64);
 #undef ZK_RT
+}
+
+// State-space recurrence (Mamba-2): xbc float32 [n, >= H*e + 2*groups*d] with rows `ld` floats apart, a row [values (H*e) | keys
+// (groups*d) | queries (groups*d)]; z float32 [n, >= H] rows ld_z apart (raw step sizes); dt_bias, a_log, skip float32 [H]; state
+// (per slot [H, d, e]), o [n, H*e], cu_q, seq_slot as for zk_hgrn2_scan.  d: state channels, e: values per head.
+int zk_ssd_scan(const float* xbc, int ld, const float* z, int ld_z, const float* dt_bias, const float* a_log, const float* skip,
+                float* state, long long state_stride, float* o, const int* cu_q, const int* seq_slot, int n, int n_seqs, int H,
+                int groups, int d, int e, cudaStream_t stream) {
+  if (n_seqs <= 0 || n <= 0) return 0;
+  if (H <= 0 || groups <= 0 || H % groups || d <= 0 || e <= 0 || d > HG_MAX_D) return ZK_EINVAL;
+  if (ld < H * e + 2 * groups * d || ld_z < H || !z || !dt_bias || !a_log || !skip) return ZK_EINVAL;
+  const Stepped sp{z, dt_bias, a_log, skip, ld_z, H * e, H * e + groups * d, H / groups};
+  dim3 grid(n_seqs, H, (e + 31) / 32);
+#define ZK_SS(DP)                                                                                                    \
+  return zk_launch_dependent(hgrn2_scan_kernel<DP, (DP > 32 ? 4 : (DP > 16 ? 8 : 16)), REC_STEPPED>, grid, dim3(HG_R * 32), 0, stream, xbc, ld, \
+                             state, state_stride, o, cu_q, seq_slot, H, d, e, (const float*)nullptr, sp)
+  const int dpt = (d + HG_R - 1) / HG_R;
+  if (dpt <= 1) ZK_SS(1);
+  if (dpt <= 2) ZK_SS(2);
+  if (dpt <= 4) ZK_SS(4);
+  if (dpt <= 8) ZK_SS(8);
+  if (dpt <= 16) ZK_SS(16);
+  if (dpt <= 32) ZK_SS(32);
+  ZK_SS(64);
+#undef ZK_SS
 }
 
 }  // extern "C"

@@ -70,7 +70,8 @@ class StepContext:
     arrays tokens, tok_seq, tok_pos [n_tokens], cu_q [n_seqs + 1], seq_start, seq_slot [n_seqs];
     `status` (the device's status word), `sm_count`, and `host_tokens` (the ids on the host, or None).  `memo` keeps what parts derive from the
     batch's shape alone (tile tables and the like), so that equal parts derive it once a step; a
-    step that is recorded and replayed keeps its memo with the recording."""
+    step that is recorded and replayed keeps its memo with the recording.  `shared` holds what a part of this very step
+    leaves for a later one (the values of a layer that later layers mix into theirs)."""
 
     def __init__(self, dtype: torch.dtype, device, status: torch.Tensor, buf: torch.Tensor, n_tokens: int,
                  n_seqs: int, q_lens: Sequence[int], max_kv_len: int, memo: Optional[dict] = None,
@@ -95,6 +96,7 @@ class StepContext:
             o, size = lay[name]
             setattr(self, name, buf[o:o + size])
         self._memo: dict = {} if memo is None else memo
+        self.shared: dict = {}      # what one part of this step leaves for another (never kept beyond the step)
 
     def memo(self, key, make):
         """`make()` once per step (or recording) and key."""

@@ -138,6 +138,8 @@ class Engine:
                                   self.dtype, self.device)
         self.calls = [CallContext(c, call.layer, self.cache.kv_view(c), self.cache.writes_kv(c),
                                   self.cache.state_view(c)) for c, call in enumerate(model.schedule)]
+        # an embedding with per-sequence state has the cache's last entry, behind the schedule's
+        self.embedding_state = self.cache.state_view(len(self.calls)) if model.embedding.state_request() is not None else None
         self.status = kernels.status_word(self.device)      # one status word per device, shared by all kernels
         self.sm_count = kernels.sm_count(self.device)
         self.vocab_size = cfg.vocab_size
@@ -247,9 +249,9 @@ class Engine:
         cu = np.concatenate([[0], np.cumsum(lens)])
         rows = [int(cu[b]) + int(i) for b, w in enumerate(want) for i in w]
         if rows == list(range(n)):      # every row in order (a step of single tokens): no gather before the head
-            return self.model.forward(ctx, self.calls, None, want_all=True)
+            return self.model.forward(ctx, self.calls, None, want_all=True, embedding_state=self.embedding_state)
         want_rows = torch.tensor(rows, dtype=torch.int32).pin_memory().to(self.device, non_blocking=True) if rows else None
-        return self.model.forward(ctx, self.calls, want_rows)
+        return self.model.forward(ctx, self.calls, want_rows, embedding_state=self.embedding_state)
 
     # ------------------------------------------------------------------ single-token steps
 
@@ -304,7 +306,7 @@ class Engine:
         """The step's kernels: the model, then the arg-max of every row of logits.  The arg-max goes to
         `batch.greedy` (with the status word behind it: one small copy brings both to the host) and into
         the token slots of the batch description, where the next step of the same batch finds it."""
-        self.model.forward(ctx, self.calls, None, want_all=True, out=batch.logits)
+        self.model.forward(ctx, self.calls, None, want_all=True, out=batch.logits, embedding_state=self.embedding_state)
         kernels.argmax(batch.logits, out=batch.greedy, feed=batch.meta_dev[:batch.n_seqs], status=self.status,
                        ring=batch.ring, ring_pos=batch.ring_pos)
 

@@ -24,7 +24,7 @@ _C = {"p": ctypes.c_void_p, "i": ctypes.c_int, "f": ctypes.c_float, "l": ctypes.
 # pointer of every launcher is the stream
 _SIGNATURES = {
     "elementwise": {
-        "zk_embed": "pppiiifip" + "ppi" + "p",
+        "zk_embed": "pppiiifip" + "ppi" + "pillplpppiii" + "p",
         "zk_rmsnorm": "ppppiifip",
         "zk_silu_mul": "ppiiiip",
         "zk_fill_normal": "pllffip",
@@ -44,6 +44,13 @@ _SIGNATURES = {
         "zk_layernorm": "pppppiifip",
         "zk_value_gate": "ppiiiiiip",
         "zk_unit_norm_gate": "ppipiiifip",
+        "zk_gated_act": "ppiiiiip",
+        "zk_gated_group_norm": "ppippiiifip",
+    },
+    "streams": {
+        "zk_stream_norm": "plpippp" + "iifip",
+        "zk_stream_step": "plpppippp" + "iifip",
+        "zk_stream_max": "",
     },
     "latent": {
         "zk_latent_prepare": "pppi" + "ppppppp" + "iiiiii" + "f" + "iii" + "ppp",
@@ -55,10 +62,11 @@ _SIGNATURES = {
         "zk_hgrn2_scan": "pippplpppiiiiip",
         "zk_hgrn2_max_dim": "",
         "zk_retention_scan": "pippifpplpppiiiiip",
+        "zk_ssd_scan": "pipipppplppp" + "iiiiii" + "p",
     },
     "seqconv": {
-        "zk_seqconv_forward": "ppppppp" + "iiiliiip",
-        "zk_seqconv_state_update": "ppppiiilp",
+        "zk_seqconv_forward": "ppppppp" + "iiiliii" + "ipi" + "p",
+        "zk_seqconv_state_update": "ppppiiilip",
         "zk_seqconv_max_taps": "",
     },
     "moe": {
@@ -74,7 +82,7 @@ _SIGNATURES = {
     },
     "gemm_skinny": {
         "zk_gemm_skinny": "pppfpppiiiiiiii" + "pippp" + "pi" + "p",
-        "zk_gemm_skinny_swiglu": "pppfppiiiiii" + "pi" + "p",
+        "zk_gemm_skinny_swiglu": "pppfppiiiiii" + "pi" + "i" + "p",
         "zk_gemm_skinny_conv": "pppfppppppp" + "iiiiiiil" + "pi" + "p",
         "zk_gemm_skinny_max_m": "",
         "zk_gemm_skinny_fused_max_m": "",
@@ -99,7 +107,7 @@ _SIGNATURES = {
         "zk_attn_decode_noalloc_bytes": "iiii",
     },
     "attention_prefill": {
-        "zk_attn_prefill": "pppppppppp" + "iiiiiiiif" + "pp" + "pp" + "ip" + "f" + "p",
+        "zk_attn_prefill": "pppppppppp" + "iiiiiiiif" + "pp" + "pp" + "ip" + "f" + "piipi" + "p",
         "zk_attn_prefill_takes": "iiii",
         "zk_attn_prefill_tile_tokens": "ii",
     },
@@ -113,7 +121,7 @@ _SIGNATURES = {
         "zk_attn_decode_latent_takes": "iiii",
     },
     "attention_decode_tc": {
-        "zk_attn_decode_tc": "pppppppppiiiiiiifii" + "pp" + "i" + "ip" + "f" + "p",
+        "zk_attn_decode_tc": "pppppppppiiiiiiifii" + "pp" + "i" + "ip" + "f" + "piipi" + "p",
         "zk_attn_decode_tc_takes": "iiii",
     },
     "sampling": {
@@ -125,11 +133,11 @@ _SIGNATURES = {
         "zk_sample": "piififfffip" + "lpp" + "pp",
     },
     "attention": {
-        "zk_qk_prepare": "pppppppppppp" + "iiiiiiifiiip" + "ii" + "fi" + "p",
+        "zk_qk_prepare": "pppppppppppp" + "iiiiiiifiiip" + "ii" + "fi" + "ipiiif" + "p",
         "zk_qk_prepare_span": "pipppppppppiiiiiifiiip" + "pi" + "p",
-        "zk_attn_fwd": "pppppp" + "pppppp" + "iiiiiiiifiiiii" + "ippi" + "ipi" + "f" + "p",
+        "zk_attn_fwd": "pppppp" + "pppppp" + "iiiiiiiifiiiii" + "ippi" + "ipi" + "f" + "piipi" + "p",
         "zk_attn_merge_talk": "ppppiiiiiip",
-        "zk_attn_merge": "pppiiii" + "pi" + "p",
+        "zk_attn_merge": "pppiiii" + "pi" + "pi" + "p",
         "zk_attn_rows_per_block": "",
         "zk_attn_max_head_dim": "",
     },
@@ -237,10 +245,15 @@ def dtype_code(dtype: torch.dtype) -> int:
 
 def embed(tokens: torch.Tensor, table: torch.Tensor, status: torch.Tensor, scale: float = 1.0,
           pos_table: Optional[torch.Tensor] = None, tok_pos: Optional[torch.Tensor] = None,
-          out: Optional[torch.Tensor] = None) -> torch.Tensor:
+          out: Optional[torch.Tensor] = None, bigram: Optional[tuple] = None, batch: Optional[tuple] = None,
+          prev: Optional[torch.Tensor] = None, single_token: bool = False, copies: int = 1) -> torch.Tensor:
     """x[t] = float32(table[tokens[t]]) * scale; bad ids set status to 1.  With `pos_table`
     [positions, dim] (the table's dtype) the row pos_table[tok_pos[t]] is added, unscaled; a position
-    outside it sets status to 3.  `out`: float32 [n, dim] to write into."""
+    outside it sets status to 3.  `out`: float32 [n, dim] to write into.
+    `bigram` = (rows [buckets + 1, dim], mul_prev, mul_cur): the row (token before * mul_prev + token * mul_cur) mod buckets
+    is added, unscaled, the last row for a sequence's first token; `batch` = (tok_seq, tok_pos, cu_q, seq_slot, n_seqs) then
+    describes the batch and `prev` int32 [slots, 1] holds every sequence's last token, which moves on.  `copies` > 1: the rows go
+    to that many planes, [copies, n, dim]."""
     _need(tokens, "tokens", torch.int32)
     _need(table, "table", (torch.float32, torch.bfloat16), (None, None))
     _need(status, "status", torch.int32)
@@ -250,12 +263,25 @@ def embed(tokens: torch.Tensor, table: torch.Tensor, status: torch.Tensor, scale
         _need(pos_table, "pos_table", table.dtype, (None, dim))
         _need(tok_pos, "tok_pos", torch.int32, (n,))
         max_pos = pos_table.shape[0]
+    rows = buckets = tok_seq = cu_q = seq_slot = None
+    mul_prev = mul_cur = n_seqs = 0
+    if bigram is not None:
+        rows, mul_prev, mul_cur = bigram
+        _need(rows, "bigram table", table.dtype, (None, dim))
+        buckets = rows.shape[0] - 1
+        tok_seq, tok_pos, cu_q, seq_slot, n_seqs = batch
+        for t, nm in ((tok_seq, "tok_seq"), (tok_pos, "tok_pos"), (cu_q, "cu_q"), (seq_slot, "seq_slot")):
+            _need(t, nm, torch.int32)
+        _need(prev, "prev", torch.int32, (None, 1), contiguous=False)
+    shape = (n, dim) if copies == 1 else (copies, n, dim)
     if out is None:
-        out = torch.empty((n, dim), dtype=torch.float32, device=table.device)
-    _need(out, "out", torch.float32, (n, dim))
+        out = torch.empty(shape, dtype=torch.float32, device=table.device)
+    _need(out, "out", torch.float32, shape)
     _check(_fn("elementwise", "zk_embed")(_ptr(tokens), _ptr(table), _ptr(out), n, dim, vocab, scale,
                                           dtype_code(table.dtype), _ptr(status), _ptr(pos_table), _ptr(tok_pos), max_pos,
-                                          _stream()), "embed")
+                                          _ptr(rows), buckets or 0, int(mul_prev), int(mul_cur), _ptr(prev),
+                                          prev.stride(0) if prev is not None else 0, _ptr(tok_seq), _ptr(cu_q), _ptr(seq_slot),
+                                          int(n_seqs), 1 if single_token else 0, int(copies), _stream()), "embed")
     return out
 
 
@@ -453,6 +479,30 @@ def retention_scan(qkv: torch.Tensor, decay: torch.Tensor, inv_freq: Optional[to
     return o
 
 
+def ssd_scan(xbc: torch.Tensor, z: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor,
+             state: torch.Tensor, cu_q, seq_slot, n_seqs: int, n_heads: int, groups: int, dim: int, value_dim: int) -> torch.Tensor:
+    """Per head, with dt = softplus(z + dt_bias): S_t = exp(-exp(a_log) dt_t) S_{t-1} + dt_t k_t v_t^T, o_t = S_t^T q_t + skip v_t
+    over each sequence's tokens, from the state the step before left to the state this one leaves.  xbc float32
+    [n, H*e + 2*groups*d], a row [v | k | q], k and q shared by the H / groups heads of a group; z float32 [n, H], row stride
+    used; state float32 [slots, H*d*e] (rows `state.stride(0)` apart); returns o float32 [n, H*e]."""
+    H, G, d, e = n_heads, groups, dim, value_dim
+    _need(xbc, "xbc", torch.float32, (None, H * e + 2 * G * d))
+    n = xbc.shape[0]
+    _need(z, "z", torch.float32, (n, H), contiguous=False)
+    for t, nm in ((dt_bias, "dt_bias"), (a_log, "a_log"), (skip, "skip")):
+        _need(t, nm, torch.float32, (H,))
+    _need(state, "state", torch.float32, contiguous=False)
+    if state.dim() != 2 or state.shape[1] != H * d * e or state.stride(1) != 1 or z.stride(1) != 1:
+        raise KernelError(f"ssd_scan: state {tuple(state.shape)} must hold {H * d * e} values per slot")
+    for t, nm in ((cu_q, "cu_q"), (seq_slot, "seq_slot")):
+        _need(t, nm, torch.int32)
+    o = torch.empty((n, H * e), dtype=torch.float32, device=xbc.device)
+    _check(_fn("hgrn2", "zk_ssd_scan")(_ptr(xbc), xbc.stride(0), _ptr(z), z.stride(0), _ptr(dt_bias), _ptr(a_log), _ptr(skip),
+                                       _ptr(state), state.stride(0), _ptr(o), _ptr(cu_q), _ptr(seq_slot), n, n_seqs, H, G, d, e,
+                                       _stream()), "ssd_scan")
+    return o
+
+
 # ------------------------------------------------------------------------------- convolution over time on a mixer's input
 
 def seqconv_max_taps() -> int:
@@ -460,25 +510,31 @@ def seqconv_max_taps() -> int:
 
 
 def seqconv(x: torch.Tensor, state: torch.Tensor, taps: torch.Tensor, tok_seq, cu_q, seq_slot, n_seqs: int,
-            out_dtype: torch.dtype, residual: bool = True, single_token: bool = False) -> torch.Tensor:
+            out_dtype: torch.dtype, residual: bool = True, single_token: bool = False, bias: Optional[torch.Tensor] = None,
+            silu: bool = False) -> torch.Tensor:
     """h_t = (x_t +) sum_j taps[j] * x_{t - (K-1) + j} per channel over each sequence's tokens, the
     K-1 inputs before the step taken from `state` [slots, K-1, D], which then moves on to the step's
-    last inputs.  x float32 [n, D] packed; taps float32 [K, D]; h [n, D] in `out_dtype`."""
-    _need(x, "x", torch.float32, (None, None))
+    last inputs.  x float32 [n, D] (row stride used); taps float32 [K, D]; h [n, D] in `out_dtype`.  `bias` float32 [D] is added
+    last; `silu`: silu(h) in place of h."""
+    _need(x, "x", torch.float32, (None, None), contiguous=False)
     n, D = x.shape
     _need(taps, "taps", torch.float32, (None, D))
     K = taps.shape[0]
-    _need(state, "state", torch.float32, (None, K - 1, D))
+    _need(state, "state", torch.float32, (None, K - 1, D), contiguous=False)
+    if x.stride(1) != 1 or (K > 1 and (state.stride(2) != 1 or state.stride(1) != D)):
+        raise KernelError("seqconv: the values of a row must lie side by side, and so must a slot's rows of state")
+    if bias is not None:
+        _need(bias, "bias", torch.float32, (D,))
     for t, nm in ((tok_seq, "tok_seq"), (cu_q, "cu_q"), (seq_slot, "seq_slot")):
         _need(t, nm, torch.int32)
     h = torch.empty((n, D), dtype=out_dtype, device=x.device)
     _check(_fn("seqconv", "zk_seqconv_forward")(_ptr(x), _ptr(state), _ptr(taps), _ptr(tok_seq), _ptr(cu_q),
                                                 _ptr(seq_slot), _ptr(h), n, D, K, state.stride(0),
                                                 1 if residual else 0, 1 if single_token else 0, dtype_code(out_dtype),
-                                                _stream()), "seqconv")
+                                                x.stride(0), _ptr(bias), 1 if silu else 0, _stream()), "seqconv")
     if not single_token and K > 1:
         _check(_fn("seqconv", "zk_seqconv_state_update")(_ptr(x), _ptr(state), _ptr(cu_q), _ptr(seq_slot), n_seqs, D, K,
-                                                         state.stride(0), _stream()), "seqconv state")
+                                                         state.stride(0), x.stride(0), _stream()), "seqconv state")
     return h
 
 
@@ -588,6 +644,76 @@ def silu_mul(gu: torch.Tensor, interleave: int = 0) -> torch.Tensor:
     return h
 
 
+def gated_act(gu: torch.Tensor, kind: str, interleave: int = 0) -> torch.Tensor:
+    """h = act(gate) * up for gu [n, 2F] laid out as for `silu_mul`; kind one of ACTIVATIONS, float32 arithmetic."""
+    _need(gu, "gu", (torch.float32, torch.bfloat16), (None, None))
+    n, F2 = gu.shape
+    h = torch.empty((n, F2 // 2), dtype=gu.dtype, device=gu.device)
+    _check(_fn("elementwise", "zk_gated_act")(_ptr(gu), _ptr(h), n, F2 // 2, int(interleave), ACTIVATIONS[kind], dtype_code(gu.dtype),
+                                              _stream()), "gated_act")
+    return h
+
+
+def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, parts: int, eps: float,
+                     out_dtype: torch.dtype) -> torch.Tensor:
+    """u = y * silu(z); every one of `parts` equal stretches of a row of u is divided by its own root mean square; times
+    `weight`.  y float32 [n, inner]; z float32 [n, inner], row stride used; out [n, inner] in `out_dtype`."""
+    _need(y, "y", torch.float32, (None, None))
+    n, inner = y.shape
+    _need(z, "z", torch.float32, (n, inner), contiguous=False)
+    _need(weight, "weight", torch.float32, (inner,))
+    if parts <= 0 or inner % parts or z.stride(1) != 1:
+        raise KernelError(f"gated_group_norm: {inner} values cannot be cut into {parts} equal parts")
+    out = torch.empty((n, inner), dtype=out_dtype, device=y.device)
+    _check(_fn("elementwise", "zk_gated_group_norm")(_ptr(y), _ptr(z), z.stride(0), _ptr(weight), _ptr(out), n, inner, int(parts),
+                                                     eps, dtype_code(out_dtype), _stream()), "gated_group_norm")
+    return out
+
+
+# ------------------------------------------------------------------------------- residual streams
+
+def stream_max() -> int:
+    return _constant("streams", "zk_stream_max")
+
+
+def stream_norm(x: torch.Tensor, read: Optional[torch.Tensor], weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
+                rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """RMSNorm of u = sum_s read[s] x[s] (read None: the plain sum) for float32 streams x [S, n, D], all rows or those listed."""
+    _need(x, "x", torch.float32, (None, None, None))
+    S, n, D = x.shape
+    if read is not None:
+        _need(read, "read", torch.float32, (S,))
+    _need(weight, "weight", torch.float32, (D,))
+    n_out = n
+    if rows is not None:
+        _need(rows, "rows", torch.int32)
+        n_out = rows.numel()
+    y = torch.empty((n_out, D), dtype=out_dtype, device=x.device)
+    _check(_fn("streams", "zk_stream_norm")(_ptr(x), x.stride(0), _ptr(read), S, _ptr(rows), _ptr(weight), _ptr(y), n_out, D, eps,
+                                            dtype_code(out_dtype), _stream()), "stream_norm")
+    return y
+
+
+def stream_step(x: torch.Tensor, y: torch.Tensor, mix: torch.Tensor, out: torch.Tensor, read: Optional[torch.Tensor] = None,
+                weight: Optional[torch.Tensor] = None, eps: float = 0.0, out_dtype: torch.dtype = torch.float32):
+    """x[t] <- sum_s mix[s, t] x[s] + out[t] * y, in place on float32 streams x [S, n, D]; with `weight` the rows that
+    `stream_norm` would then make of the new streams are returned, from the same pass (else None)."""
+    _need(x, "x", torch.float32, (None, None, None))
+    S, n, D = x.shape
+    _need(y, "y", torch.float32, (n, D))
+    _need(mix, "mix", torch.float32, (S, S))
+    _need(out, "out", torch.float32, (S,))
+    h = None
+    if weight is not None:
+        _need(weight, "weight", torch.float32, (D,))
+        if read is not None:
+            _need(read, "read", torch.float32, (S,))
+        h = torch.empty((n, D), dtype=out_dtype, device=x.device)
+    _check(_fn("streams", "zk_stream_step")(_ptr(x), x.stride(0), _ptr(y), _ptr(mix), _ptr(out), S, _ptr(read), _ptr(weight), _ptr(h),
+                                            n, D, eps, dtype_code(out_dtype), _stream()), "stream_step")
+    return h
+
+
 def clamped_glu(gu: torch.Tensor, limit: float, alpha: float, interleave: int = 0) -> torch.Tensor:
     """h = g' * sigmoid(alpha * g') * (u' + 1) with g' = min(gate, limit), u' = clamp(up, -limit, limit), in float32
     arithmetic.  Rows of gu as in `silu_mul`."""
@@ -659,6 +785,7 @@ def status_word(device) -> torch.Tensor:
     return st["status"]
 
 
+GATED_EPILOGUES = ("silu", "relu")      # activations of the gate that the contractions' gated epilogues know
 GEMM_TC_SWAPPED_MAX_M = 64     # up to this many rows the weights take the 128-row side of the tiles
 
 
@@ -687,10 +814,10 @@ def gemm_tc_emits(a, out: Optional[torch.Tensor]) -> bool:
 def gemm_tc(a, w: torch.Tensor, out: Optional[torch.Tensor] = None, out_dtype=None,
             accumulate: bool = False, bias: Optional[torch.Tensor] = None, splits: int = 1,
             swiglu: bool = False, emit: Optional["NormEmit"] = None, col_scale: Optional[torch.Tensor] = None,
-            act: Optional[str] = None, glu_clamp: Optional[tuple] = None) -> torch.Tensor:
+            act: Optional[str] = None, glu_clamp: Optional[tuple] = None, glu_act: str = "silu") -> torch.Tensor:
     """out (+)= a @ w.T (+ bias) with TMA-fed tcgen05 MMAs and the accumulator in tensor memory.
     `glu_clamp` = (limit, alpha), with `swiglu`: the unit is min(g, limit) * sigmoid(alpha * min(g, limit)) *
-    (clamp(u, -limit, limit) + 1) in place of silu(g) * u.
+    (clamp(u, -limit, limit) + 1) in place of silu(g) * u.  `glu_act` "relu", with `swiglu`: relu(g) * u.
     `act` ("relu_squared") and `col_scale` (float32 [N]) as in `gemm_skinny`, where `gemm_tc_fuses` says so.
     More than 64 rows: persistent blocks on 256-wide tiles when N is a multiple of 256 (pairs of
     blocks with tcgen05.mma.cta_group::2 above 128 rows, TMA stores), else one 128 x 128 tile of
@@ -712,6 +839,9 @@ def gemm_tc(a, w: torch.Tensor, out: Optional[torch.Tensor] = None, out_dtype=No
         raise KernelError("gemm_tc: the SwiGLU epilogue needs N a multiple of 32, no bias and no accumulation")
     if glu_clamp is not None and (not swiglu or not glu_clamp[0] > 0):
         raise KernelError("gemm_tc: the clamped unit goes with the gated epilogue and a positive limit")
+    if glu_act not in GATED_EPILOGUES or (glu_act != "silu" and (not swiglu or glu_clamp is not None)):
+        raise KernelError(f"gemm_tc: no gated epilogue with the activation {glu_act!r} here")
+    glu_limit = float(glu_clamp[0]) if glu_clamp else (-1.0 if glu_act == "relu" else 0.0)     # how the kernel is told
     n_out = N // 2 if swiglu else N
     if out is None:
         if accumulate:
@@ -738,7 +868,7 @@ def gemm_tc(a, w: torch.Tensor, out: Optional[torch.Tensor] = None, out_dtype=No
                                         1 if swiglu else 0, ssq, ssq_parts, eps,
                                         _ptr(emit.weight) if emit else None, _ptr(emit.xw) if emit else None,
                                         _ptr(emit.ssq) if emit else None, _ptr(status_word(a.device)), _ptr(col_scale),
-                                        1 if act else 0, float(glu_clamp[0]) if glu_clamp else 0.0,
+                                        1 if act else 0, glu_limit,
                                         float(glu_clamp[1]) if glu_clamp else 0.0, _stream()),
            "gemm_tc")
     return out
@@ -936,9 +1066,11 @@ def gemm_skinny(a, w: torch.Tensor, out: Optional[torch.Tensor] = None, out_dtyp
     return out
 
 
-def gemm_skinny_swiglu(a, w_gate_up: torch.Tensor) -> torch.Tensor:
-    """h = silu(a W_gate^T) * (a W_up^T) in one kernel; w_gate_up [2F, K] holds groups of 16 gate
+def gemm_skinny_swiglu(a, w_gate_up: torch.Tensor, act: str = "silu") -> torch.Tensor:
+    """h = act(a W_gate^T) * (a W_up^T) (act one of GATED_EPILOGUES) in one kernel; w_gate_up [2F, K] holds groups of 16 gate
     rows followed by their 16 up rows."""
+    if act not in GATED_EPILOGUES:
+        raise KernelError(f"gemm_skinny_swiglu: no gated epilogue with the activation {act!r}")
     if not gemm_skinny_fused_takes(a, w_gate_up) or w_gate_up.shape[0] % 32:
         raise KernelError("gemm_skinny_swiglu: at most 16 rows, K a multiple of 8, 16-byte aligned rows")
     X, Xf, nw, eps, M, K, ldx, ssq, ssq_parts = _skinny_input(a)
@@ -946,7 +1078,7 @@ def gemm_skinny_swiglu(a, w_gate_up: torch.Tensor) -> torch.Tensor:
     h = torch.empty((M, F), dtype=torch.bfloat16, device=w_gate_up.device)
     _check(_fn("gemm_skinny", "zk_gemm_skinny_swiglu")(X, Xf, nw, eps, _ptr(w_gate_up), _ptr(h), M, F, K, ldx,
                                                        w_gate_up.stride(0), h.stride(0), ssq, ssq_parts,
-                                                       _stream()),
+                                                       GATED_EPILOGUES.index(act), _stream()),
            "gemm_skinny_swiglu")
     return h
 
@@ -1247,17 +1379,29 @@ def attn_max_head_dim() -> int:
 def qk_prepare(qkv, k_cache, v_cache, q_w, k_w, inv_freq, tok_seq, tok_pos, seq_slot, page_table, n_heads: int,
                n_kv: int, head_dim: int, n_rot: int, interleaved: bool, eps: float, status, write_kv: bool = True,
                value_dim: Optional[int] = None, unit_norm_after: bool = False,
-               query_temperature: Optional[tuple] = None):
+               query_temperature: Optional[tuple] = None, mix_values: Optional[tuple] = None):
     """Per-head RMSNorm of q and k (if weights are given), rotary encoding (if `inv_freq` is
     given), then with `unit_norm_after` q and k heads divided by their root mean square (no weight);
     q out as [n, H*hd], and k, v written to their pages.  k_cache is one layer's
     [pages, Hkv, page_size, hd], v_cache [pages, Hkv, page_size, value_dim (default hd)].
     `query_temperature` = (coef, every): the query at position p is multiplied, last of all, by
-    1 + coef * ln(floor((p + 1) / every) + 1)."""
+    1 + coef * ln(floor((p + 1) / every) + 1).
+    A row of qkv may hold more behind its values (row stride used).  `mix_values` = (first, share): value heads of the same
+    tokens, a tensor [n, Hkv, width <= value_dim] in qkv's dtype (strides used), mixed in before a value is cached,
+    v <- (1 - share) v + share first, in float32."""
     qt_coef, qt_every = (float(query_temperature[0]), int(query_temperature[1])) if query_temperature else (0.0, 0)
     vd = head_dim if value_dim is None else int(value_dim)
-    _need(qkv, "qkv", (torch.float32, torch.bfloat16), (None, (n_heads + n_kv) * head_dim + n_kv * vd))
+    _need(qkv, "qkv", (torch.float32, torch.bfloat16), (None, None), contiguous=False)
+    if qkv.shape[1] < (n_heads + n_kv) * head_dim + n_kv * vd or qkv.stride(1) != 1:
+        raise KernelError(f"qk_prepare: rows of {qkv.shape[1]} values hold no q, k and v of these heads")
     n = qkv.shape[0]
+    first, first_ld, first_hs, first_vd, share = None, 0, 0, 0, 0.0
+    if mix_values is not None:
+        first, share = mix_values
+        _need(first, "first values", qkv.dtype, (n, n_kv, None), contiguous=False)
+        first_ld, first_hs, first_vd = first.stride(0), first.stride(1), first.shape[2]
+        if first.stride(2) != 1 or first_vd > vd:
+            raise KernelError("qk_prepare: mixed values must lie side by side and be no wider than the heads'")
     _need(k_cache, "k_cache", qkv.dtype, (None, n_kv, None, head_dim))
     _need(v_cache, "v_cache", qkv.dtype, (None, n_kv, None, vd))
     page_size = k_cache.shape[2]
@@ -1275,7 +1419,8 @@ def qk_prepare(qkv, k_cache, v_cache, q_w, k_w, inv_freq, tok_seq, tok_pos, seq_
         _ptr(qkv), _ptr(q), None, _ptr(k_cache), _ptr(v_cache), _ptr(q_w), _ptr(k_w), _ptr(inv_freq), _ptr(tok_seq),
         _ptr(tok_pos), _ptr(seq_slot), _ptr(page_table), page_table.stride(0), n, n_heads, n_kv, head_dim, n_rot,
         1 if interleaved else 0, eps, page_size, 1 if write_kv else 0, dtype_code(qkv.dtype), _ptr(status), vd,
-        1 if unit_norm_after else 0, qt_coef, qt_every, _stream()),
+        1 if unit_norm_after else 0, qt_coef, qt_every, qkv.stride(0), _ptr(first), first_ld, first_hs, first_vd, float(share),
+        _stream()),
         "qk_prepare")
     return q
 
@@ -1323,7 +1468,7 @@ def qk_normed(qkv, q_w, k_w, n_heads: int, n_kv: int, head_dim: int, eps: float,
     _check(_fn("attention", "zk_qk_prepare")(
         _ptr(qkv), None, _ptr(dense), None, None, _ptr(q_w), _ptr(k_w), None, None, _ptr(tok_pos), None, None, 0,
         qkv.shape[0], n_heads, n_kv, head_dim, 0, 0, eps, 1, 0, dtype_code(qkv.dtype), _ptr(status), head_dim, 0, 0.0, 0,
-        _stream()),
+        qkv.shape[1], None, 0, 0, 0, 0.0, _stream()),
         "qk_normed")
     return dense
 
@@ -1358,7 +1503,7 @@ def _takes(lib: str, fn: str, n_heads: int, n_kv: int, head_dim: int, page_size:
 def attention_plan(dtype: torch.dtype, n_heads: int, n_kv: int, head_dim: int, page_size: int,
                    single_token: bool, window: int = 0, value_dim: Optional[int] = None,
                    biased: bool = False, talking: bool = False, extras: bool = False,
-                   kept_or_sink: bool = False, capped: bool = False) -> tuple[str, int]:
+                   kept_or_sink: bool = False, capped: bool = False, plain_only: bool = False) -> tuple[str, int]:
     """Which attention kernel runs for these sizes and how many tokens its query tiles hold:
     ("single_token_tc" | "single_token" | "prompt_tc5" | "prompt_tc" | "general", tokens per tile).
     Values of another width than the keys go to the general kernel; a distance bias on the scores is
@@ -1366,7 +1511,11 @@ def attention_plan(dtype: torch.dtype, n_heads: int, n_kv: int, head_dim: int, p
     are mixed across the heads after the softmax (`talking`) by those three and the tcgen05 prompt kernel.
     `kept_or_sink`: kept first tokens or a sink in the softmax, which the general kernel and the two mma.sync kernels
     take (without a bias or mixed weights); `extras`: values read from the key rows, the general kernel's; `capped`:
-    scores through a tanh cap, which the same three kernels take."""
+    scores through a tanh cap, which the same three kernels take; `plain_only`: something else that only those three take (a
+    table of distance biases, a mask in stretches, a gate per head), without mixed weights."""
+    capped = capped or plain_only
+    if plain_only and talking:
+        raise KernelError("attention: no kernel takes a distance table, stretches or a gate together with mixed weights")
     same_width = value_dim is None or value_dim == head_dim
     if extras or (kept_or_sink and (biased or talking)):
         return "general", attn_tile_shape(n_heads, n_kv)[0]
@@ -1388,12 +1537,17 @@ def attention(q, k_cache, v_cache, tile_seq, tile_q0, cu_q, seq_start, seq_slot,
               head_dim: int, scale: float, window: int = 0, num_splits: int = 1, split_keys: int = 0,
               single_token: bool = False, kind: Optional[str] = None, value_dim: Optional[int] = None,
               bias: Optional[tuple] = None, talk: Optional[torch.Tensor] = None, keep_first: int = 0,
-              sink: Optional[torch.Tensor] = None, values_in_keys: bool = False, softcap: float = 0.0) -> torch.Tensor:
+              sink: Optional[torch.Tensor] = None, values_in_keys: bool = False, softcap: float = 0.0,
+              distance_table: Optional[torch.Tensor] = None, chunk: int = 0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal grouped-query attention of a packed batch against the paged cache.
     `keep_first`: with a window, the first so many positions of a sequence stay visible to every later query.
     `sink` float32 [H]: exp(sink_h) is one more term of head h's softmax denominator (no key, no value, not scaled).
     `values_in_keys`: there is no value cache; a value row is the first `value_dim` entries of the key row.
     `softcap` > 0: a scaled score s becomes softcap * tanh(s / softcap) (the general kernel's and the two mma.sync kernels').
+    `distance_table` float32 [H, n]: table[h, min(i - j, n - 1)] is added to head h's scaled score of query position i and key
+    position j.  `chunk` > 0: a query sees only keys of its own stretch of `chunk` positions, counted from position 0 (the cuts
+    of the keys then lie at multiples of `split_keys` from the stretch's start).  `gate` [n, H] in q's dtype, row stride used:
+    head h's output is multiplied by sigmoid(gate[:, h]).  These three are the general kernel's and the two mma.sync kernels'.
     The last is the general kernel's; the first two also the two mma.sync kernels' ("prompt_tc", "single_token_tc").  With
     num_splits > 1 the keys are cut at multiples of `split_keys` and merged afterwards.
     `single_token` says that every sequence brings exactly one query (row b = sequence b); the
@@ -1434,6 +1588,21 @@ def attention(q, k_cache, v_cache, tile_seq, tile_q0, cu_q, seq_start, seq_slot,
     softcap = float(softcap or 0.0)
     if softcap > 0 and kind not in (None, "general", "prompt_tc", "single_token_tc"):
         raise KernelError(f"attention: the '{kind}' kernel caps no scores")
+    dist_len, ld_gate = 0, 0
+    plain_only = distance_table is not None or chunk > 0 or gate is not None
+    if plain_only and (talk is not None or kind not in (None, "general", "prompt_tc", "single_token_tc")):
+        raise KernelError(f"attention: the '{kind}' kernel takes no distance table, no stretches and no gate")
+    if plain_only and kind is None:
+        kind = "general"
+    if distance_table is not None:
+        _need(distance_table, "distance table", torch.float32, (n_heads, None))
+        dist_len = distance_table.shape[1]
+    if gate is not None:
+        _need(gate, "gate", q.dtype, (n, n_heads), contiguous=False)
+        if gate.stride(1) != 1:
+            raise KernelError("attention: a token's gate logits must lie side by side")
+        ld_gate = gate.stride(0)
+    more = (_ptr(distance_table), dist_len, int(chunk), _ptr(gate), ld_gate)
     if vd != head_dim and kind not in (None, "general"):
         raise KernelError(f"attention: the '{kind}' kernel takes no value width of its own")
     if bias is not None and kind not in (None, "general", "prompt_tc", "single_token_tc"):
@@ -1477,7 +1646,7 @@ def attention(q, k_cache, v_cache, tile_seq, tile_q0, cu_q, seq_start, seq_slot,
             _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(tile_seq), _ptr(tile_q0), _ptr(cu_q),
             _ptr(seq_start), _ptr(seq_slot), _ptr(page_table), page_table.stride(0), n_tiles, n_heads, n_kv, head_dim,
             head_dim, page_size, window, scale, r1, r2, _ptr(part_o) if talk is not None else None,
-            _ptr(part_ml) if talk is not None else None, int(keep_first), _ptr(sink), softcap, _stream()),
+            _ptr(part_ml) if talk is not None else None, int(keep_first), _ptr(sink), softcap, *more, _stream()),
             "attention (prompt, tensor cores)")
         return out if talk is None else _merge_talk(part_o, part_ml, talk, out, n, n_heads, n_kv, vd, 1)
     if (single_token and kind in (None, "single_token_tc") and q.dtype == torch.bfloat16
@@ -1485,14 +1654,15 @@ def attention(q, k_cache, v_cache, tile_seq, tile_q0, cu_q, seq_start, seq_slot,
         _check(_fn("attention_decode_tc", "zk_attn_decode_tc")(
             _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(part_o), _ptr(part_ml), _ptr(seq_start),
             _ptr(seq_slot), _ptr(page_table), page_table.stride(0), n, n_heads, n_kv, head_dim, page_size, window,
-            scale, num_splits, split_keys, r1, r2, 1 if talk is not None else 0, int(keep_first), _ptr(sink), softcap,
+            scale, num_splits, split_keys, r1, r2, 1 if talk is not None else 0, int(keep_first), _ptr(sink), softcap, *more,
             _stream()),
             "attention (single token, tensor cores)")
         if talk is not None:
             return _merge_talk(part_o, part_ml, talk, out, n, n_heads, n_kv, vd, num_splits)
         if num_splits > 1:
             _check(_fn("attention", "zk_attn_merge")(_ptr(part_o), _ptr(part_ml), _ptr(out), n * n_heads, head_dim,
-                                                     num_splits, dtype_code(q.dtype), _ptr(sink), n_heads, _stream()), "attention merge")
+                                                     num_splits, dtype_code(q.dtype), _ptr(sink), n_heads, _ptr(gate), ld_gate,
+                                                     _stream()), "attention merge")
         return out
     if kind == "single_token_tc":
         raise KernelError("attention: the tensor-core single-token kernel does not take these sizes")
@@ -1504,20 +1674,20 @@ def attention(q, k_cache, v_cache, tile_seq, tile_q0, cu_q, seq_start, seq_slot,
             scale, num_splits, split_keys, _stream()), "attention (single token)")
         if num_splits > 1:
             _check(_fn("attention", "zk_attn_merge")(_ptr(part_o), _ptr(part_ml), _ptr(out), n * n_heads, head_dim,
-                                                     num_splits, dtype_code(q.dtype), None, n_heads, _stream()), "attention merge")
+                                                     num_splits, dtype_code(q.dtype), None, n_heads, None, 0, _stream()), "attention merge")
         return out
     _check(_fn("attention", "zk_attn_fwd")(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(part_o), _ptr(part_ml), _ptr(tile_seq), _ptr(tile_q0),
         _ptr(cu_q), _ptr(seq_start), _ptr(seq_slot), _ptr(page_table), page_table.stride(0), n_tiles, n, n_heads, n_kv,
         head_dim, page_size, window, scale, bq, gc, num_splits, split_keys, dtype_code(q.dtype), vd, r1, r2,
-        1 if talk is not None else 0, int(keep_first), _ptr(sink), 1 if values_in_keys else 0, softcap, _stream()),
+        1 if talk is not None else 0, int(keep_first), _ptr(sink), 1 if values_in_keys else 0, softcap, *more, _stream()),
         "attention")
     if talk is not None:
         return _merge_talk(part_o, part_ml, talk, out, n, n_heads, n_kv, vd, num_splits)
     if num_splits > 1:
         _check(_fn("attention", "zk_attn_merge")(_ptr(part_o), _ptr(part_ml), _ptr(out), n * n_heads, vd,
-                                                 num_splits, dtype_code(q.dtype), _ptr(sink), n_heads, _stream()),
-               "attention merge")
+                                                 num_splits, dtype_code(q.dtype), _ptr(sink), n_heads, _ptr(gate), ld_gate,
+                                                 _stream()), "attention merge")
     return out
 
 
@@ -1552,7 +1722,7 @@ def attention_step_rows(q, k_rows, v_rows, tile_seq, tile_q0, cu_q, seq_start, s
     _check(_fn("attention_prefill", "zk_attn_prefill")(
         _ptr(q), _ptr(k_rows), _ptr(v_rows), _ptr(out), _ptr(tile_seq), _ptr(tile_q0), _ptr(cu_q), _ptr(seq_start),
         _ptr(seq_page0), None, 0, tile_seq.numel(), n_heads, n_heads, hd, vd, page_size, 0, scale, None, None, None, None,
-        0, _ptr(sink), 0.0, _stream()), "attention (prompt, a step's own rows)")
+        0, _ptr(sink), 0.0, None, 0, 0, None, 0, _stream()), "attention (prompt, a step's own rows)")
     return out
 
 
@@ -1591,7 +1761,7 @@ def attention_latent_single(q, cache, seq_start, seq_slot, page_table, n_heads: 
         "attention (single token, latent rows)")
     if part_o is not None:
         _check(_fn("attention", "zk_attn_merge")(_ptr(part_o), _ptr(part_ml), _ptr(out), n * n_heads, value_dim, num_splits,
-                                                 dtype_code(q.dtype), _ptr(sink), n_heads, _stream()), "attention merge")
+                                                 dtype_code(q.dtype), _ptr(sink), n_heads, None, 0, _stream()), "attention merge")
     return out
 
 

@@ -5,3 +5,4 @@ from . import ponusun  # noqa: F401  (registers Ponusun)
 from . import zosurax  # noqa: F401  (registers Zosurax)
 from . import kerotar  # noqa: F401  (registers Kerotar)
 from . import pirisun  # noqa: F401  (registers Pirisun)
+from . import varolorn  # noqa: F401  (registers Varolorn)

@@ -82,22 +82,26 @@ class Model:
         for call in self.schedule:
             mixer = self.layers[call.layer].mixer
             specs.append(CallCacheSpec(kv=mixer.kv_request(), kv_owner=call.cache_of, state=mixer.state_request()))
+        if self.embedding.state_request() is not None:      # behind the schedule's entries
+            specs.append(CallCacheSpec(state=self.embedding.state_request()))
         return specs
 
     # ------------------------------------------------------------------ forward
     def forward(self, ctx, calls, want_rows: Optional[torch.Tensor], want_all: bool = False,
-                out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                out: Optional[torch.Tensor] = None, embedding_state: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
         """Runs the step's tokens through every schedule entry; returns float32 logits of the rows
         listed in `want_rows` (row indices into the packed tokens), of every row with `want_all`
         (written into `out` if given), or None when none is wanted.  Only wanted rows meet the
-        final norm and the head (src/model.zig:2482-2490)."""
+        final norm and the head (src/model.zig:2482-2490).  `embedding_state`: the per-sequence state the embedding asked
+        for.  A model of several residual streams has rows [streams, tokens, width] between its embedding and its final
+        norm; its blocks and norms know."""
         mix = self.depth_mix
         if mix is not None:
             planes = mix.planes(ctx, len(calls), self.embedding.dim)
-            self.embedding.forward(ctx, ctx.tokens, out=planes[0])
+            self.embedding.forward(ctx, ctx.tokens, out=planes[0], state=embedding_state)
             x = mix.first_input(planes)
         else:
-            x = self.embedding.forward(ctx, ctx.tokens)
+            x = self.embedding.forward(ctx, ctx.tokens, state=embedding_state)
         passes, x_emb = self.pass_input, None
         if passes is not None:
             if mix is not None:

@@ -5,11 +5,12 @@ from .attention import GqaAttention
 from .block import ParallelBlock, PreNormBlock, SublayerNormBlock
 from .depth import DepthAverage
 from .embedding import LMHead, TokenEmbedding
-from .feedforward import ActMlp, ClampedGLU, SwiGLU
+from .feedforward import ActMlp, ClampedGLU, ReluGLU, SwiGLU
 from .hgrn2 import Hgrn2
 from .latent import LatentAttention
 from .linear import linear
 from .loop import PassInput
+from .mamba2 import Mamba2
 from .moe import RoutedMoE, TableMoE
 from .norm import LayerNorm, RMSNorm
 from .pair import MixerPair
@@ -18,3 +19,4 @@ from .rope import RotaryEncoding
 from .seqconv import InputConv
 from .shift import TokenShift
 from .shortconv import ShortConv
+from .streams import StreamBlock, StreamNorm

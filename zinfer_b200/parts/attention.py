@@ -25,10 +25,22 @@ one more term of head h's softmax denominator, with no key and no value, and is 
 `query_temperature` = (coef, every): the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)
 (positions enter through that factor alone when there is no position encoding).  `softcap`: a scaled score s becomes
 softcap * tanh(s / softcap) before the softmax.
+`bias_names` = (q, k, v, out): vectors added in the four projections.
+`distance_rows` = (name, most): a learned number per (distance bucket, head), a tensor [buckets, heads] added to the scaled
+score of query position i and key position j in row `distance_buckets(...)[i - j]`: one row per distance up to half the
+buckets, then rows whose edges grow geometrically up to the distance `most`.  The number of buckets is the tensor's.
+`chunk`: a query sees only the keys of its own stretch of `chunk` positions, counted from the sequence's position 0; the cache
+gives the pages of earlier stretches back.
+`head_gate_name`: a matrix [heads, hidden]; head h's output is multiplied by sigmoid of row h's product with the mixer's
+input before the output projection.  Its rows are part of the one q/k/v contraction.
+`value_mix` = (name, is_first): layers that share their first layer's values.  The layer with is_first leaves the values of
+the step's tokens for the others (its own number of that name is loaded and unused); in every other layer a value becomes
+(1 - lambda) v + lambda v_first before it is cached, lambda the layer's number of that name.
 `pad_heads`: in a bfloat16 run, heads whose keys and values are not both 64 or both 128 wide (and at most 128) are
 padded at load to the next of those widths, with zero rows in W_q, W_k and W_v and zero columns in W_o, so that the
 tensor-core kernels take them; a padded entry adds nothing to a score and meets a zero column of W_o, the cache holds
-the padded rows.  Only without q/k norms (a norm would count the padding).
+the padded rows.  Per-head q/k norms count the padding; their weights and eps are scaled so that the result is the same
+(with P the padded width and d the head's: x / sqrt(ssq/P + eps d/P) * w sqrt(d/P) = x / sqrt(ssq/d + eps) * w).
 
 How the kernels are launched is decided here, not by the engine: the table of query tiles of a
 step, and for single-token steps the cut of a sequence's keys into chunks that separate blocks
@@ -38,14 +50,15 @@ src/model.zig:1941-1955).
 from __future__ import annotations
 
 import math
+from fractions import Fraction
 from typing import Optional, Sequence
 
 import numpy as np
 import torch
 
 from .. import kernels
-from .base import MIXERS, KVRequest, Mixer, PositionEncoding, WeightSpec
-from .linear import linear
+from .base import ANY_SIZE, MIXERS, KVRequest, Mixer, PositionEncoding, WeightSpec
+from .linear import linear, pad_rows
 
 
 def query_tiles(q_lens: Sequence[int], bq: int) -> np.ndarray:
@@ -72,17 +85,21 @@ def key_capacity(longest: int) -> int:
 CHUNK_ALIGN = 64            # chunk boundaries the single-token kernels take (their key tile)
 
 
-def key_chunks(n_seqs: int, n_kv_heads: int, longest: int, sm_count: int, split_keys: int = 0) -> tuple[int, int]:
+def key_chunks(n_seqs: int, n_kv_heads: int, longest: int, sm_count: int, split_keys: int = 0,
+               most: int = 0) -> tuple[int, int]:
     """(number of key chunks, keys per chunk) for single-token attention of `n_seqs` sequences up to
     `longest` tokens long.  The cuts lie at multiples of the chunk size, whatever the batch, and
     the chunks are added in order by the merge kernel, so a sequence's result does not depend on its
     neighbours.  split_keys > 0 fixes the chunk size; otherwise it is chosen so that about four
     blocks per SM have work, between 128 and 4096 keys: with unequal sequences a longer chunk
     leaves the SMs that drew a short sequence idle (64 sequences of 1K to 32K tokens on a B200:
-    3.90 ms a step with chunks of 16K keys, 3.27 ms with 4K)."""
+    3.90 ms a step with chunks of 16K keys, 3.27 ms with 4K).  most > 0: no query sees more keys than that, and the cuts
+    are counted from the first key it sees."""
     if longest <= 0:
         return 1, 0
     cap = key_capacity(longest)
+    if most > 0:
+        cap = min(cap, most)
     keys = split_keys
     if keys <= 0:
         blocks = max(1, n_seqs * n_kv_heads)
@@ -91,6 +108,27 @@ def key_chunks(n_seqs: int, n_kv_heads: int, longest: int, sm_count: int, split_
         keys = -(-keys // CHUNK_ALIGN) * CHUNK_ALIGN
     n = -(-cap // keys)
     return (n, keys) if n > 1 else (1, 0)
+
+
+def distance_buckets(rows: int, most, count: int) -> list[int]:
+    """The bucket of every distance 0 .. count - 1: n below rows/2, else min(rows - 1, h + floor(ln(n/h) / ln(most/h) * (rows - h)))
+    with h = rows/2.  The edges are found in whole numbers ((n/h)^(rows-h) >= (most/h)^k), so no rounding of a logarithm moves one."""
+    half = rows // 2
+    most = Fraction(most)
+    if rows < 2 or most <= half:
+        raise ValueError(f"distance buckets: {rows} rows and a largest distance of {most} leave no geometric buckets")
+    ratio, span = most / half, rows - half
+    out, k, step = [], 0, ratio           # k: bucket above half reached so far; step = ratio^(k + 1)
+    for n in range(count):
+        if n < half:
+            out.append(n)
+            continue
+        reached = Fraction(n, half) ** span
+        while k < span - 1 and reached >= step:
+            k += 1
+            step *= ratio
+        out.append(half + k)
+    return out
 
 
 class GqaAttention(Mixer):
@@ -103,7 +141,9 @@ class GqaAttention(Mixer):
                  qk_norm_span: str = "head", distance_bias: Optional[tuple[str, str]] = None, own_kv: bool = True,
                  unit_norm_after_rotation: bool = False, talk_name: Optional[str] = None, keep_first: int = 0,
                  sink_name: Optional[str] = None, query_temperature: Optional[tuple[float, int]] = None,
-                 softcap: Optional[float] = None, pad_heads: bool = False):
+                 softcap: Optional[float] = None, pad_heads: bool = False,
+                 bias_names: Optional[tuple[str, str, str, str]] = None, distance_rows: Optional[tuple[str, float]] = None,
+                 chunk: int = 0, head_gate_name: Optional[str] = None, value_mix: Optional[tuple[str, bool]] = None):
         """split_keys: keys per chunk of single-token attention, a multiple of 64 (0 = chosen per
         step from the batch and the GPU's size)."""
         if n_heads % n_kv_heads:
@@ -130,8 +170,23 @@ class GqaAttention(Mixer):
         if softcap is not None and (not softcap > 0 or talk_name is not None):
             raise ValueError("attention: a score cap must be positive and does not go with weights mixed across heads")
         self.softcap = 0.0 if softcap is None else float(softcap)
-        if pad_heads and (q_norm_name or k_norm_name or unit_norm_after_rotation or not own_kv or qk_norm_span == "all"):
-            raise ValueError("attention: padded heads go with key/value weights of the mixer's own and no q/k norms")
+        if pad_heads and (unit_norm_after_rotation or not own_kv or qk_norm_span == "all"
+                          or (position is not None and (q_norm_name or k_norm_name))):
+            raise ValueError("attention: padded heads go with key/value weights of the mixer's own and no norms but per-head ones "
+                             "without a position encoding")
+        newer = any(o is not None for o in (bias_names, distance_rows, head_gate_name, value_mix)) or chunk > 0
+        if newer and (self.span_prepare or talk_name is not None or not own_kv):
+            raise ValueError("attention: projection biases, distance buckets, chunks, a gate per head and mixed values go with "
+                             "per-head preparation, key/value weights of the mixer's own and weights not mixed across heads")
+        if chunk < 0 or (chunk > 0 and window > 0):
+            raise ValueError("attention: a mask in stretches and a window exclude each other")
+        if position is not None and newer and not hasattr(position, "rotary"):
+            raise ValueError("attention: these options take a rotation table or no position encoding")
+        self.bias_names, self.distance_rows, self.chunk = bias_names, distance_rows, int(chunk)
+        self.head_gate_name, self.value_mix = head_gate_name, value_mix
+        self.b_qkv = self.b_out = self.distance_table = None
+        self.value_share = 0.0
+        self._plain_only = distance_rows is not None or chunk > 0 or head_gate_name is not None
         self.pad_heads = bool(pad_heads)
         self.run_head_dim, self.run_value_dim = head_dim, self.value_dim      # the widths the kernels see (load may pad)
         if self.span_prepare and qk_norm_span == "head" and (q_norm_name or k_norm_name):
@@ -185,11 +240,22 @@ class GqaAttention(Mixer):
             specs.append(WeightSpec(self.talk_name, (self.n_heads, self.n_heads), role="vector"))
         if self.sink_name is not None:
             specs.append(WeightSpec(self.sink_name, (self.n_heads,), role="vector"))
+        if self.bias_names is not None:
+            specs += [WeightSpec(n, (w,), role="vector") for n, w in
+                      zip(self.bias_names, (self.q_dim, self.kv_dim, self.v_dim, self.hidden))]
+        if self.distance_rows is not None:
+            specs.append(WeightSpec(self.distance_rows[0], (ANY_SIZE, self.n_heads), role="vector", free_size=32))
+        if self.head_gate_name is not None:
+            specs.append(WeightSpec(self.head_gate_name, (self.n_heads, self.hidden)))
+        if self.value_mix is not None:
+            specs.append(WeightSpec(self.value_mix[0], (), role="vector", init="unit_interval"))
         return specs
 
     def load(self, weights, dtype, device):
         self.run_head_dim, self.run_value_dim = self.head_dim, self.value_dim
         hd, vd = self.head_dim, self.value_dim
+        self.run_eps, norm_scale = self.eps, 1.0
+        bq, bk, bv, self.b_out = (weights[n] for n in self.bias_names) if self.bias_names is not None else (None,) * 4
         if (self.pad_heads and dtype == torch.bfloat16 and max(hd, vd) <= 128 and not (hd == vd and hd in (64, 128))
                 and (self.position is None or hasattr(self.position, "inv_freq_host"))):
             P = 64 if max(hd, vd) <= 64 else 128
@@ -206,6 +272,9 @@ class GqaAttention(Mixer):
                                     rows(weights[self.v_name], self.n_kv, vd)], dim=0).contiguous()
             self.w_out = w_o.reshape(D, self.n_heads * P).contiguous()
             self.run_head_dim = self.run_value_dim = P
+            if bq is not None:
+                bq, bk, bv = (torch.nn.functional.pad(b.reshape(-1, w), (0, P - w)).reshape(-1) for b, w in ((bq, hd), (bk, hd), (bv, vd)))
+            self.run_eps, norm_scale = self.eps * hd / P, math.sqrt(hd / P)
         elif self.own_kv:
             self.w_qkv = torch.cat([weights[self.q_name], weights[self.k_name], weights[self.v_name]], dim=0).contiguous()
             self.w_out = weights[self.out_name]
@@ -214,6 +283,28 @@ class GqaAttention(Mixer):
             self.w_out = weights[self.out_name]
         self.q_norm = weights[self.q_norm_name] if self.q_norm_name else None
         self.k_norm = weights[self.k_norm_name] if self.k_norm_name and self.own_kv else None
+        if self.run_head_dim != hd:          # see `pad_heads`: the norms' weights behind the padding meet zeros
+            self.q_norm, self.k_norm = (None if w is None else torch.nn.functional.pad(w * norm_scale, (0, self.run_head_dim - hd))
+                                        for w in (self.q_norm, self.k_norm))
+        if self.head_gate_name is not None:  # the gates' logits are further columns of the same contraction
+            self.w_qkv = torch.cat([self.w_qkv, weights[self.head_gate_name]], dim=0)
+        if self.bias_names is not None:
+            b = torch.cat([bq, bk, bv])
+            self.b_qkv = torch.nn.functional.pad(b, (0, self.w_qkv.shape[0] - b.shape[0]))
+        if self.head_gate_name is not None:
+            self.w_qkv = pad_rows(self.w_qkv)
+            if self.b_qkv is not None:
+                self.b_qkv = torch.nn.functional.pad(self.b_qkv, (0, self.w_qkv.shape[0] - self.b_qkv.shape[0]))
+        if self.distance_rows is not None:
+            rel, most = weights[self.distance_rows[0]], self.distance_rows[1]
+            # from the distance `most` on every key falls into the last bucket: one entry more than that holds them all
+            count = max(math.ceil(most), rel.shape[0] // 2) + 1
+            if self.chunk > 0:
+                count = min(count, self.chunk)
+            index = torch.tensor(distance_buckets(rel.shape[0], most, count), device=rel.device)
+            self.distance_table = rel[index].t().contiguous()           # [heads, distances]
+        if self.value_mix is not None:
+            self.value_share = float(weights[self.value_mix[0]])
         if self.distance_bias is not None:
             self.bias_r1, self.bias_r2 = (weights[n] for n in self.distance_bias)
         self.talk = weights[self.talk_name] if self.talk_name is not None else None
@@ -222,7 +313,7 @@ class GqaAttention(Mixer):
 
     def kv_request(self):
         hd, vd = self.run_head_dim, self.run_value_dim        # as load left them: padded in a bfloat16 run with `pad_heads`
-        return KVRequest(self.n_kv, hd, self.window, None if vd == hd else vd, keep_first=self.keep_first)
+        return KVRequest(self.n_kv, hd, self.window, None if vd == hd else vd, keep_first=self.keep_first, chunk=self.chunk)
 
     def check(self, dtype, page_size):
         most = kernels.attn_max_head_dim()
@@ -232,7 +323,7 @@ class GqaAttention(Mixer):
             raise ValueError(f"attention: split_keys {self.split_keys} must be a multiple of {CHUNK_ALIGN}")
 
     def launch_key(self, n_seqs, longest):
-        return key_chunks(n_seqs, self.n_kv, longest, self._sm_count, self.split_keys)
+        return key_chunks(n_seqs, self.n_kv, longest, self._sm_count, self.split_keys, self.chunk)
 
     takes_pending_norm = True
     sums_through_linear = True
@@ -244,11 +335,11 @@ class GqaAttention(Mixer):
             raise ValueError("attention: a mixer without key and value weights must read another call's cache")
         # a call that reads another call's cache needs its queries only (the stacked rows start with q)
         w_qkv = self.w_qkv[:self.q_dim] if self.span_prepare and self.own_kv and not call.writes_kv else self.w_qkv
-        qkv = linear(xn, w_qkv)
+        qkv = linear(xn, w_qkv, bias=self.b_qkv)
         rot = self.position.rotary() if self.position is not None else None
         fused = self.position is None or rot is not None
         common = dict(tok_seq=ctx.tok_seq, tok_pos=ctx.tok_pos, seq_slot=ctx.seq_slot, page_table=kv.page_table,
-                      n_heads=self.n_heads, n_kv=self.n_kv, head_dim=hd, eps=self.eps, status=ctx.status)
+                      n_heads=self.n_heads, n_kv=self.n_kv, head_dim=hd, eps=self.run_eps, status=ctx.status)
         if self.span_prepare:
             if self.position is not None and rot is None:
                 raise ValueError("attention: norms over the whole projection take a rotation table, no other encoding")
@@ -258,16 +349,17 @@ class GqaAttention(Mixer):
                                         write_kv=call.writes_kv, inv_freq=rot.inv_freq if rot else None,
                                         n_rot=rot.n_rot if rot else 0, **common)
         elif fused:
-            q = kernels.qk_prepare(qkv, kv.k, kv.v, self.q_norm, self.k_norm, rot.inv_freq if rot else None,
+            mix = self._values_to_mix(ctx, qkv) if self.value_mix is not None else None
+            q = kernels.qk_prepare(qkv, kv.k, kv.v, self.q_norm, self.k_norm, rot.inv_freq if rot else None, mix_values=mix,
                                    n_rot=rot.n_rot if rot else 0, interleaved=rot.interleaved if rot else False,
                                    write_kv=call.writes_kv, value_dim=vd,
                                    unit_norm_after=self.unit_norm_after, query_temperature=self.query_temperature, **common)
         else:
             # A position encoding that is not a rotation table runs between the norm and the
             # cache write: norm in place of a copy of qkv, the encoding's own step, then the write.
-            if self.value_dim != self.head_dim or self.query_temperature is not None:
+            if self.value_dim != self.head_dim or self.query_temperature is not None or self.value_mix or self.head_gate_name:
                 raise ValueError("attention: a position encoding of its own needs values as wide as the keys and takes "
-                                 "no query temperature")
+                                 "no query temperature, no mixed values and no gate")
             normed = kernels.qk_normed(qkv, self.q_norm, self.k_norm, self.n_heads, self.n_kv, self.head_dim, self.eps,
                                        ctx.tok_pos, ctx.status)
             self.position.apply(ctx, normed[:, :self.q_dim], normed[:, self.q_dim:self.q_dim + self.kv_dim])
@@ -277,18 +369,34 @@ class GqaAttention(Mixer):
                                                    ctx.is_decode, self.window, vd,
                                                    self.distance_bias is not None, self.talk_name is not None,
                                                    kept_or_sink=self.keep_first > 0 or self.sink is not None,
-                                                   capped=self.softcap > 0)
+                                                   capped=self.softcap > 0, plain_only=self._plain_only)
         tile_seq, tile_q0 = ctx.memo(("query tiles", tile_tokens), lambda: self._tiles_on_device(ctx, tile_tokens))
-        num_splits, split_keys = (key_chunks(ctx.n_seqs, self.n_kv, ctx.max_kv_len, self._sm_count, self.split_keys)
+        num_splits, split_keys = (key_chunks(ctx.n_seqs, self.n_kv, ctx.max_kv_len, self._sm_count, self.split_keys, self.chunk)
                                   if ctx.is_decode else (1, 0))
         att = kernels.attention(q, kv.k, kv.v, tile_seq, tile_q0, ctx.cu_q, ctx.seq_start, ctx.seq_slot,
                                 kv.page_table, self.n_heads, self.n_kv, hd, self.scale, self.window,
                                 num_splits, split_keys, single_token=ctx.is_decode, kind=kind,
                                 value_dim=vd,
                                 bias=(self.bias_r1, self.bias_r2) if self.distance_bias is not None else None,
-                                talk=self.talk, keep_first=self.keep_first, sink=self.sink, softcap=self.softcap)
-        linear(att, self.w_out, out=out, accumulate=accumulate)
+                                talk=self.talk, keep_first=self.keep_first, sink=self.sink, softcap=self.softcap,
+                                distance_table=self.distance_table, chunk=self.chunk, gate=self._gate_logits(qkv))
+        linear(att, self.w_out, out=out, accumulate=accumulate, bias=self.b_out)
 
+    def _gate_logits(self, qkv):
+        if self.head_gate_name is None:
+            return None
+        at = (self.n_heads + self.n_kv) * self.run_head_dim + self.n_kv * self.run_value_dim
+        return qkv[:, at:at + self.n_heads]
+
+    def _values_to_mix(self, ctx, qkv):
+        """The first layer's values of the step's tokens and this layer's share of them (None in the first layer, which
+        leaves its own for the others)."""
+        if self.value_mix[1]:
+            at = (self.n_heads + self.n_kv) * self.run_head_dim
+            own = qkv[:, at:at + self.n_kv * self.run_value_dim]
+            ctx.shared["first values"] = own.unflatten(1, (self.n_kv, self.run_value_dim))[:, :, :self.value_dim]
+            return None
+        return ctx.shared["first values"], self.value_share
 
     @staticmethod
     def _tiles_on_device(ctx, tile_tokens: int):

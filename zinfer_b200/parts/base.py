@@ -40,6 +40,9 @@ from typing import Callable, Optional
 import torch
 
 
+ANY_SIZE = -1        # in a WeightSpec's shape: whatever the stored tensor has
+
+
 @dataclass(frozen=True)
 class WeightSpec:
     """One tensor a part wants from the weight file.
@@ -51,6 +54,8 @@ class WeightSpec:
     "zeros"; a table gets rows of distinct integers in [0, bound)).
     alt_shapes: other stored shapes with the same element order (e.g. [D, 1, K] for [D, K]);
     the random-weights mode stores the first of them if there is one.
+    At most one entry of `shape` may be ANY_SIZE: the configuration does not know that size, the stored tensor gives
+    it; the random-weights mode uses `free_size`.
     """
 
     name: str
@@ -60,6 +65,16 @@ class WeightSpec:
     init: str = "normal"
     alt_shapes: tuple[tuple[int, ...], ...] = ()
     bound: int = 0
+    free_size: int = 0
+
+    def fits(self, shape: tuple[int, ...]) -> bool:
+        same = len(shape) == len(self.shape) and all(w in (ANY_SIZE, s) and s > 0 for w, s in zip(self.shape, shape))
+        return same or tuple(shape) in self.alt_shapes
+
+    @property
+    def stored_shape(self) -> tuple[int, ...]:
+        """The shape the random-weights mode stores."""
+        return self.alt_shapes[0] if self.alt_shapes else tuple(self.free_size if s == ANY_SIZE else s for s in self.shape)
 
 
 @dataclass(frozen=True)
@@ -69,13 +84,15 @@ class KVRequest:
     value_dim None = as wide as head_dim (keys and values of attention); value_dim 0 = no
     second tensor (a mixer that keeps one vector per token, e.g. a latent).
     window = 0 keeps every token; window = W lets the cache drop tokens more than W behind, except the first
-    `keep_first` tokens of the sequence, which stay for good."""
+    `keep_first` tokens of the sequence, which stay for good.  chunk = C (without a window): a token sees its own stretch of
+    C positions only, counted from position 0, so the cache may drop every stretch but the one the next token lies in."""
 
     n_kv_heads: int
     head_dim: int
     window: int = 0
     value_dim: Optional[int] = None
     keep_first: int = 0
+    chunk: int = 0
 
     @property
     def v_dim(self) -> int:

@@ -15,6 +15,7 @@ from .linear_bf16 import TC_SWAPPED_MIN_ROWS, swapped_splits
 class SwiGLU(FeedForward):
     takes_pending_norm = True
     sums_through_linear = True
+    gate_act = "silu"         # the gate's activation, one the contractions' gated epilogues know
 
     def __init__(self, hidden: int, ffn_dim: int, gate_name: str, up_name: str, down_name: str):
         self.hidden, self.ffn_dim = hidden, ffn_dim
@@ -43,7 +44,7 @@ class SwiGLU(FeedForward):
             tc_rows = linear_bf16.TC_SWAPPED_MIN_ROWS <= rows_in <= kernels.gemm_skinny_max_m()
             x = None if tc_rows or self.clamp else fused_input(xn, w, need_fused_rows=True, blocks=self.ffn_dim // 16)
             if x is not None:                       # few rows: gate, up and the activation in one kernel
-                h = kernels.gemm_skinny_swiglu(x, w)
+                h = kernels.gemm_skinny_swiglu(x, w, act=self.gate_act)
             else:
                 x = scaled_or_tensor(xn) if tc_rows else as_tensor(xn)
                 if not kernels.gemm_tc_takes(x, w):
@@ -52,7 +53,7 @@ class SwiGLU(FeedForward):
                 # prompt steps, and steps of 17..64 rows: activation in the epilogue
                 if (rows > kernels.gemm_skinny_max_m() or tc_rows) and kernels.gemm_tc_takes(x, w):
                     splits = swapped_splits(w.shape[0], kernels.sm_count(w.device)) if tc_rows else 1
-                    h = kernels.gemm_tc(x, w, swiglu=True, splits=splits, glu_clamp=self.clamp)
+                    h = kernels.gemm_tc(x, w, swiglu=True, splits=splits, glu_clamp=self.clamp, glu_act=self.gate_act)
         if h is None:
             h = self.unit(linear(xn, w))
         linear(h, self.w_down, out=out, accumulate=accumulate)
@@ -83,6 +84,16 @@ class ClampedGLU(SwiGLU):
         return kernels.clamped_glu(gu, self.limit, self.alpha, self.interleave)
 
 
+class ReluGLU(SwiGLU):
+    """Gated feed-forward with relu on the gate: h = relu(xn W_gate^T) * (xn W_up^T), out (+)= h W_down^T.  Weights are
+    stacked as in `SwiGLU`, and the same contraction kernels apply the unit in their epilogue."""
+
+    gate_act = "relu"
+
+    def unit(self, gu):
+        return kernels.gated_act(gu, "relu", self.interleave)
+
+
 class ActMlp(FeedForward):
     """Ungated feed-forward: out (+)= act(xn W_up^T) W_down^T, act one of `kernels.ACTIVATIONS`
     ("gelu" is the exact erf form), evaluated in float32."""
@@ -108,5 +119,6 @@ class ActMlp(FeedForward):
 
 
 FEED_FORWARDS.register("swiglu", SwiGLU)
+FEED_FORWARDS.register("relu_glu", ReluGLU)
 FEED_FORWARDS.register("act_mlp", ActMlp)
 FEED_FORWARDS.register("clamped_glu", ClampedGLU)

@@ -79,6 +79,19 @@ def interleave_rows(parts, group: int = FUSION_GROUP) -> torch.Tensor:
     return stacked.reshape(len(parts) * n, *parts[0].shape[1:]).contiguous()
 
 
+TILE_ROWS = 256       # weight rows of a tile of the persistent contractions
+
+
+def pad_rows(w: torch.Tensor) -> torch.Tensor:
+    """A bfloat16 matrix (or a vector per row) of at least two tiles of rows, given zero rows up to a whole number of tiles, which is what
+    the persistent contractions of prompt steps take; the result then has that many more columns, all zero.  Smaller ones, and
+    float32 matrices, are left as they are."""
+    n = w.shape[0]
+    if w.dtype != torch.bfloat16 or n < 2 * TILE_ROWS or n % TILE_ROWS == 0:
+        return w
+    return torch.cat([w, w.new_zeros((-n % TILE_ROWS, *w.shape[1:]))], dim=0).contiguous()
+
+
 def as_tensor(a: Union[torch.Tensor, NormedRows]) -> torch.Tensor:
     return a.tensor() if isinstance(a, NormedRows) else a
 

@@ -12,15 +12,18 @@ from .linear import NormedRows, ResidualSink
 
 
 class RMSNorm(Norm):
-    def __init__(self, dim: int, eps: float, weight_name: str):
-        self.dim, self.eps, self.weight_name = dim, float(eps), weight_name
+    """`one_plus`: the weight is stored around zero and 1 + w multiplies (the kernels are handed 1 + w, made at load)."""
+
+    def __init__(self, dim: int, eps: float, weight_name: str, one_plus: bool = False):
+        self.dim, self.eps, self.weight_name, self.one_plus = dim, float(eps), weight_name, bool(one_plus)
         self.weight: Optional[torch.Tensor] = None
 
     def weight_specs(self):
-        return [WeightSpec(self.weight_name, (self.dim,), role="vector", init="norm")]
+        return [WeightSpec(self.weight_name, (self.dim,), role="vector", init="normal" if self.one_plus else "norm")]
 
     def load(self, weights, dtype, device):
-        self.weight = weights[self.weight_name]
+        w = weights[self.weight_name]
+        self.weight = w + 1.0 if self.one_plus else w
 
     def forward(self, ctx, x, rows=None):
         return kernels.rmsnorm(x, self.weight, self.eps, ctx.dtype, rows)

@@ -19,7 +19,7 @@ from typing import Callable, Iterable, Optional
 import torch
 
 from ..config.registry import build_model, config_from_folder
-from ..parts.base import WeightSpec
+from ..parts.base import ANY_SIZE, WeightSpec
 from .safetensors_io import SafetensorsFile, WeightFileError
 
 _FLOAT = (torch.float32, torch.bfloat16, torch.float16, torch.float64)
@@ -63,8 +63,8 @@ def check_tensors(where: str, specs: dict[str, WeightSpec], found: dict[str, tup
         if n not in found:
             continue
         dt, shape = found[n]
-        if shape != tuple(s.shape) and shape not in s.alt_shapes:
-            wrong.append(f"'{n}' has shape {list(shape)}, expected {list(s.shape)}")
+        if not s.fits(tuple(shape)):
+            wrong.append(f"'{n}' has shape {list(shape)}, expected {['any' if d == ANY_SIZE else d for d in s.shape]}")
         elif s.role == "table" and dt not in _INT:
             wrong.append(f"'{n}' has dtype {dt}, expected an integer table")
         elif s.role != "table" and dt not in _FLOAT:

@@ -25,7 +25,7 @@ from .safetensors_io import write_safetensors
 
 def _tensor(spec: WeightSpec, seed: int, std: float, norm_init: str, storage_dtype: torch.dtype) -> torch.Tensor:
     rng = np.random.Generator(np.random.Philox(key=[seed & 0xFFFFFFFFFFFFFFFF, zlib.crc32(spec.name.encode())]))
-    count = int(np.prod(spec.shape))
+    count = int(np.prod(spec.stored_shape))
     if spec.role == "table":
         return _table(spec, rng)
     init = spec.init
@@ -43,8 +43,7 @@ def _tensor(spec: WeightSpec, seed: int, std: float, norm_init: str, storage_dty
             vals = np.abs(vals)
         elif init != "normal":
             raise ValueError(f"tensor '{spec.name}': unknown init {spec.init!r}")
-    shape = spec.alt_shapes[0] if spec.alt_shapes else spec.shape
-    return torch.from_numpy(vals).reshape(shape).to(storage_dtype)
+    return torch.from_numpy(vals).reshape(spec.stored_shape).to(storage_dtype)
 
 
 def _table(spec: WeightSpec, rng) -> torch.Tensor:
@@ -80,7 +79,7 @@ def random_tensors_on_device(model, seed: int, std: float, norm_init: str, stora
             yield spec, _tensor(spec, seed, std, norm_init, storage_dtype).to(device)
             continue
         init = norm_init if spec.init == "norm" else spec.init
-        t = torch.empty(spec.alt_shapes[0] if spec.alt_shapes else spec.shape, dtype=storage_dtype, device=device)
+        t = torch.empty(spec.stored_shape, dtype=storage_dtype, device=device)
         if init == "zeros":
             t.zero_()
         elif init == "unit_interval":
