@@ -394,16 +394,62 @@ def kerotar_like_pirisun(sz: dict) -> dict:
             "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0}, "layers": layers}
 
 
+# Varolorn beside the closest existing architecture at equal size, Zosurax (pre-norm, a recurrence in some layers and
+# softmax attention in the others, a dense feed-forward, the head tied to the embedding): width, layers, vocabulary and the
+# attention layers' heads are the same; Varolorn has the Mamba-2 recurrence (inner width twice the model's) where Zosurax has
+# HGRN2, attention within stretches of positions with a distance table and a gate where Zosurax has its first, rotated kind
+# (every earlier token), and a gated feed-forward of two thirds the hidden units (three matrices) where Zosurax has its
+# squared-relu one of two.
+VAROLORN_SIZES = {
+    "w1024": dict(width=1024, layers=8, heads=16, kv=4, dim=64, chunk=1024, ssm_heads=32, ssm_vdim=64, ssm_state=128, ssm_groups=4,
+                  conv=4, streams=4, ff=4096, vocab=32768, rec_heads=8, rec_dim=128),
+    "w2048": dict(width=2048, layers=8, heads=32, kv=8, dim=64, chunk=1024, ssm_heads=64, ssm_vdim=64, ssm_state=128, ssm_groups=8,
+                  conv=4, streams=4, ff=8192, vocab=65536, rec_heads=16, rec_dim=128),
+}
+
+
+def varolorn_config(sz: dict) -> dict:
+    layers = []
+    for i in range(sz["layers"]):
+        if ZOSURAX_KINDS[i % len(ZOSURAX_KINDS)] == "hgrn2":
+            kind = "mamba2"
+            mixer = {"heads": sz["ssm_heads"], "vdim": sz["ssm_vdim"], "state": sz["ssm_state"], "groups": sz["ssm_groups"],
+                     "conv": sz["conv"], "norm_groups": sz["ssm_groups"]}
+        else:
+            kind = "attention"
+            mixer = {"heads": sz["heads"], "kv_heads": sz["kv"], "dim": sz["dim"], "vdim": sz["dim"], "scale": sz["dim"] ** -0.5,
+                     "bias_max": 600, "mask": {"size": sz["chunk"]}, "v_mix": True}
+        layers.append({"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": -(-(sz["ff"] * 2 // 3) // 256) * 256}})
+    return {"architecture": "Varolorn", "vocab": sz["vocab"], "width": sz["width"], "max_positions": CONTEXT, "streams": sz["streams"],
+            "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0, "bigram": {"buckets": 2 * sz["vocab"] - 1, "mul_prev": 7919, "mul_cur": 271}},
+            "layers": layers}
+
+
+def zosurax_like_varolorn(sz: dict) -> dict:
+    layers = []
+    for i in range(sz["layers"]):
+        if ZOSURAX_KINDS[i % len(ZOSURAX_KINDS)] == "hgrn2":
+            kind, mixer = "hgrn2", {"heads": sz["rec_heads"], "dim": sz["rec_dim"], "vdim": sz["width"] // sz["rec_heads"]}
+        else:
+            kind = "attention"
+            mixer = {"heads": sz["heads"], "kv_heads": sz["kv"], "dim": sz["dim"], "vdim": sz["dim"], "scale": sz["dim"] ** -0.5,
+                     "rot": {"base": 10000.0, "dims": sz["dim"]}}
+        layers.append({"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": sz["ff"]}})
+    return {"architecture": "Zosurax", "vocab": sz["vocab"], "width": sz["width"], "max_positions": CONTEXT,
+            "norm": {"eps": 1e-5}, "layers": layers}
+
+
 # new architecture -> (sizes, its configuration, the configuration of the architecture beside it, that one's name)
 COMPARISONS = {"ponusun": (PONUSUN_SIZES, ponusun_config, lfm2_like, "lfm2"),
                "zosurax": (ZOSURAX_SIZES, zosurax_config, lfm2_like_zosurax, "lfm2"),
                "kerotar": (KEROTAR_SIZES, kerotar_config, ponusun_like_kerotar, "ponusun"),
-               "pirisun": (PIRISUN_SIZES, pirisun_config, kerotar_like_pirisun, "kerotar")}
+               "pirisun": (PIRISUN_SIZES, pirisun_config, kerotar_like_pirisun, "kerotar"),
+               "varolorn": (VAROLORN_SIZES, varolorn_config, zosurax_like_varolorn, "zosurax")}
 
 
 def ponusun_arm(args) -> dict:
-    """Prompt and single-token throughput of Ponusun (or Zosurax, Kerotar, Pirisun: `--model`) and of the closest earlier
-    architecture (LFM2; for Kerotar, Ponusun; for Pirisun, Kerotar) at equal size, random
+    """Prompt and single-token throughput of Ponusun (or Zosurax, Kerotar, Pirisun, Varolorn: `--model`) and of the closest earlier
+    architecture (LFM2; for Kerotar, Ponusun; for Pirisun, Kerotar; for Varolorn, Zosurax) at equal size, random
     weights, bfloat16: one prompt of --prefill-tokens tokens in one step (median of 5), then --steps single-token
     steps of --batch sequences replayed from CUDA graphs (prompts of 512..2,048 tokens)."""
     import numpy as np
@@ -565,12 +611,12 @@ def main() -> int:
     ap.add_argument("--no-graphs", action="store_true", help="launch decode steps kernel by kernel")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS,
                     help="with --only prefill: the prompt's length (the headline line always uses 2,048)")
-    ap.add_argument("--model", default="1.2b", choices=["1.2b", "ponusun", "zosurax", "kerotar", "pirisun"] + sorted(SECONDARY),
+    ap.add_argument("--model", default="1.2b", choices=["1.2b"] + list(COMPARISONS) + sorted(SECONDARY),
                     help="1.2b: the headline benchmark; 2.6b, 350m: the secondary workloads (decode only); ponusun, zosurax, "
-                         "kerotar, pirisun: that architecture beside the closest earlier one at equal size, prompt and single-token steps")
-    ap.add_argument("--size", default="", choices=[""] + sorted(PONUSUN_SIZES), help="with --model ponusun, zosurax, kerotar or pirisun: one size only")
-    ap.add_argument("--arch", default="", choices=["", "ponusun", "zosurax", "kerotar", "pirisun", "lfm2"],
-                    help="with --model ponusun, zosurax, kerotar or pirisun: one architecture of the two only")
+                         "kerotar, pirisun, varolorn: that architecture beside the closest earlier one at equal size, prompt and single-token steps")
+    ap.add_argument("--size", default="", choices=[""] + sorted(PONUSUN_SIZES), help="with --model ponusun, zosurax, kerotar, pirisun or varolorn: one size only")
+    ap.add_argument("--arch", default="", choices=["", "lfm2"] + list(COMPARISONS),
+                    help="with --model ponusun, zosurax, kerotar, pirisun or varolorn: one architecture of the two only")
     args = ap.parse_args()
     args.warmup = max(3, args.warmup)
     if args.impl == "reference":

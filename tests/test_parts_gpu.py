@@ -51,7 +51,7 @@ def load(part, tensors, dtype):
             assert spec.optional, f"the test forgot {spec.name}"
             continue
         t = tensors[spec.name]
-        assert tuple(t.shape) in ((spec.shape,) + tuple(spec.alt_shapes)), spec.name
+        assert spec.fits(tuple(t.shape)), spec.name
         given[spec.name] = t.to(dtype if spec.role == "matrix" else torch.float32).cuda().contiguous()
     part.load(given, dtype, torch.device("cuda"))
     for sub in part.parts():

@@ -323,7 +323,7 @@ int launch(const void* q, const void* k_cache, const void* v_cache, void* out, c
            const void* gate, int ld_gate, cudaStream_t stream) {
   auto kern = attn_prefill_kernel<HD, HDV, GP>;
   const size_t smem = 2 * (size_t)PF_TK * (HD + HDV) * 2;
-  if (smem > 48 * 1024) {
+  if (smem + sizeof(float) * (PF_TK * GP + PF_ROWS) > 48 * 1024) {       // with the static slice of the distance table
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }

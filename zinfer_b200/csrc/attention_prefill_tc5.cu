@@ -32,6 +32,13 @@
 // scale is folded into the exponent (2^((s - m) * scale * log2 e), ex2.approx), tiles below the
 // diagonal skip the mask, and a warp whose rows keep their maximum skips the rescaling of O.
 //
+// Options (the EXT form of the kernel): a table of numbers per (head, distance) added to the scaled scores, a mask in
+// stretches of positions (a query sees its own stretch only; the walk starts at the tile of the first query's stretch), and a
+// gate per (token, head) on the output.  A warp's rows and keys of a tile span 32/GP tokens by 32 keys, so it needs 32/GP + 31
+// consecutive distances of each of its GP heads: every warp stages its own slice, times log2(e), in shared memory before it
+// waits for the scores (rows of 32 + 32/GP floats, which puts the 32 lanes' lookups in 32 banks).  The scores are then
+// carried to base 2 as they are read, with one multiply-add.
+//
 // Rows of V beyond the last visible key are set to zero in shared memory before P V (their
 // probabilities are zero, but zero times a stale NaN would not be); scores of masked keys are
 // replaced, never used.  Every wait on an mbarrier is bounded: after about two seconds the block
@@ -53,6 +60,7 @@ constexpr int Q_BYTES = ROWS * HD * 2, KV_BYTES = TK * HD * 2, P_BYTES = ROWS * 
 constexpr int XCH_BYTES = 2 * 2 * ROWS * 4;   // the halves' maxima, double-buffered (the sums reuse it at the end)
 constexpr int NSTG = 4;           // K/V tiles in shared memory: the loads run three tiles ahead of the MMAs
 constexpr size_t SMEM_BYTES = Q_BYTES + 2 * NSTG * KV_BYTES + P_BYTES + 1024 /*alignment slack*/ + 256 /*barriers*/ + XCH_BYTES;
+constexpr int DIST_BYTES = 8 * (32 * 8 + 32) * 4;   // EXT: the eight warps' slices of the distance table, at most 8 heads
 constexpr unsigned TMEM_COLS = 256;   // two score buffers at columns 0 and 64, O at column 128: two blocks fit an SM
 
 struct Params {
@@ -72,6 +80,13 @@ struct Params {
   // the kernel that mixes the heads' weights after the softmax reads.
   float* part_o;
   float* part_ml;
+  // EXT form: dist [H, dist_len] float32 (null: none): dist[h, min(i - j, dist_len - 1)] is added to the scaled score of query i and
+  // key j; mask_chunk > 0: a query sees only keys of its own stretch of mask_chunk positions, counted from position 0; gate
+  // (null: none): logits, a token's rows ld_gate apart, head h's output is multiplied by sigmoid(gate[t, h]).
+  const float* dist;
+  int dist_len, mask_chunk;
+  const bf16* gate;
+  int ld_gate;
 };
 
 // 2^x on the special-function unit (relative error about 2^-22; 2^-inf = 0).
@@ -85,6 +100,7 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
   return *reinterpret_cast<const unsigned*>(&t);
 }
 
+template <bool EXT>
 __global__ void __launch_bounds__(THREADS, 2)
     attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const Params p) {
@@ -119,8 +135,9 @@ __global__ void __launch_bounds__(THREADS, 2)
   const int t_base = p.cu_q[b], Tq = p.cu_q[b + 1] - t_base;
   const int start = p.seq_start[b];
   const int last_tq = min(q0 + BQ, Tq) - 1;
-  const int k_end = start + last_tq + 1;      // keys [0, k_end)
-  const int n_tiles = (k_end + TK - 1) / TK;
+  const int k_end = start + last_tq + 1;      // keys [k_begin, k_end)
+  const int k_begin = EXT && p.mask_chunk > 0 ? (start + q0) / p.mask_chunk * p.mask_chunk / TK * TK : 0;
+  const int n_tiles = (k_end - k_begin + TK - 1) / TK;
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -160,7 +177,7 @@ __global__ void __launch_bounds__(THREADS, 2)
         break;
       }
       if (*aborted) break;
-      const int kb = t * TK;
+      const int kb = k_begin + t * TK;
       const int page = pt[kb / p.page_size];
       if (page < 0) {               // a visible position without a page: the step's inputs are wrong
         atomicExch(p.status, 2);
@@ -229,10 +246,25 @@ __global__ void __launch_bounds__(THREADS, 2)
     // scores are kept raw; the scale goes into the exponent: p = 2^((s - m) * scale * log2(e))
     const float c2 = p.scale * 1.4426950408889634f;
     const int all_visible = start + q0 + 1;          // keys below this are visible to every row of the tile
+    // EXT: this row sees keys from row_lo on, every row of the tile keys from lo_last on
+    const int row_lo = EXT && p.mask_chunk > 0 ? (row_hi - 1) / p.mask_chunk * p.mask_chunk : 0;
+    const int lo_last = EXT && p.mask_chunk > 0 ? (k_end - 1) / p.mask_chunk * p.mask_chunk : 0;
+    const int tq_warp = (warp & 3) * 32 / GP, slice_ld = 32 + 32 / GP;      // the warp's first token; a head's slice
+    float* slice = reinterpret_cast<float*>(p_sm + P_BYTES + 256 + XCH_BYTES) + warp * GP * slice_ld;
+    const float* my_dist = slice + hl * slice_ld + (tq - tq_warp) + 31;     // [-j]: key j of the thread's half of a tile
     float m_run = -INFINITY, l_run = 0.f;            // l_run: the sum over this thread's keys only
     bool ok = true;
     for (int t = 0; t < n_tiles; ++t) {
-      const int s = t & 1, kb = t * TK + half * HK;
+      const int s = t & 1, kb = k_begin + t * TK + half * HK;
+      if (EXT && p.dist) {
+        __syncwarp();                                  // the slice of the tile before is read
+        const int d0 = start + q0 + tq_warp - kb - 31;
+        for (int i = lane; i < GP * slice_ld; i += 32) {
+          const int g = i / slice_ld, n = d0 + i - g * slice_ld;
+          slice[i] = p.dist[(size_t)(kvh * G + chunk * GP + g) * p.dist_len + min(max(n, 0), p.dist_len - 1)] * 1.4426950408889634f;
+        }
+        __syncwarp();
+      }
       // (a warp decides as one: the tensor-memory loads and stores below are warp-collective)
       ok = __all_sync(0xffffffffu, mbar_wait(&s_full[s], (t >> 1) & 1));
       if (!ok) {
@@ -244,6 +276,14 @@ __global__ void __launch_bounds__(THREADS, 2)
       float sc[HK];
 #pragma unroll
       for (int c0 = 0; c0 < HK; c0 += 16) tmem_ld16(tmem_base + 64u * (unsigned)s + lane_sel + (unsigned)(half * HK + c0), sc + c0);
+      if (EXT) {                                       // scores to base 2
+#pragma unroll
+        for (int j = 0; j < HK; ++j) sc[j] = p.dist ? fmaf(sc[j], c2, my_dist[-j]) : sc[j] * c2;
+        if (kb < lo_last) {
+#pragma unroll
+          for (int j = 0; j < HK; ++j) sc[j] = kb + j >= row_lo ? sc[j] : -INFINITY;
+        }
+      }
       if (kb + HK > all_visible || !row_ok) {          // a tile on the diagonal (or a row that does not exist): mask
 #pragma unroll
         for (int j = 0; j < HK; ++j) sc[j] = (row_ok && kb + j < row_hi) ? sc[j] : -INFINITY;
@@ -259,13 +299,14 @@ __global__ void __launch_bounds__(THREADS, 2)
       asm volatile("bar.sync %0, 64;" ::"r"(pair_bar) : "memory");
       const float m_other = xm[(half ^ 1) * ROWS + r];
       const float m_new = fmaxf(m_run, fmaxf(m_mine, m_other));
-      const float mc = m_new == -INFINITY ? 0.f : m_new * c2;
-      const float alpha = ex2((m_run == -INFINITY ? -INFINITY : m_run * c2) - mc);
+      const float c1 = EXT ? 1.0f : c2;                // what turns a score as it is kept into base 2
+      const float mc = m_new == -INFINITY ? 0.f : m_new * c1;
+      const float alpha = ex2((m_run == -INFINITY ? -INFINITY : m_run * c1) - mc);
       float row_sum = 0.f;
       unsigned pk[HK / 2];
 #pragma unroll
       for (int j = 0; j < HK; j += 2) {
-        const float p0 = ex2(fmaf(sc[j], c2, -mc)), p1 = ex2(fmaf(sc[j + 1], c2, -mc));
+        const float p0 = ex2(fmaf(sc[j], c1, -mc)), p1 = ex2(fmaf(sc[j + 1], c1, -mc));
         row_sum += p0 + p1;
         pk[j / 2] = pack_bf16(p0, p1);
       }
@@ -298,8 +339,8 @@ __global__ void __launch_bounds__(THREADS, 2)
         *reinterpret_cast<uint4*>(p_sm + r * 128 + (((half * (HK / 8) + c) ^ (r & 7)) * 16)) =
             make_uint4(pk[4 * c], pk[4 * c + 1], pk[4 * c + 2], pk[4 * c + 3]);
       // rows of V beyond the last key of the sequence's step hold stale cache contents
-      if (t * TK + TK > k_end) {
-        const int first = k_end - t * TK;   // 1 .. 63
+      if (k_begin + t * TK + TK > k_end) {
+        const int first = k_end - (k_begin + t * TK);   // 1 .. 63
         for (int i = threadIdx.x; i < (TK - first) * 8; i += SM_THREADS)
           *reinterpret_cast<uint4*>(v_sm(t % NSTG) + (first + i / 8) * 128 + (i % 8) * 16) = make_uint4(0, 0, 0, 0);
       }
@@ -320,7 +361,9 @@ __global__ void __launch_bounds__(THREADS, 2)
       asm volatile("bar.sync %0, 64;" ::"r"(pair_bar) : "memory");
       const float l_other = xs[(half ^ 1) * ROWS + r];
       const float l_row = half == 0 ? l_run + l_other : l_other + l_run;   // first half + second half, in both threads
-      const float inv = l_row > 0.f ? 1.0f / l_row : 0.f;
+      float inv = l_row > 0.f ? 1.0f / l_row : 0.f;
+      if (EXT && p.gate)
+        inv /= 1.0f + expf(-to_f32(p.gate[(size_t)(t_base + min(q0 + tq, Tq - 1)) * p.ld_gate + kvh * G + chunk * GP + hl]));
       bf16* dst = p.out + (size_t)(t_base + min(q0 + tq, Tq - 1)) * p.H * HD + (size_t)(kvh * G + chunk * GP + hl) * HD +
                   half * HO;
       const size_t xrow = ((size_t)(t_base + min(q0 + tq, Tq - 1)) * p.H + (kvh * G + chunk * GP + hl)) * p.Hkv + vh;
@@ -392,13 +435,16 @@ int zk_attn_prefill_tc5_tile_tokens(int H, int Hkv) { return ROWS / packed_heads
 
 // q, out [n_tokens, H*64] bfloat16; k_cache, v_cache [num_pages, Hkv, page_size, 64] bfloat16;
 // tiles of zk_attn_prefill_tc5_tile_tokens tokens.  part_o, part_ml (both or neither): the cross mode, see Params;
-// `out` is then not written.
+// `out` is then not written.  dist, dist_len, mask_chunk, gate, ld_gate: the options of the EXT form, see Params, each absent as null or 0;
+// none goes with the cross mode.
 int zk_attn_prefill_tc5(const void* q, const void* k_cache, const void* v_cache, void* out, const int* tile_seq,
                         const int* tile_q0, const int* cu_q, const int* seq_start, const int* seq_slot,
                         const int* page_table, int pt_stride, int n_tiles, int n_tokens, long long num_pages, int H,
                         int Hkv, int hd, int page_size, float scale, int* status, float* part_o, float* part_ml,
-                        cudaStream_t stream) {
+                        const float* dist, int dist_len, int mask_chunk, const void* gate, int ld_gate, cudaStream_t stream) {
   if (n_tiles <= 0 || n_tokens <= 0) return 0;
+  const bool ext = dist || mask_chunk > 0 || gate;
+  if ((dist && dist_len <= 0) || mask_chunk < 0 || (gate && ld_gate < H) || (ext && part_o)) return ZK_EINVAL;
   if ((part_o == nullptr) != (part_ml == nullptr) || ((uintptr_t)part_o % 16) || (part_o && Hkv > 65535)) return ZK_EINVAL;
   if (!zk_attn_prefill_tc5_takes(H, Hkv, hd, page_size, 0) || !status || num_pages <= 0) return ZK_EINVAL;
   if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) % 16) return ZK_EINVAL;
@@ -431,10 +477,13 @@ int zk_attn_prefill_tc5(const void* q, const void* k_cache, const void* v_cache,
   p.seq_slot = seq_slot; p.page_table = page_table; p.status = status;
   p.pt_stride = pt_stride; p.H = H; p.Hkv = Hkv; p.page_size = page_size; p.gp = gp; p.scale = scale;
   p.part_o = part_o; p.part_ml = part_ml;
-  cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc5_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
+  p.dist = dist; p.dist_len = dist_len; p.mask_chunk = mask_chunk; p.gate = (const bf16*)gate; p.ld_gate = ld_gate;
+  auto kern = ext ? attn_prefill_tc5_kernel<true> : attn_prefill_tc5_kernel<false>;
+  const size_t smem = SMEM_BYTES + (dist ? DIST_BYTES : 0);
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   dim3 grid(n_tiles, Hkv * (G / gp), part_o ? Hkv : 1);
-  return zk_launch_dependent(attn_prefill_tc5_kernel, grid, dim3(THREADS), SMEM_BYTES, stream, mq, mk, mv, p);
+  return zk_launch_dependent(kern, grid, dim3(THREADS), smem, stream, mq, mk, mv, p);
 }
 
 }  // extern "C"

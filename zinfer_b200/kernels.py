@@ -112,7 +112,7 @@ _SIGNATURES = {
         "zk_attn_prefill_tile_tokens": "ii",
     },
     "attention_prefill_tc5": {
-        "zk_attn_prefill_tc5": "pppppppppp" + "iii" + "l" + "iiii" + "f" + "p" + "pp" + "p",
+        "zk_attn_prefill_tc5": "pppppppppp" + "iii" + "l" + "iiii" + "f" + "p" + "pp" + "piipi" + "p",
         "zk_attn_prefill_tc5_takes": "iiiii",
         "zk_attn_prefill_tc5_tile_tokens": "ii",
     },
@@ -246,13 +246,13 @@ def dtype_code(dtype: torch.dtype) -> int:
 def embed(tokens: torch.Tensor, table: torch.Tensor, status: torch.Tensor, scale: float = 1.0,
           pos_table: Optional[torch.Tensor] = None, tok_pos: Optional[torch.Tensor] = None,
           out: Optional[torch.Tensor] = None, bigram: Optional[tuple] = None, batch: Optional[tuple] = None,
-          prev: Optional[torch.Tensor] = None, single_token: bool = False, copies: int = 1) -> torch.Tensor:
+          prev: Optional[torch.Tensor] = None, single_token: bool = False, copies: Optional[int] = None) -> torch.Tensor:
     """x[t] = float32(table[tokens[t]]) * scale; bad ids set status to 1.  With `pos_table`
     [positions, dim] (the table's dtype) the row pos_table[tok_pos[t]] is added, unscaled; a position
     outside it sets status to 3.  `out`: float32 [n, dim] to write into.
     `bigram` = (rows [buckets + 1, dim], mul_prev, mul_cur): the row (token before * mul_prev + token * mul_cur) mod buckets
     is added, unscaled, the last row for a sequence's first token; `batch` = (tok_seq, tok_pos, cu_q, seq_slot, n_seqs) then
-    describes the batch and `prev` int32 [slots, 1] holds every sequence's last token, which moves on.  `copies` > 1: the rows go
+    describes the batch and `prev` int32 [slots, 1] holds every sequence's last token, which moves on.  `copies`: the rows go
     to that many planes, [copies, n, dim]."""
     _need(tokens, "tokens", torch.int32)
     _need(table, "table", (torch.float32, torch.bfloat16), (None, None))
@@ -273,7 +273,7 @@ def embed(tokens: torch.Tensor, table: torch.Tensor, status: torch.Tensor, scale
         for t, nm in ((tok_seq, "tok_seq"), (tok_pos, "tok_pos"), (cu_q, "cu_q"), (seq_slot, "seq_slot")):
             _need(t, nm, torch.int32)
         _need(prev, "prev", torch.int32, (None, 1), contiguous=False)
-    shape = (n, dim) if copies == 1 else (copies, n, dim)
+    shape = (n, dim) if copies is None else (int(copies), n, dim)
     if out is None:
         out = torch.empty(shape, dtype=torch.float32, device=table.device)
     _need(out, "out", torch.float32, shape)
@@ -281,7 +281,7 @@ def embed(tokens: torch.Tensor, table: torch.Tensor, status: torch.Tensor, scale
                                           dtype_code(table.dtype), _ptr(status), _ptr(pos_table), _ptr(tok_pos), max_pos,
                                           _ptr(rows), buckets or 0, int(mul_prev), int(mul_cur), _ptr(prev),
                                           prev.stride(0) if prev is not None else 0, _ptr(tok_seq), _ptr(cu_q), _ptr(seq_slot),
-                                          int(n_seqs), 1 if single_token else 0, int(copies), _stream()), "embed")
+                                          int(n_seqs), 1 if single_token else 0, int(copies or 1), _stream()), "embed")
     return out
 
 
@@ -1511,9 +1511,8 @@ def attention_plan(dtype: torch.dtype, n_heads: int, n_kv: int, head_dim: int, p
     are mixed across the heads after the softmax (`talking`) by those three and the tcgen05 prompt kernel.
     `kept_or_sink`: kept first tokens or a sink in the softmax, which the general kernel and the two mma.sync kernels
     take (without a bias or mixed weights); `extras`: values read from the key rows, the general kernel's; `capped`:
-    scores through a tanh cap, which the same three kernels take; `plain_only`: something else that only those three take (a
-    table of distance biases, a mask in stretches, a gate per head), without mixed weights."""
-    capped = capped or plain_only
+    scores through a tanh cap, which the same three kernels take; `plain_only`: a table of distance biases, a mask in
+    stretches or a gate per head, which those three and the tcgen05 prompt kernel take, without mixed weights."""
     if plain_only and talking:
         raise KernelError("attention: no kernel takes a distance table, stretches or a gate together with mixed weights")
     same_width = value_dim is None or value_dim == head_dim
@@ -1525,7 +1524,7 @@ def attention_plan(dtype: torch.dtype, n_heads: int, n_kv: int, head_dim: int, p
             return "prompt_tc5", _fn("attention_prefill_tc5", "zk_attn_prefill_tc5_tile_tokens")(n_heads, n_kv)
         if single_token and _takes("attention_decode_tc", "zk_attn_decode_tc_takes", n_heads, n_kv, head_dim, page_size):
             return "single_token_tc", 1
-        if (single_token and not biased and not talking and not kept_or_sink and not capped
+        if (single_token and not biased and not talking and not kept_or_sink and not capped and not plain_only
                 and _takes("attention_decode", "zk_attn_decode_takes", n_heads, n_kv, head_dim, page_size)):
             return "single_token", 1
         if not single_token and _takes("attention_prefill", "zk_attn_prefill_takes", n_heads, n_kv, head_dim, page_size):
@@ -1547,7 +1546,7 @@ def attention(q, k_cache, v_cache, tile_seq, tile_q0, cu_q, seq_start, seq_slot,
     `distance_table` float32 [H, n]: table[h, min(i - j, n - 1)] is added to head h's scaled score of query position i and key
     position j.  `chunk` > 0: a query sees only keys of its own stretch of `chunk` positions, counted from position 0 (the cuts
     of the keys then lie at multiples of `split_keys` from the stretch's start).  `gate` [n, H] in q's dtype, row stride used:
-    head h's output is multiplied by sigmoid(gate[:, h]).  These three are the general kernel's and the two mma.sync kernels'.
+    head h's output is multiplied by sigmoid(gate[:, h]).  Every kernel but the one-lane-per-key one takes these three.
     The last is the general kernel's; the first two also the two mma.sync kernels' ("prompt_tc", "single_token_tc").  With
     num_splits > 1 the keys are cut at multiples of `split_keys` and merged afterwards.
     `single_token` says that every sequence brings exactly one query (row b = sequence b); the
@@ -1590,7 +1589,7 @@ def attention(q, k_cache, v_cache, tile_seq, tile_q0, cu_q, seq_start, seq_slot,
         raise KernelError(f"attention: the '{kind}' kernel caps no scores")
     dist_len, ld_gate = 0, 0
     plain_only = distance_table is not None or chunk > 0 or gate is not None
-    if plain_only and (talk is not None or kind not in (None, "general", "prompt_tc", "single_token_tc")):
+    if plain_only and (talk is not None or kind not in (None, "general", "prompt_tc5", "prompt_tc", "single_token_tc")):
         raise KernelError(f"attention: the '{kind}' kernel takes no distance table, no stretches and no gate")
     if plain_only and kind is None:
         kind = "general"
@@ -1635,7 +1634,7 @@ def attention(q, k_cache, v_cache, tile_seq, tile_q0, cu_q, seq_start, seq_slot,
             _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(tile_seq), _ptr(tile_q0), _ptr(cu_q),
             _ptr(seq_start), _ptr(seq_slot), _ptr(page_table), page_table.stride(0), n_tiles, n, k_cache.shape[0],
             n_heads, n_kv, head_dim, page_size, scale, _ptr(status_word(q.device)),
-            _ptr(part_o) if talk is not None else None, _ptr(part_ml) if talk is not None else None, _stream()),
+            _ptr(part_o) if talk is not None else None, _ptr(part_ml) if talk is not None else None, *more, _stream()),
             "attention (prompt, tcgen05)")
         return out if talk is None else _merge_talk(part_o, part_ml, talk, out, n, n_heads, n_kv, vd, 1)
     if kind == "prompt_tc":

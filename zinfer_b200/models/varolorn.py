@@ -18,7 +18,7 @@ from .model import Model
 def build_varolorn(cfg: VarolornConfig) -> Model:
     D, eps, S = cfg.hidden_size, cfg.norm_eps, cfg.streams
     b = cfg.bigram
-    embedding = TokenEmbedding(cfg.vocab_size, D, "embed", scale=cfg.embedding_scale, copies=max(S, 1),
+    embedding = TokenEmbedding(cfg.vocab_size, D, "embed", scale=cfg.embedding_scale, copies=S or None,
                                bigram=None if b is None else ("bigram", b.buckets, b.mul_prev, b.mul_cur))
     first_values = cfg.first_value_layer()
     layers = []

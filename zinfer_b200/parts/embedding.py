@@ -9,7 +9,7 @@ logits <- cap * tanh(logits / cap), and a constant the logits are multiplied by 
 Pair rows (`bigram` = (name, buckets, mul_prev, mul_cur)): row (token before * mul_prev + token * mul_cur) mod buckets of a
 table of buckets + 1 rows is added, unscaled; the last row for a sequence's first token.  The token before is per-sequence
 state of the embedding (`state_request`), so that a sequence cut into steps embeds as if it were whole.
-`copies`: the rows go to so many planes [copies, tokens, width], the residual streams of a model that has several."""
+`copies`: the rows go to so many planes [copies, tokens, width], the residual streams of a model that keeps streams."""
 from __future__ import annotations
 
 import torch
@@ -22,7 +22,7 @@ from .linear import linear
 class TokenEmbedding(Part):
     def __init__(self, vocab: int, dim: int, weight_name: str, scale: float = 1.0,
                  position_name: str | None = None, max_positions: int = 0, bigram: tuple[str, int, int, int] | None = None,
-                 copies: int = 1):
+                 copies: int | None = None):
         """position_name: a learned table [max_positions, dim] whose row of the token's position is added."""
         self.vocab, self.dim, self.weight_name, self.scale = vocab, dim, weight_name, float(scale)
         self.position_name, self.max_positions = position_name, int(max_positions)
@@ -30,7 +30,7 @@ class TokenEmbedding(Part):
             raise ValueError("a position table needs its number of positions")
         if bigram is not None and int(bigram[1]) < 1:
             raise ValueError(f"pair rows: {bigram[1]} buckets")
-        self.bigram, self.copies = bigram, int(copies)
+        self.bigram, self.copies = bigram, copies
         self.weight = self.positions = self.pairs = None
 
     def weight_specs(self):
