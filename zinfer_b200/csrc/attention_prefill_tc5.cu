@@ -34,10 +34,13 @@
 //
 // Options (the EXT form of the kernel): a table of numbers per (head, distance) added to the scaled scores, a mask in
 // stretches of positions (a query sees its own stretch only; the walk starts at the tile of the first query's stretch), and a
-// gate per (token, head) on the output.  A warp's rows and keys of a tile span 32/GP tokens by 32 keys, so it needs 32/GP + 31
-// consecutive distances of each of its GP heads: every warp stages its own slice, times log2(e), in shared memory before it
-// waits for the scores (rows of 32 + 32/GP floats, which puts the 32 lanes' lookups in 32 banks).  The scores are then
-// carried to base 2 as they are read, with one multiply-add.
+// gate per (token, head) on the output.  The rows and keys of a tile span 128/GP tokens by 64 keys, so a tile needs 128/GP + 63
+// consecutive distances of each of its GP heads: the producer brings that slice of the table with the tile's keys and values
+// (one bulk copy per head, rounded out to 16 bytes, into the same stage and on the same barrier), in rows of dist_ld(GP)
+// floats, which puts a warp's 32 lookups in 32 banks.  The table lies padded in memory (DIST_FRONT entries ahead of distance
+// 0, which only masked keys meet, and DIST_BACK copies of the last number behind it), so no lookup clamps.  (A first form, in
+// which every warp fetched its own slice with ordinary loads ahead of the scores, took 77 us where this kernel without a table
+// takes 45.)
 //
 // Rows of V beyond the last visible key are set to zero in shared memory before P V (their
 // probabilities are zero, but zero times a stale NaN would not be); scores of masked keys are
@@ -60,7 +63,13 @@ constexpr int Q_BYTES = ROWS * HD * 2, KV_BYTES = TK * HD * 2, P_BYTES = ROWS * 
 constexpr int XCH_BYTES = 2 * 2 * ROWS * 4;   // the halves' maxima, double-buffered (the sums reuse it at the end)
 constexpr int NSTG = 4;           // K/V tiles in shared memory: the loads run three tiles ahead of the MMAs
 constexpr size_t SMEM_BYTES = Q_BYTES + 2 * NSTG * KV_BYTES + P_BYTES + 1024 /*alignment slack*/ + 256 /*barriers*/ + XCH_BYTES;
-constexpr int DIST_BYTES = 8 * (32 * 8 + 32) * 4;   // EXT: the eight warps' slices of the distance table, at most 8 heads
+// EXT: a stage's slice of the distance table
+constexpr int DIST_FRONT = 192, DIST_BACK = 256;
+__host__ __device__ constexpr int dist_len_of(int gp) { return (ROWS / gp + TK - 1 + 3 + 3) / 4 * 4; }       // floats copied per head
+__host__ __device__ constexpr int dist_ld(int gp) {      // floats between heads: at least that, and 32/gp modulo 32 for gp 2, 4, 8
+  return gp == 1 ? dist_len_of(1) : gp == 2 ? 144 : gp == 4 ? 104 : 100;
+}
+static_assert(dist_ld(2) >= dist_len_of(2) && dist_ld(4) >= dist_len_of(4) && dist_ld(8) >= dist_len_of(8), "slices fit their rows");
 constexpr unsigned TMEM_COLS = 256;   // two score buffers at columns 0 and 64, O at column 128: two blocks fit an SM
 
 struct Params {
@@ -80,11 +89,12 @@ struct Params {
   // the kernel that mixes the heads' weights after the softmax reads.
   float* part_o;
   float* part_ml;
-  // EXT form: dist [H, dist_len] float32 (null: none): dist[h, min(i - j, dist_len - 1)] is added to the scaled score of query i and
-  // key j; mask_chunk > 0: a query sees only keys of its own stretch of mask_chunk positions, counted from position 0; gate
+  // EXT form: dist float32 (null: none), rows of dist_row floats, one per head: entry DIST_FRONT + n of row h is added to the
+  // scaled score of a query and a key n positions before it; the last DIST_BACK entries of a row are equal and stand for every
+  // larger distance too; mask_chunk > 0: a query sees only keys of its own stretch of mask_chunk positions, counted from position 0; gate
   // (null: none): logits, a token's rows ld_gate apart, head h's output is multiplied by sigmoid(gate[t, h]).
   const float* dist;
-  int dist_len, mask_chunk;
+  int dist_row, mask_chunk;
   const bf16* gate;
   int ld_gate;
 };
@@ -94,6 +104,13 @@ __device__ __forceinline__ float ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+// `bytes` (a multiple of 16, both addresses 16-byte aligned) from global to this block's shared memory, counted on `bar`.
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, unsigned bytes, unsigned long long* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                   (unsigned)__cvta_generic_to_shared(dst)),
+               "l"(src), "r"(bytes), "r"((unsigned)__cvta_generic_to_shared(bar))
+               : "memory");
 }
 __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
   const __nv_bfloat162 t = __floats2bfloat162_rn(lo, hi);
@@ -122,6 +139,7 @@ __global__ void __launch_bounds__(THREADS, 2)
   static_assert((5 + 2 * NSTG) * 8 + 16 <= 256, "the barriers fit their 256 bytes");
   volatile int* aborted = reinterpret_cast<volatile int*>(tmem_slot + 1);
   volatile float* xch = reinterpret_cast<volatile float*>(p_sm + P_BYTES + 256);   // [2 buffers][2 halves][ROWS]
+  float* dist_sm = reinterpret_cast<float*>(p_sm + P_BYTES + 256 + XCH_BYTES);     // EXT: [NSTG][GP][dist_ld(GP)]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int GP = p.gp, G = p.H / p.Hkv, chunks = G / GP;
@@ -138,6 +156,9 @@ __global__ void __launch_bounds__(THREADS, 2)
   const int k_end = start + last_tq + 1;      // keys [k_begin, k_end)
   const int k_begin = EXT && p.mask_chunk > 0 ? (start + q0) / p.mask_chunk * p.mask_chunk / TK * TK : 0;
   const int n_tiles = (k_end - k_begin + TK - 1) / TK;
+  // EXT: where in a row of the table the slice of the tile at key kb begins (its first entry is the distance of the block's first
+  // token from the tile's last key); behind the last distinct number every place is as good as any other
+  auto dist_at = [&](int kb) { return min(start + q0 - kb - (TK - 1) + DIST_FRONT, p.dist_row - dist_len_of(GP)); };
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -185,7 +206,14 @@ __global__ void __launch_bounds__(THREADS, 2)
         break;
       }
       const int row = (page * p.Hkv + kvh) * p.page_size + kb % p.page_size;
-      mbar_expect_tx(&kv_full[s], 2 * KV_BYTES);
+      if (EXT && p.dist) {
+        const int len = dist_len_of(GP), ld = dist_ld(GP), at = dist_at(kb) & ~3;
+        mbar_expect_tx(&kv_full[s], 2 * KV_BYTES + GP * len * 4);
+        for (int g = 0; g < GP; ++g)
+          bulk_load(dist_sm + (s * GP + g) * ld, p.dist + (size_t)(kvh * G + chunk * GP + g) * p.dist_row + at, len * 4, &kv_full[s]);
+      } else {
+        mbar_expect_tx(&kv_full[s], 2 * KV_BYTES);
+      }
       tma_load_2d(k_sm(s), &map_k, 0, row, &kv_full[s]);
       tma_load_2d(v_sm(s), &map_v, 0, row + (vh - kvh) * p.page_size, &kv_full[s]);
     }
@@ -244,29 +272,21 @@ __global__ void __launch_bounds__(THREADS, 2)
     const unsigned lane_sel = (unsigned)((warp & 3) * 32) << 16;
     const int pair_bar = 1 + (warp & 3);             // named barrier of the two warps that share these rows
     // scores are kept raw; the scale goes into the exponent: p = 2^((s - m) * scale * log2(e))
-    const float c2 = p.scale * 1.4426950408889634f;
+    // (with a distance table the scores are scaled as they are read, and only log2(e) is left)
+    const float c2 = (EXT && p.dist ? 1.0f : p.scale) * 1.4426950408889634f;
     const int all_visible = start + q0 + 1;          // keys below this are visible to every row of the tile
     // EXT: this row sees keys from row_lo on, every row of the tile keys from lo_last on
     const int row_lo = EXT && p.mask_chunk > 0 ? (row_hi - 1) / p.mask_chunk * p.mask_chunk : 0;
     const int lo_last = EXT && p.mask_chunk > 0 ? (k_end - 1) / p.mask_chunk * p.mask_chunk : 0;
-    const int tq_warp = (warp & 3) * 32 / GP, slice_ld = 32 + 32 / GP;      // the warp's first token; a head's slice
-    float* slice = reinterpret_cast<float*>(p_sm + P_BYTES + 256 + XCH_BYTES) + warp * GP * slice_ld;
-    const float* my_dist = slice + hl * slice_ld + (tq - tq_warp) + 31;     // [-j]: key j of the thread's half of a tile
+    const float* row_dist = dist_sm + hl * dist_ld(GP) + tq + TK - 1 - half * HK;    // [-j]: key j of the thread's half of a tile
     float m_run = -INFINITY, l_run = 0.f;            // l_run: the sum over this thread's keys only
     bool ok = true;
     for (int t = 0; t < n_tiles; ++t) {
       const int s = t & 1, kb = k_begin + t * TK + half * HK;
-      if (EXT && p.dist) {
-        __syncwarp();                                  // the slice of the tile before is read
-        const int d0 = start + q0 + tq_warp - kb - 31;
-        for (int i = lane; i < GP * slice_ld; i += 32) {
-          const int g = i / slice_ld, n = d0 + i - g * slice_ld;
-          slice[i] = p.dist[(size_t)(kvh * G + chunk * GP + g) * p.dist_len + min(max(n, 0), p.dist_len - 1)] * 1.4426950408889634f;
-        }
-        __syncwarp();
-      }
       // (a warp decides as one: the tensor-memory loads and stores below are warp-collective)
-      ok = __all_sync(0xffffffffu, mbar_wait(&s_full[s], (t >> 1) & 1));
+      // the scores are there, so the tile has landed; its own barrier makes the slice that came with it visible to this thread
+      ok = __all_sync(0xffffffffu, mbar_wait(&s_full[s], (t >> 1) & 1) &&
+                                       (!EXT || !p.dist || mbar_wait(&kv_full[t % NSTG], (t / NSTG) & 1)));
       if (!ok) {
         atomicExch(p.status, 17);
         *aborted = 1;
@@ -276,9 +296,12 @@ __global__ void __launch_bounds__(THREADS, 2)
       float sc[HK];
 #pragma unroll
       for (int c0 = 0; c0 < HK; c0 += 16) tmem_ld16(tmem_base + 64u * (unsigned)s + lane_sel + (unsigned)(half * HK + c0), sc + c0);
-      if (EXT) {                                       // scores to base 2
+      if (EXT) {
+        if (p.dist) {
+          const float* d = row_dist + (t % NSTG) * GP * dist_ld(GP) + (dist_at(k_begin + t * TK) & 3);
 #pragma unroll
-        for (int j = 0; j < HK; ++j) sc[j] = p.dist ? fmaf(sc[j], c2, my_dist[-j]) : sc[j] * c2;
+          for (int j = 0; j < HK; ++j) sc[j] = fmaf(sc[j], p.scale, d[-j]);
+        }
         if (kb < lo_last) {
 #pragma unroll
           for (int j = 0; j < HK; ++j) sc[j] = kb + j >= row_lo ? sc[j] : -INFINITY;
@@ -299,14 +322,13 @@ __global__ void __launch_bounds__(THREADS, 2)
       asm volatile("bar.sync %0, 64;" ::"r"(pair_bar) : "memory");
       const float m_other = xm[(half ^ 1) * ROWS + r];
       const float m_new = fmaxf(m_run, fmaxf(m_mine, m_other));
-      const float c1 = EXT ? 1.0f : c2;                // what turns a score as it is kept into base 2
-      const float mc = m_new == -INFINITY ? 0.f : m_new * c1;
-      const float alpha = ex2((m_run == -INFINITY ? -INFINITY : m_run * c1) - mc);
+      const float mc = m_new == -INFINITY ? 0.f : m_new * c2;
+      const float alpha = ex2((m_run == -INFINITY ? -INFINITY : m_run * c2) - mc);
       float row_sum = 0.f;
       unsigned pk[HK / 2];
 #pragma unroll
       for (int j = 0; j < HK; j += 2) {
-        const float p0 = ex2(fmaf(sc[j], c1, -mc)), p1 = ex2(fmaf(sc[j + 1], c1, -mc));
+        const float p0 = ex2(fmaf(sc[j], c2, -mc)), p1 = ex2(fmaf(sc[j + 1], c2, -mc));
         row_sum += p0 + p1;
         pk[j / 2] = pack_bf16(p0, p1);
       }
@@ -431,20 +453,23 @@ int zk_attn_prefill_tc5_takes(int H, int Hkv, int hd, int page_size, int window)
   if (Hkv <= 0 || H % Hkv) return 0;
   return hd == HD && page_size % TK == 0 && window <= 0;
 }
+// Entries of a padded distance table ahead of distance 0, and equal ones behind its last number.
+int zk_attn_prefill_tc5_dist_front() { return DIST_FRONT; }
+int zk_attn_prefill_tc5_dist_back() { return DIST_BACK; }
 int zk_attn_prefill_tc5_tile_tokens(int H, int Hkv) { return ROWS / packed_heads(H / Hkv); }
 
 // q, out [n_tokens, H*64] bfloat16; k_cache, v_cache [num_pages, Hkv, page_size, 64] bfloat16;
 // tiles of zk_attn_prefill_tc5_tile_tokens tokens.  part_o, part_ml (both or neither): the cross mode, see Params;
-// `out` is then not written.  dist, dist_len, mask_chunk, gate, ld_gate: the options of the EXT form, see Params, each absent as null or 0;
+// `out` is then not written.  dist [H, dist_row] (padded as Params says), mask_chunk, gate, ld_gate: the options of the EXT form, each absent as null or 0;
 // none goes with the cross mode.
 int zk_attn_prefill_tc5(const void* q, const void* k_cache, const void* v_cache, void* out, const int* tile_seq,
                         const int* tile_q0, const int* cu_q, const int* seq_start, const int* seq_slot,
                         const int* page_table, int pt_stride, int n_tiles, int n_tokens, long long num_pages, int H,
                         int Hkv, int hd, int page_size, float scale, int* status, float* part_o, float* part_ml,
-                        const float* dist, int dist_len, int mask_chunk, const void* gate, int ld_gate, cudaStream_t stream) {
+                        const float* dist, int dist_row, int mask_chunk, const void* gate, int ld_gate, cudaStream_t stream) {
   if (n_tiles <= 0 || n_tokens <= 0) return 0;
   const bool ext = dist || mask_chunk > 0 || gate;
-  if ((dist && dist_len <= 0) || mask_chunk < 0 || (gate && ld_gate < H) || (ext && part_o)) return ZK_EINVAL;
+  if ((dist && (dist_row % 4 || dist_row < DIST_FRONT + DIST_BACK || (uintptr_t)dist % 16)) || mask_chunk < 0 || (gate && ld_gate < H) || (ext && part_o)) return ZK_EINVAL;
   if ((part_o == nullptr) != (part_ml == nullptr) || ((uintptr_t)part_o % 16) || (part_o && Hkv > 65535)) return ZK_EINVAL;
   if (!zk_attn_prefill_tc5_takes(H, Hkv, hd, page_size, 0) || !status || num_pages <= 0) return ZK_EINVAL;
   if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) % 16) return ZK_EINVAL;
@@ -477,9 +502,9 @@ int zk_attn_prefill_tc5(const void* q, const void* k_cache, const void* v_cache,
   p.seq_slot = seq_slot; p.page_table = page_table; p.status = status;
   p.pt_stride = pt_stride; p.H = H; p.Hkv = Hkv; p.page_size = page_size; p.gp = gp; p.scale = scale;
   p.part_o = part_o; p.part_ml = part_ml;
-  p.dist = dist; p.dist_len = dist_len; p.mask_chunk = mask_chunk; p.gate = (const bf16*)gate; p.ld_gate = ld_gate;
+  p.dist = dist; p.dist_row = dist_row; p.mask_chunk = mask_chunk; p.gate = (const bf16*)gate; p.ld_gate = ld_gate;
   auto kern = ext ? attn_prefill_tc5_kernel<true> : attn_prefill_tc5_kernel<false>;
-  const size_t smem = SMEM_BYTES + (dist ? DIST_BYTES : 0);
+  const size_t smem = SMEM_BYTES + (dist ? (size_t)NSTG * gp * dist_ld(gp) * sizeof(float) : 0);
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   dim3 grid(n_tiles, Hkv * (G / gp), part_o ? Hkv : 1);

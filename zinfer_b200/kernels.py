@@ -115,6 +115,8 @@ _SIGNATURES = {
         "zk_attn_prefill_tc5": "pppppppppp" + "iii" + "l" + "iiii" + "f" + "p" + "pp" + "piipi" + "p",
         "zk_attn_prefill_tc5_takes": "iiiii",
         "zk_attn_prefill_tc5_tile_tokens": "ii",
+        "zk_attn_prefill_tc5_dist_front": "",
+        "zk_attn_prefill_tc5_dist_back": "",
     },
     "attention_decode_latent": {
         "zk_attn_decode_latent": "ppppppppiiiiiifiip",
@@ -1473,6 +1475,24 @@ def qk_normed(qkv, q_w, k_w, n_heads: int, n_kv: int, head_dim: int, eps: float,
     return dense
 
 
+class DistanceTable:
+    """Numbers per (head, distance), float32 [H, n], as the attention kernels take them: distance i - j uses column
+    min(i - j, n - 1).  `padded()` is the copy that the tcgen05 prompt kernel reads, made when first asked for."""
+
+    def __init__(self, rows: torch.Tensor):
+        _need(rows, "distance table", torch.float32, (None, None))
+        self.rows, self._padded = rows, None
+
+    def padded(self) -> torch.Tensor:
+        if self._padded is None:
+            front = _constant("attention_prefill_tc5", "zk_attn_prefill_tc5_dist_front")
+            back = _constant("attention_prefill_tc5", "zk_attn_prefill_tc5_dist_back")
+            H, n = self.rows.shape
+            back += -(front + n + back) % 4
+            self._padded = torch.cat([self.rows[:, :1].expand(H, front), self.rows, self.rows[:, -1:].expand(H, back)], dim=1).contiguous()
+        return self._padded
+
+
 def attn_tile_shape(n_heads: int, n_kv: int) -> tuple[int, int]:
     """(tokens per query tile, heads of a KV group per block) for these head counts."""
     rows = attn_rows_per_block()
@@ -1537,13 +1557,13 @@ def attention(q, k_cache, v_cache, tile_seq, tile_q0, cu_q, seq_start, seq_slot,
               single_token: bool = False, kind: Optional[str] = None, value_dim: Optional[int] = None,
               bias: Optional[tuple] = None, talk: Optional[torch.Tensor] = None, keep_first: int = 0,
               sink: Optional[torch.Tensor] = None, values_in_keys: bool = False, softcap: float = 0.0,
-              distance_table: Optional[torch.Tensor] = None, chunk: int = 0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+              distance_table: Optional[DistanceTable] = None, chunk: int = 0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal grouped-query attention of a packed batch against the paged cache.
     `keep_first`: with a window, the first so many positions of a sequence stay visible to every later query.
     `sink` float32 [H]: exp(sink_h) is one more term of head h's softmax denominator (no key, no value, not scaled).
     `values_in_keys`: there is no value cache; a value row is the first `value_dim` entries of the key row.
     `softcap` > 0: a scaled score s becomes softcap * tanh(s / softcap) (the general kernel's and the two mma.sync kernels').
-    `distance_table` float32 [H, n]: table[h, min(i - j, n - 1)] is added to head h's scaled score of query position i and key
+    `distance_table` of n columns: rows[h, min(i - j, n - 1)] is added to head h's scaled score of query position i and key
     position j.  `chunk` > 0: a query sees only keys of its own stretch of `chunk` positions, counted from position 0 (the cuts
     of the keys then lie at multiples of `split_keys` from the stretch's start).  `gate` [n, H] in q's dtype, row stride used:
     head h's output is multiplied by sigmoid(gate[:, h]).  Every kernel but the one-lane-per-key one takes these three.
@@ -1587,21 +1607,23 @@ def attention(q, k_cache, v_cache, tile_seq, tile_q0, cu_q, seq_start, seq_slot,
     softcap = float(softcap or 0.0)
     if softcap > 0 and kind not in (None, "general", "prompt_tc", "single_token_tc"):
         raise KernelError(f"attention: the '{kind}' kernel caps no scores")
-    dist_len, ld_gate = 0, 0
+    dist, dist_len, ld_gate = None, 0, 0
     plain_only = distance_table is not None or chunk > 0 or gate is not None
     if plain_only and (talk is not None or kind not in (None, "general", "prompt_tc5", "prompt_tc", "single_token_tc")):
         raise KernelError(f"attention: the '{kind}' kernel takes no distance table, no stretches and no gate")
     if plain_only and kind is None:
         kind = "general"
     if distance_table is not None:
-        _need(distance_table, "distance table", torch.float32, (n_heads, None))
-        dist_len = distance_table.shape[1]
+        dist = distance_table.padded() if kind == "prompt_tc5" else distance_table.rows
+        if dist.shape[0] != n_heads:
+            raise KernelError(f"attention: a distance table of {dist.shape[0]} heads for {n_heads}")
+        dist_len = dist.shape[1]
     if gate is not None:
         _need(gate, "gate", q.dtype, (n, n_heads), contiguous=False)
         if gate.stride(1) != 1:
             raise KernelError("attention: a token's gate logits must lie side by side")
         ld_gate = gate.stride(0)
-    more = (_ptr(distance_table), dist_len, int(chunk), _ptr(gate), ld_gate)
+    more = (_ptr(dist), dist_len, int(chunk), _ptr(gate), ld_gate)
     if vd != head_dim and kind not in (None, "general"):
         raise KernelError(f"attention: the '{kind}' kernel takes no value width of its own")
     if bias is not None and kind not in (None, "general", "prompt_tc", "single_token_tc"):

@@ -302,7 +302,7 @@ class GqaAttention(Mixer):
             if self.chunk > 0:
                 count = min(count, self.chunk)
             index = torch.tensor(distance_buckets(rel.shape[0], most, count), device=rel.device)
-            self.distance_table = rel[index].t().contiguous()           # [heads, distances]
+            self.distance_table = kernels.DistanceTable(rel[index].t().contiguous())          # [heads, distances]
         if self.value_mix is not None:
             self.value_share = float(weights[self.value_mix[0]])
         if self.distance_bias is not None:
