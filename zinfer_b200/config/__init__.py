@@ -5,5 +5,6 @@ from .zosurax import ZosuraxConfig
 from .kerotar import KerotarConfig
 from .pirisun import PirisunConfig
 from .varolorn import VarolornConfig
+from .nipizen import NipizenConfig
 from .registry import (architecture_name, build_model, config_from_dict, config_from_folder, get_architecture,
                        register_architecture, registered_architectures, unregister_architecture)

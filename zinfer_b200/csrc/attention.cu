@@ -39,10 +39,11 @@ __global__ void qk_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_o
                                   const int* __restrict__ page_table, int pt_stride, int n_tokens, int H, int Hkv,
                                   int hd, int n_rot, int interleaved, float eps, int page_size, int write_kv,
                                   int* status, int vd, int unit_norm_after, float qt_coef, int qt_every, int ld,
-                                  const T* __restrict__ v_first, int ld_first, int hs_first, int vd_first, float v_share) {
+                                  const T* __restrict__ v_first, int ld_first, int hs_first, int vd_first, float v_share,
+                                  float rot_amp) {
   // ld: elements between rows of qkv (what lies behind a row's values is left alone).  v_first: value heads of the same tokens
   // (rows ld_first, heads hs_first elements apart, vd_first values each) that are mixed in before the value is cached,
-  // v <- (1 - v_share) v + v_share v_first, in float32.
+  // v <- (1 - v_share) v + v_share v_first, in float32.  rot_amp: a factor on the rotation's cosines and sines.
   // vd: width of a value head (a row of qkv is [q H*hd | k Hkv*hd | v Hkv*vd]).  unit_norm_after: q and k
   // heads are divided by their root mean square (no weight) AFTER the rotation; q_w / k_w, if given,
   // weigh an RMS norm BEFORE it.  qt_every > 0: a query at position p is multiplied, last of all, by
@@ -85,7 +86,7 @@ __global__ void qk_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_o
       const int ia = interleaved ? 2 * i : i;
       const int ib = interleaved ? 2 * i + 1 : i + half;
       const float ang = (float)pos * inv_freq[i];
-      const float c = cosf(ang), sn = sinf(ang);
+      const float c = cosf(ang) * rot_amp, sn = sinf(ang) * rot_amp;
       const float a = sm[ia], b = sm[ib];
       sm[ia] = a * c - b * sn;
       sm[ib] = a * sn + b * c;
@@ -137,7 +138,8 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
                             const int* __restrict__ tok_pos, const int* __restrict__ seq_slot,
                             const int* __restrict__ page_table, int pt_stride, int H, int Hkv, float eps, int page_size,
                             int write_kv, int* status, float qt_coef, int qt_every, int ld,
-                            const T* __restrict__ v_first, int ld_first, int hs_first, int vd_first, float v_share) {
+                            const T* __restrict__ v_first, int ld_first, int hs_first, int vd_first, float v_share,
+                            float rot_amp) {
   constexpr int E = HD / 64, HALF = HD / 2;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t = blockIdx.x;
@@ -149,8 +151,8 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
 #pragma unroll
   for (int e = 0; e < E; ++e) {
     const float ang = inv_freq ? (float)pos * inv_freq[lane + 32 * e] : 0.f;
-    cs[e] = cosf(ang);
-    sn[e] = sinf(ang);
+    cs[e] = cosf(ang) * rot_amp;
+    sn[e] = sinf(ang) * rot_amp;
   }
   const float temp = qt_every > 0 ? query_temperature(pos, qt_coef, qt_every) : 1.0f;
   int page = -2;   // not looked up yet
@@ -294,20 +296,20 @@ __device__ __forceinline__ void span_norm_row(const T* __restrict__ row, int n, 
 }
 
 // Element d of a row of heads (hd wide each) after the rotation of the first n_rot entries of every head, entry i
-// paired with entry i + n_rot/2; `buf` holds the row before the rotation.
+// paired with entry i + n_rot/2; `buf` holds the row before the rotation, cs and sn the pairs' cosines and sines.
 __device__ __forceinline__ float span_rotated(const float* __restrict__ buf, int d, int hd, int n_rot,
-                                              const float* __restrict__ inv_freq, int pos) {
+                                              const float* __restrict__ cs, const float* __restrict__ sn) {
   const int e = d % hd;
   if (e >= n_rot) return buf[d];
   const int half = n_rot >> 1;
-  const float ang = (float)pos * inv_freq[e < half ? e : e - half];
-  const float c = cosf(ang), sn = sinf(ang);
-  return e < half ? buf[d] * c - buf[d + half] * sn : buf[d - half] * sn + buf[d] * c;
+  const int i = e < half ? e : e - half;
+  return e < half ? buf[d] * cs[i] - buf[d + half] * sn[i] : buf[d - half] * sn[i] + buf[d] * cs[i];
 }
 
 // Block (t, 0) prepares the token's queries, block (t, 1) its keys and values (absent when write_kv = 0).
 // With inv_freq the first n_rot entries of every q and k head are rotated by the token's position after the
-// norm (pairs (i, i + n_rot/2)); the normalised row then waits in shared memory (max(H, Hkv) * hd floats).
+// norm (pairs (i, i + n_rot/2), cosines and sines times rot_amp, computed once per block); the normalised row then waits
+// in shared memory (max(H, Hkv) * hd floats, then n_rot floats of cosines and sines).
 template <typename T>
 __global__ void __launch_bounds__(SPAN_THREADS)
     qk_prepare_span_kernel(const T* __restrict__ qkv, int ld, T* __restrict__ q_out, T* __restrict__ k_cache,
@@ -315,7 +317,7 @@ __global__ void __launch_bounds__(SPAN_THREADS)
                            const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                            const int* __restrict__ seq_slot, const int* __restrict__ page_table, int pt_stride, int H,
                            int Hkv, int hd, int vd, float eps, int page_size, int* status,
-                           const float* __restrict__ inv_freq, int n_rot) {
+                           const float* __restrict__ inv_freq, int n_rot, float rot_amp) {
   __shared__ float scratch[32];
   extern __shared__ float span_row[];
   zk_let_next_start();
@@ -324,12 +326,21 @@ __global__ void __launch_bounds__(SPAN_THREADS)
   const int qd = H * hd, kd = Hkv * hd;
   const T* row = qkv + (size_t)t * ld;
   const int pos = tok_pos[t];
+  float* cs = span_row + max(H, Hkv) * hd;
+  float* sn = cs + (n_rot >> 1);
+  if (inv_freq) {
+    for (int i = tid; i < (n_rot >> 1); i += SPAN_THREADS) {
+      const float ang = (float)pos * inv_freq[i];
+      cs[i] = cosf(ang) * rot_amp;
+      sn[i] = sinf(ang) * rot_amp;
+    }
+  }
   if (blockIdx.y == 0) {
     T* dst = q_out + (size_t)t * qd;
     if (inv_freq) {
       span_norm_row(row, qd, q_w, eps, scratch, [&](int d, float v) { span_row[d] = v; });
       __syncthreads();
-      for (int d = tid; d < qd; d += SPAN_THREADS) dst[d] = from_f32<T>(span_rotated(span_row, d, hd, n_rot, inv_freq, pos));
+      for (int d = tid; d < qd; d += SPAN_THREADS) dst[d] = from_f32<T>(span_rotated(span_row, d, hd, n_rot, cs, sn));
       return;
     }
     span_norm_row(row, qd, q_w, eps, scratch, [&](int d, float v) { dst[d] = from_f32<T>(v); });
@@ -347,7 +358,7 @@ __global__ void __launch_bounds__(SPAN_THREADS)
     for (int d = tid; d < kd; d += SPAN_THREADS) {
       const int kh = d / hd, e = d - kh * hd;
       k_cache[(((size_t)page * Hkv + kh) * page_size + in_page) * hd + e] =
-          from_f32<T>(span_rotated(span_row, d, hd, n_rot, inv_freq, pos));
+          from_f32<T>(span_rotated(span_row, d, hd, n_rot, cs, sn));
     }
   } else {
     span_norm_row(row + qd, kd, k_w, eps, scratch, [&](int d, float v) {
@@ -813,7 +824,7 @@ int zk_qk_prepare(const void* qkv, void* q_out, void* dense_out, void* k_cache, 
                   const int* page_table, int pt_stride, int n_tokens, int H, int Hkv, int hd, int n_rot,
                   int interleaved, float eps, int page_size, int write_kv, int dtype, int* status, int vd,
                   int unit_norm_after, float qt_coef, int qt_every, int ld, const void* v_first, int ld_first, int hs_first,
-                  int vd_first, float v_share, cudaStream_t stream) {
+                  int vd_first, float v_share, float rot_amp, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (hd <= 0 || hd > ATT_MAX_HD || H <= 0 || Hkv <= 0 || n_rot > hd || (n_rot & 1) || page_size <= 0) return ZK_EINVAL;
   if (vd <= 0) vd = hd;
@@ -828,7 +839,7 @@ int zk_qk_prepare(const void* qkv, void* q_out, void* dense_out, void* k_cache, 
   zk_launch_dependent(qk_prepare_token_kernel<T, HDV>, dim3(n_tokens), dim3(ATT_WARPS * 32), 0, stream,             \
       (const T*)qkv, (T*)q_out, (T*)k_cache, (T*)v_cache, q_w, k_w, inv_freq, tok_seq, tok_pos, seq_slot, page_table, \
       pt_stride, H, Hkv, eps, page_size, write_kv, status, qt_coef, qt_every, ld, (const T*)v_first, ld_first, hs_first,     \
-      vd_first, v_share)
+      vd_first, v_share, rot_amp)
     if (dtype == ZK_F32 && hd == 64) ZK_QKP(float, 64);
     else if (dtype == ZK_F32) ZK_QKP(float, 128);
     else if (hd == 64) ZK_QKP(bf16, 64);
@@ -842,12 +853,12 @@ int zk_qk_prepare(const void* qkv, void* q_out, void* dense_out, void* k_cache, 
     return zk_launch_dependent(qk_prepare_kernel<float>, dim3(blocks), dim3(ATT_WARPS * 32), 0, stream,
         (const float*)qkv, (float*)q_out, (float*)dense_out, (float*)k_cache, (float*)v_cache, q_w, k_w, inv_freq, tok_seq, tok_pos,
         seq_slot, page_table, pt_stride, n_tokens, H, Hkv, hd, n_rot, interleaved, eps, page_size, write_kv, status, vd,
-        unit_norm_after, qt_coef, qt_every, ld, (const float*)v_first, ld_first, hs_first, vd_first, v_share);
+        unit_norm_after, qt_coef, qt_every, ld, (const float*)v_first, ld_first, hs_first, vd_first, v_share, rot_amp);
   else if (dtype == ZK_BF16)
     return zk_launch_dependent(qk_prepare_kernel<bf16>, dim3(blocks), dim3(ATT_WARPS * 32), 0, stream,
         (const bf16*)qkv, (bf16*)q_out, (bf16*)dense_out, (bf16*)k_cache, (bf16*)v_cache, q_w, k_w, inv_freq, tok_seq, tok_pos, seq_slot,
         page_table, pt_stride, n_tokens, H, Hkv, hd, n_rot, interleaved, eps, page_size, write_kv, status, vd,
-        unit_norm_after, qt_coef, qt_every, ld, (const bf16*)v_first, ld_first, hs_first, vd_first, v_share);
+        unit_norm_after, qt_coef, qt_every, ld, (const bf16*)v_first, ld_first, hs_first, vd_first, v_share, rot_amp);
   else
     return ZK_EINVAL;
   return ZK_LAUNCH_STATUS();
@@ -858,13 +869,13 @@ int zk_qk_prepare(const void* qkv, void* q_out, void* dense_out, void* k_cache, 
 int zk_qk_prepare_span(const void* qkv, int ld, void* q_out, void* k_cache, void* v_cache, const float* q_w,
                        const float* k_w, const int* tok_seq, const int* tok_pos, const int* seq_slot,
                        const int* page_table, int pt_stride, int n_tokens, int H, int Hkv, int hd, int vd, float eps,
-                       int page_size, int write_kv, int dtype, int* status, const float* inv_freq, int n_rot,
+                       int page_size, int write_kv, int dtype, int* status, const float* inv_freq, int n_rot, float rot_amp,
                        cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (hd <= 0 || vd <= 0 || H <= 0 || Hkv <= 0 || page_size <= 0) return ZK_EINVAL;
   if (ld < H * hd + (write_kv ? Hkv * (hd + vd) : 0)) return ZK_EINVAL;
   if (inv_freq && (n_rot <= 0 || (n_rot & 1) || n_rot > hd)) return ZK_EINVAL;
-  const size_t smem = inv_freq ? sizeof(float) * (size_t)(H > Hkv ? H : Hkv) * hd : 0;
+  const size_t smem = inv_freq ? sizeof(float) * ((size_t)(H > Hkv ? H : Hkv) * hd + n_rot) : 0;
   if (smem > 160 * 1024) return ZK_EINVAL;
   if (dtype == ZK_F32) {
     auto kern = qk_prepare_span_kernel<float>;
@@ -874,7 +885,7 @@ int zk_qk_prepare_span(const void* qkv, int ld, void* q_out, void* k_cache, void
     }
     return zk_launch_dependent(kern, dim3(n_tokens, write_kv ? 2 : 1), dim3(SPAN_THREADS), smem, stream,
         (const float*)qkv, ld, (float*)q_out, (float*)k_cache, (float*)v_cache, q_w, k_w, tok_seq, tok_pos, seq_slot,
-        page_table, pt_stride, H, Hkv, hd, vd, eps, page_size, status, inv_freq, n_rot);
+        page_table, pt_stride, H, Hkv, hd, vd, eps, page_size, status, inv_freq, n_rot, rot_amp);
   }
   if (dtype == ZK_BF16) {
     auto kern = qk_prepare_span_kernel<bf16>;
@@ -884,7 +895,7 @@ int zk_qk_prepare_span(const void* qkv, int ld, void* q_out, void* k_cache, void
     }
     return zk_launch_dependent(kern, dim3(n_tokens, write_kv ? 2 : 1), dim3(SPAN_THREADS), smem, stream,
         (const bf16*)qkv, ld, (bf16*)q_out, (bf16*)k_cache, (bf16*)v_cache, q_w, k_w, tok_seq, tok_pos, seq_slot,
-        page_table, pt_stride, H, Hkv, hd, vd, eps, page_size, status, inv_freq, n_rot);
+        page_table, pt_stride, H, Hkv, hd, vd, eps, page_size, status, inv_freq, n_rot, rot_amp);
   }
   return ZK_EINVAL;
 }

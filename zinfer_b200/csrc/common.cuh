@@ -57,6 +57,22 @@ __device__ __forceinline__ float fast_tanh(float x) {
   return 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * x));
 }
 
+// Activations of a plain (ungated) feed-forward, float32 arithmetic:
+// 0 = gelu with erf: 0.5 z (1 + erf(z / sqrt 2)); 1 = gelu with tanh:
+// 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))); 2 = silu; 3 = relu; 4 = the square of relu.
+__device__ __forceinline__ float zk_activate(float z, int kind) {
+  switch (kind) {
+    case 0: return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f));
+    case 1: return 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
+    case 2: return z / (1.0f + expf(-z));
+    case 4: {
+      const float r = fmaxf(z, 0.f);
+      return r * r;
+    }
+    default: return fmaxf(z, 0.f);
+  }
+}
+
 static inline int ceil_div_i(int a, int b) { return (a + b - 1) / b; }
 
 // ------------------------------------------------------------------------------ dependent launches

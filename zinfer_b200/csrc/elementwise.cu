@@ -404,9 +404,9 @@ __global__ void layernorm_vec4_kernel(const float* __restrict__ x, const int* __
 }
 
 // A gate per value: rows[t, h, j] *= sigmoid(gate[t * ld_gate + h * valid + j]) for j < valid, in place; a head's row is
-// `width` values of which the first `valid` are gated (the rest is padding and left alone).  gate float32.
-template <typename T>
-__global__ void value_gate_kernel(T* __restrict__ rows, const float* __restrict__ gate, int ld_gate, int n, int H, int width,
+// `width` values of which the first `valid` are gated (the rest is padding and left alone).  gate float32 or bfloat16.
+template <typename T, typename TG>
+__global__ void value_gate_kernel(T* __restrict__ rows, const TG* __restrict__ gate, int ld_gate, int n, int H, int width,
                                   int valid) {
   zk_let_next_start();
   zk_wait_prior();
@@ -414,23 +414,36 @@ __global__ void value_gate_kernel(T* __restrict__ rows, const float* __restrict_
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     const size_t th = i / valid, t = th / H;
     const int j = (int)(i - th * valid), hh = (int)(th - t * H);
-    const float g = gate[t * ld_gate + (size_t)hh * valid + j];
+    const float g = to_f32(gate[t * ld_gate + (size_t)hh * valid + j]);
     T* v = rows + th * width + j;
     *v = from_f32<T>(to_f32(*v) / (1.0f + expf(-g)));
   }
 }
 
 // The same for bfloat16 rows in 16-byte pieces (width and valid multiples of 8, gate rows 16-byte aligned).
-__global__ void value_gate_vec8_kernel(uint4* __restrict__ rows, const float* __restrict__ gate, int ld_gate, int pieces, int H,
+template <typename TG>
+__global__ void value_gate_vec8_kernel(uint4* __restrict__ rows, const TG* __restrict__ gate, int ld_gate, int pieces, int H,
                                        int per_head, int valid_pieces) {
   zk_let_next_start();
   zk_wait_prior();
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= pieces) return;
   const int th = i / valid_pieces, j = i - th * valid_pieces, t = th / H, hh = th - t * H;
-  const float4* g4 = reinterpret_cast<const float4*>(gate + (size_t)t * ld_gate + ((size_t)hh * valid_pieces + j) * 8);
-  const float4 ga = g4[0], gb = g4[1];
-  const float g[8] = {ga.x, ga.y, ga.z, ga.w, gb.x, gb.y, gb.z, gb.w};
+  const TG* src = gate + (size_t)t * ld_gate + ((size_t)hh * valid_pieces + j) * 8;
+  float g[8];
+  if constexpr (sizeof(TG) == 4) {
+    const float4* g4 = reinterpret_cast<const float4*>(src);
+    const float4 ga = g4[0], gb = g4[1];
+    g[0] = ga.x, g[1] = ga.y, g[2] = ga.z, g[3] = ga.w, g[4] = gb.x, g[5] = gb.y, g[6] = gb.z, g[7] = gb.w;
+  } else {
+    const uint4 raw = *reinterpret_cast<const uint4*>(src);
+    const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float2 f = __bfloat1622float2(h2[k]);
+      g[2 * k] = f.x, g[2 * k + 1] = f.y;
+    }
+  }
   uint4* dst = rows + (size_t)th * per_head + j;
   uint4 v = *dst;
   __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&v);
@@ -444,10 +457,15 @@ __global__ void value_gate_vec8_kernel(uint4* __restrict__ rows, const float* __
 
 // Heads divided by their root mean square and gated: y[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) *
 // silu(gate[t * ld_gate + h * e + :]).  o and gate float32 (o rows packed, H * e wide), y in the run dtype.
+// Options: a weight after the norm (`w`, w_stride floats from head to head: 0 = one of e values shared by the heads, e = one
+// per head and value); sigmoid(gate) in place of silu; and heads that come as a numerator and a denominator of a normalised
+// memory (`den_log` [n, H] not null): a head's row of o is then e + 1 values apart, its last value the product of normaliser
+// and query, and the head is out_scale * o / (max(|out_scale * o_e|, exp(-den_log)) + 1e-6).
 // One warp per (token, head); the sum of squares is added in lane order then over the warp's tree.
 template <typename TO>
 __global__ void unit_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ gate, int ld_gate,
-                                      TO* __restrict__ y, long long items, int H, int e, float eps) {
+                                      TO* __restrict__ y, long long items, int H, int e, float eps, const float* __restrict__ w,
+                                      int w_stride, int sigmoid, const float* __restrict__ den_log, float out_scale) {
   zk_let_next_start();
   zk_wait_prior();
   const int lane = threadIdx.x & 31;
@@ -455,15 +473,18 @@ __global__ void unit_norm_gate_kernel(const float* __restrict__ o, const float* 
   if (item >= items) return;
   const long long t = item / H;
   const int h = (int)(item - t * H);
-  const float* src = o + (size_t)item * e;
+  const float* src = o + (size_t)item * (den_log ? e + 1 : e);
   const float* g = gate + (size_t)t * ld_gate + (size_t)h * e;
   float ss = 0.f;
   for (int j = lane; j < e; j += 32) ss = fmaf(src[j], src[j], ss);
   ss = warp_sum(ss);
-  const float scale = 1.0f / sqrtf(ss / (float)e + eps);
+  float mul = 1.0f;          // what a value is multiplied by before the norm
+  if (den_log) mul = out_scale / (fmaxf(fabsf(out_scale * src[e]), expf(-den_log[item])) + 1e-6f);
+  const float scale = mul / sqrtf(ss * (mul * mul) / (float)e + eps);
+  const float* wh = w ? w + (size_t)h * w_stride : nullptr;
   for (int j = lane; j < e; j += 32) {
-    const float z = g[j];
-    y[(size_t)item * e + j] = from_f32<TO>((src[j] * scale) * (z / (1.0f + expf(-z))));
+    const float z = g[j], s = (sigmoid ? 1.0f : z) / (1.0f + expf(-z));
+    y[(size_t)item * e + j] = from_f32<TO>((src[j] * scale) * (wh ? wh[j] * s : s));
   }
 }
 
@@ -509,22 +530,6 @@ __global__ void rmsnorm_pair_add_kernel(const float* __restrict__ a, const float
     }
   } else {
     for (int d = threadIdx.x; d < dim; d += blockDim.x) xr[d] += share * ((ar[d] * ra) * wa[d] + (br[d] * rb) * wb[d]);
-  }
-}
-
-// Activations of a plain (ungated) feed-forward, float32 arithmetic:
-// 0 = gelu with erf: 0.5 z (1 + erf(z / sqrt 2)); 1 = gelu with tanh:
-// 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))); 2 = silu; 3 = relu; 4 = the square of relu.
-__device__ __forceinline__ float zk_activate(float z, int kind) {
-  switch (kind) {
-    case 0: return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f));
-    case 1: return 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
-    case 2: return z / (1.0f + expf(-z));
-    case 4: {
-      const float r = fmaxf(z, 0.f);
-      return r * r;
-    }
-    default: return fmaxf(z, 0.f);
   }
 }
 
@@ -1180,37 +1185,45 @@ int zk_layernorm(const float* x, const int* rows, const float* w, const float* b
   return ZK_EINVAL;
 }
 
-// rows [n, H * width] (run dtype) gated value by value: gate float32, rows `ld_gate` apart, H * valid logits a row.
-int zk_value_gate(void* rows, const float* gate, int ld_gate, int n, int H, int width, int valid, int dtype,
+// rows [n, H * width] (run dtype) gated value by value: gate float32 or bfloat16, rows `ld_gate` apart, H * valid logits a row.
+int zk_value_gate(void* rows, const void* gate, int ld_gate, int n, int H, int width, int valid, int dtype, int gate_dtype,
                   cudaStream_t stream) {
   if (n <= 0) return 0;
   if (H <= 0 || width <= 0 || valid <= 0 || valid > width || ld_gate < H * valid) return ZK_EINVAL;
-  if (dtype == ZK_BF16 && width % 8 == 0 && valid % 8 == 0 && ld_gate % 4 == 0 && (uintptr_t)rows % 16 == 0 &&
+  if (gate_dtype != ZK_F32 && gate_dtype != ZK_BF16) return ZK_EINVAL;
+  const bool gf = gate_dtype == ZK_F32;
+  if (dtype == ZK_BF16 && width % 8 == 0 && valid % 8 == 0 && ld_gate % (gf ? 4 : 8) == 0 && (uintptr_t)rows % 16 == 0 &&
       (uintptr_t)gate % 16 == 0 && (size_t)n * H * (valid / 8) < 0x7fffffffULL) {
     const int pieces = n * H * (valid / 8);
-    return zk_launch_dependent(value_gate_vec8_kernel, dim3((pieces + 255) / 256), dim3(256), 0, stream, (uint4*)rows, gate,
-                               ld_gate, pieces, H, width / 8, valid / 8);
+    const dim3 grid((pieces + 255) / 256);
+    if (gf)
+      return zk_launch_dependent(value_gate_vec8_kernel<float>, grid, dim3(256), 0, stream, (uint4*)rows, (const float*)gate, ld_gate, pieces, H, width / 8, valid / 8);
+    return zk_launch_dependent(value_gate_vec8_kernel<bf16>, grid, dim3(256), 0, stream, (uint4*)rows, (const bf16*)gate, ld_gate, pieces, H, width / 8, valid / 8);
   }
   const int threads = 256, blocks = grid_for_total((size_t)n * H * valid, threads);
-  if (dtype == ZK_F32)
-    return zk_launch_dependent(value_gate_kernel<float>, dim3(blocks), dim3(threads), 0, stream, (float*)rows, gate, ld_gate, n, H, width, valid);
-  if (dtype == ZK_BF16)
-    return zk_launch_dependent(value_gate_kernel<bf16>, dim3(blocks), dim3(threads), 0, stream, (bf16*)rows, gate, ld_gate, n, H, width, valid);
+#define ZK_VG(T, TG) \
+  return zk_launch_dependent(value_gate_kernel<T, TG>, dim3(blocks), dim3(threads), 0, stream, (T*)rows, (const TG*)gate, ld_gate, n, H, width, valid)
+  if (dtype == ZK_F32 && gf) ZK_VG(float, float);
+  if (dtype == ZK_F32) ZK_VG(float, bf16);
+  if (dtype == ZK_BF16 && gf) ZK_VG(bf16, float);
+  if (dtype == ZK_BF16) ZK_VG(bf16, bf16);
+#undef ZK_VG
   return ZK_EINVAL;
 }
 
-// y [n, H * e] (out_dtype) = every head of o [n, H * e] (float32) over its root mean square, times silu(gate).
+// y [n, H * e] (out_dtype) = every head of o [n, H * e] (float32; [n, H * (e + 1)] with den_log) over its root mean square, times
+// silu(gate); weight, gate form and denominator as unit_norm_gate_kernel says.
 int zk_unit_norm_gate(const float* o, const float* gate, int ld_gate, void* y, int n, int H, int e, float eps, int out_dtype,
-                      cudaStream_t stream) {
+                      const float* w, int w_stride, int sigmoid, const float* den_log, float out_scale, cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (H <= 0 || e <= 0 || ld_gate < H * e) return ZK_EINVAL;
+  if (H <= 0 || e <= 0 || ld_gate < H * e || (w && w_stride != 0 && w_stride != e)) return ZK_EINVAL;
   const long long items = (long long)n * H;
   const int warps = 4;
   const int blocks = (int)((items + warps - 1) / warps);
   if (out_dtype == ZK_F32)
-    return zk_launch_dependent(unit_norm_gate_kernel<float>, dim3(blocks), dim3(warps * 32), 0, stream, o, gate, ld_gate, (float*)y, items, H, e, eps);
+    return zk_launch_dependent(unit_norm_gate_kernel<float>, dim3(blocks), dim3(warps * 32), 0, stream, o, gate, ld_gate, (float*)y, items, H, e, eps, w, w_stride, sigmoid, den_log, out_scale);
   if (out_dtype == ZK_BF16)
-    return zk_launch_dependent(unit_norm_gate_kernel<bf16>, dim3(blocks), dim3(warps * 32), 0, stream, o, gate, ld_gate, (bf16*)y, items, H, e, eps);
+    return zk_launch_dependent(unit_norm_gate_kernel<bf16>, dim3(blocks), dim3(warps * 32), 0, stream, o, gate, ld_gate, (bf16*)y, items, H, e, eps, w, w_stride, sigmoid, den_log, out_scale);
   return ZK_EINVAL;
 }
 

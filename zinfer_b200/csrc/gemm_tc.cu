@@ -988,11 +988,12 @@ int zk_gemm_tc(const void* X, const void* W, void* C, const float* bias, int M, 
 
 // Grouped product: X [M, K] holds token tiles of 128 rows (M a multiple of 128), W [groups, N, K] contiguous
 // matrices, tile_group [M / 128] (device, int32) names each tile's matrix; C [M, N] (or [M, N/2] with
-// `swiglu`, W's rows then being groups of 16 gate rows and their 16 up rows), bfloat16 or float32.
+// `swiglu`, W's rows then being groups of 16 gate rows and their 16 up rows), bfloat16 or float32.  act 1: the square of relu
+// of the result, where the persistent form runs (N a multiple of 256).
 int zk_gemm_tc_grouped(const void* X, const void* W, void* C, int M, int N, int K, int groups, int ldx, int ldc,
-                       int out_dtype, int swiglu, const int* tile_group, int* status, cudaStream_t stream) {
+                       int out_dtype, int swiglu, const int* tile_group, int* status, int act, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
-  if (M % BM || groups <= 0 || !tile_group || !status) return ZK_EINVAL;
+  if (M % BM || groups <= 0 || !tile_group || !status || act < 0 || act > 1 || (act && swiglu)) return ZK_EINVAL;
   if (K <= 0 || K % 8 || ldx % 8 || ldx < K || ldc < (swiglu ? N / 2 : N) || (swiglu && N % 32)) return ZK_EINVAL;
   if ((long long)groups * N > 0x7fffffffLL) return ZK_EINVAL;
   if (((uintptr_t)X | (uintptr_t)W | (uintptr_t)C) % 16) return ZK_EINVAL;
@@ -1001,6 +1002,7 @@ int zk_gemm_tc_grouped(const void* X, const void* W, void* C, int M, int N, int 
   p.C = C; p.status = status;
   p.M = M; p.N = N; p.K = K; p.ldc = ldc; p.splits = 1; p.swiglu = swiglu;
   p.tile_group = tile_group;
+  p.act = act;
   CUtensorMap ma, mb, mc;
   const bool f32 = out_dtype == ZK_F32;
   if (N % 256 == 0 && (ldc * (f32 ? 4 : 2)) % 16 == 0 && forced_form != 0) {
@@ -1013,6 +1015,7 @@ int zk_gemm_tc_grouped(const void* X, const void* W, void* C, int M, int N, int 
     return f32 ? launch_persistent<BW, 4, false, float>(ma, mb, mc, p, n_tiles, stream)
                : launch_persistent<BW, 4, false, bf16>(ma, mb, mc, p, n_tiles, stream);
   }
+  if (act) return ZK_EINVAL;
   constexpr int BN = 128;
   if (!make_map(&ma, X, M, K, ldx, BM) || !make_map(&mb, W, groups * N, K, K, BN)) return ZK_EINVAL;
   dim3 grid(M / BM, ceil_div_i(N, BN), 1);

@@ -17,24 +17,41 @@
 // registers while the current sixteen are worked on, and go into the other half of a double buffer.  The order of every sum is fixed by the layout alone, so a
 // sequence cut into steps gives the same bits as the whole.
 //
-// The same kernel runs two more recurrences.  KEYED: a retention layer's, a key projection in place of the gate and one
+// The same kernel runs three more recurrences.  KEYED: a retention layer's, a key projection in place of the gate and one
 // fixed decay per head, S_t = decay_h S_{t-1} + k_t v_t^T; retention_prepare_kernel rotates q and k and scales k first.
 // STEPPED: a state-space layer's (Mamba-2), whose step size dt_t > 0 per head and token sets both the decay and what enters,
 // S_t = exp(-exp(A_log_h) dt_t) S_{t-1} + dt_t k_t v_t^T, o_t = S_t^T q_t + skip_h v_t, with k and q shared by the heads of
 // a group; lane i of every warp turns the raw step size of a group's token i into dt = softplus(z + bias) and the decay.
+// CAPPED: a matrix memory with exponential gates (the mLSTM of xLSTM): the logarithms of the gates, i_t = cap tanh(z_i / cap) and
+// f_t = logsigmoid(cap tanh(z_f / cap)), meet in a running maximum m_t = max(f_t + m_{t-1}, i_t), m_0 = 0, and
+// S_t = exp(f_t + m_{t-1} - m_t) S_{t-1} + exp(i_t - m_t) k_t v_t^T.  The values get one more column, which is 1 for every token:
+// that column of S is the memory's normaliser and its read-out the product of normaliser and query.  Lane i of every warp turns
+// the raw gates of a group's token i into logarithms when the group is staged; the maxima of a group are a scan over the lanes
+// (a token maps m to max(f + m, i), and such maps compose).
 #include "common.cuh"
 #include <math.h>
 
 #define HG_R 8             // warps of a block, each with a stretch of the d channels
 #define HG_MAX_D 512
 
-enum { REC_GATED = 0, REC_KEYED = 1, REC_STEPPED = 2 };
+enum { REC_GATED = 0, REC_KEYED = 1, REC_STEPPED = 2, REC_CAPPED = 3 };
 
 // Where a STEPPED recurrence's operands lie and its numbers per head.  Rows of the float32 input hold the values [H * e] at
 // column 0, the keys [groups * d] at off_k, the queries [groups * d] at off_q; z holds the raw step sizes, rows ld_z apart.
 struct Stepped {
   const float *z, *dt_bias, *a_log, *skip;
   int ld_z, off_k, off_q, heads_per_group;
+};
+
+// What a CAPPED recurrence needs besides the rows [q (H*d) | k (H*d) | v (H*ev) | ...]: raw gates zi, zf [n, H] (rows ld_z apart),
+// their biases [H], the cap; m_out [n, H]: the maximum after every token; max_at: where, behind a slot's matrices, the running
+// maxima lie ([H, column blocks]: each block of columns keeps its own copy, so none reads what another has moved on).
+struct Capped {
+  const float *zi, *zf, *bi, *bf;
+  float* m_out;
+  float cap;
+  int ld_z, ev;
+  long long max_at;
 };
 
 // In place on the rows of qfv: q <- silu(q), f <- lower + (1 - lower) * sigmoid(f + bias); v is left alone.
@@ -98,7 +115,7 @@ template <int DPT, int TT, int REC>
 __global__ void __launch_bounds__(HG_R * 32)
     hgrn2_scan_kernel(const float* __restrict__ qfv, int ld, float* __restrict__ state, long long state_stride,
                       float* __restrict__ o, const int* __restrict__ cu_q, const int* __restrict__ seq_slot, int H, int d,
-                      int e, const float* __restrict__ decay, Stepped sp) {
+                      int e, const float* __restrict__ decay, Stepped sp, Capped cp) {
   constexpr int DM = HG_R * DPT;                                     // channels the block covers, >= d
   constexpr int NL = (TT * DM + HG_R * 32 - 1) / (HG_R * 32);     // q (and f) values a thread fetches per group of tokens
   __shared__ __align__(16) float qs[2][TT][DM];
@@ -123,6 +140,9 @@ __global__ void __launch_bounds__(HG_R * 32)
   const float skip = REC == REC_STEPPED ? sp.skip[h] : 0.f, dt_bias = REC == REC_STEPPED ? sp.dt_bias[h] : 0.f;
   const float rate = REC == REC_STEPPED ? -expf(sp.a_log[h]) : 0.f;
   float* st = state + (size_t)seq_slot[b] * state_stride + (size_t)h * d * e;
+  float* st_max = REC == REC_CAPPED ? state + (size_t)seq_slot[b] * state_stride + cp.max_at + (size_t)h * gridDim.z + blockIdx.z : nullptr;
+  float m_run = REC == REC_CAPPED ? *st_max : 0.f;      // the running maximum before the group that is staged next
+  const float bias_i = REC == REC_CAPPED ? cp.bi[h] : 0.f, bias_f = REC == REC_CAPPED ? cp.bf[h] : 0.f;
   float S[DPT];
 #pragma unroll
   for (int k = 0; k < DPT; ++k) S[k] = (col && row0 + k < d) ? st[(size_t)(row0 + k) * e + c] : 0.f;
@@ -130,7 +150,8 @@ __global__ void __launch_bounds__(HG_R * 32)
   const int head_q = REC == REC_STEPPED ? sp.off_q + h / sp.heads_per_group * d : h * d;       // columns of this head's q
   const int off_f = REC == REC_STEPPED ? sp.off_k - sp.off_q : H * d, off_v = REC == REC_STEPPED ? 0 : 2 * H * d;
   float rq[NL], rf[NL], v_cur[TT], v_next[TT];
-  float rz = 0.f, lane_decay = 0.f, lane_dt = 0.f;      // REC_STEPPED: the raw step size, decay and dt of token `lane` of a group
+  // REC_STEPPED: the raw step size, decay and dt of token `lane` of a group; REC_CAPPED: its raw gates, what S keeps and what enters
+  float rz = 0.f, rz2 = 0.f, lane_decay = 0.f, lane_dt = 0.f;
   // where a thread's n-th value of a group comes from (relative to the group's first row) and goes to
   int src[NL], dst[NL];
 #pragma unroll
@@ -151,8 +172,13 @@ __global__ void __launch_bounds__(HG_R * 32)
     }
 #pragma unroll
     for (int tt = 0; tt < TT; ++tt)
-      v_next[tt] = (col && tt < nt) ? base[(size_t)tt * ld + off_v + h * e + c] : 0.f;
+      if (REC == REC_CAPPED) v_next[tt] = (col && tt < nt) ? (c < cp.ev ? base[(size_t)tt * ld + off_v + h * cp.ev + c] : 1.0f) : 0.f;
+      else v_next[tt] = (col && tt < nt) ? base[(size_t)tt * ld + off_v + h * e + c] : 0.f;
     if (REC == REC_STEPPED && lane < nt) rz = sp.z[(size_t)(tb + lane) * sp.ld_z + h];
+    if (REC == REC_CAPPED && lane < nt) {
+      rz = cp.zi[(size_t)(tb + lane) * cp.ld_z + h];
+      rz2 = cp.zf[(size_t)(tb + lane) * cp.ld_z + h];
+    }
   };
   auto stage = [&](int buf, int tb) {
     const int nt = min(TT, t1 - tb);
@@ -169,6 +195,26 @@ __global__ void __launch_bounds__(HG_R * 32)
       const float z = rz + dt_bias;
       lane_dt = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));      // softplus
       lane_decay = expf(rate * lane_dt);
+    }
+    if (REC == REC_CAPPED) {
+      const float gi = cp.cap * tanhf((rz + bias_i) / cp.cap), zf = cp.cap * tanhf((rz2 + bias_f) / cp.cap);
+      const float gf = -(fmaxf(-zf, 0.f) + log1pf(expf(-fabsf(zf))));      // the logarithm of a sigmoid
+      float A = gf, B = gi;            // tokens 0 .. lane as one map of m: max(A + m, B)
+#pragma unroll
+      for (int s = 1; s < TT; s <<= 1) {
+        const float pa = __shfl_up_sync(0xffffffffu, A, s), pb = __shfl_up_sync(0xffffffffu, B, s);
+        if (lane >= s) {
+          B = fmaxf(A + pb, B);
+          A += pa;
+        }
+      }
+      const float m = fmaxf(A + m_run, B);
+      float before = __shfl_up_sync(0xffffffffu, m, 1);
+      if (lane == 0) before = m_run;
+      lane_decay = expf(gf + before - m);
+      lane_dt = expf(gi - m);
+      if (warp == 0 && blockIdx.z == 0 && lane < nt) cp.m_out[(size_t)(tb + lane) * H + h] = m;
+      m_run = __shfl_sync(0xffffffffu, m, nt - 1);
     }
   };
 
@@ -187,6 +233,10 @@ __global__ void __launch_bounds__(HG_R * 32)
       float acc = 0.f;
       if (REC == REC_STEPPED) {
         if (warp == 0) acc = skip * v;
+        keep = __shfl_sync(0xffffffffu, lane_decay, tt);
+        v *= __shfl_sync(0xffffffffu, lane_dt, tt);
+      }
+      if (REC == REC_CAPPED) {
         keep = __shfl_sync(0xffffffffu, lane_decay, tt);
         v *= __shfl_sync(0xffffffffu, lane_dt, tt);
       }
@@ -243,6 +293,7 @@ __global__ void __launch_bounds__(HG_R * 32)
     for (int k = 0; k < DPT; ++k)
       if (row0 + k < d) st[(size_t)(row0 + k) * e + c] = S[k];
   }
+  if (REC == REC_CAPPED && tid == 0) *st_max = m_run;
 }
 
 extern "C" {
@@ -268,7 +319,7 @@ int zk_hgrn2_scan(float* qfv, int ld, const float* f_bias, const float* lower, f
   dim3 grid(n_seqs, H, (e + 31) / 32);
 #define ZK_HG(DP)                                                                                                    \
   return zk_launch_dependent(hgrn2_scan_kernel<DP, (DP > 32 ? 4 : (DP > 16 ? 8 : 16)), REC_GATED>, grid, dim3(HG_R * 32), 0, stream, (const float*)qfv, ld, \
-                             state, state_stride, o, cu_q, seq_slot, H, d, e, (const float*)nullptr, Stepped{})
+                             state, state_stride, o, cu_q, seq_slot, H, d, e, (const float*)nullptr, Stepped{}, Capped{})
   const int dpt = (d + HG_R - 1) / HG_R;
   if (dpt <= 1) ZK_HG(1);
   if (dpt <= 2) ZK_HG(2);
@@ -299,7 +350,7 @@ int zk_retention_scan(float* qkv, int ld, const float* decay, const float* inv_f
   dim3 grid(n_seqs, H, (e + 31) / 32);
 #define ZK_RT(DP)                                                                                                    \
   return zk_launch_dependent(hgrn2_scan_kernel<DP, (DP > 32 ? 4 : (DP > 16 ? 8 : 16)), REC_KEYED>, grid, dim3(HG_R * 32), 0, stream, (const float*)qkv, ld, \
-                             state, state_stride, o, cu_q, seq_slot, H, d, e, decay, Stepped{})
+                             state, state_stride, o, cu_q, seq_slot, H, d, e, decay, Stepped{}, Capped{})
   const int dpt = (d + HG_R - 1) / HG_R;
   if (dpt <= 1) ZK_RT(1);
   if (dpt <= 2) ZK_RT(2);
@@ -324,7 +375,7 @@ int zk_ssd_scan(const float* xbc, int ld, const float* z, int ld_z, const float*
   dim3 grid(n_seqs, H, (e + 31) / 32);
 #define ZK_SS(DP)                                                                                                    \
   return zk_launch_dependent(hgrn2_scan_kernel<DP, (DP > 32 ? 4 : (DP > 16 ? 8 : 16)), REC_STEPPED>, grid, dim3(HG_R * 32), 0, stream, xbc, ld, \
-                             state, state_stride, o, cu_q, seq_slot, H, d, e, (const float*)nullptr, sp)
+                             state, state_stride, o, cu_q, seq_slot, H, d, e, (const float*)nullptr, sp, Capped{})
   const int dpt = (d + HG_R - 1) / HG_R;
   if (dpt <= 1) ZK_SS(1);
   if (dpt <= 2) ZK_SS(2);
@@ -334,6 +385,35 @@ int zk_ssd_scan(const float* xbc, int ld, const float* z, int ld_z, const float*
   if (dpt <= 32) ZK_SS(32);
   ZK_SS(64);
 #undef ZK_SS
+}
+
+// Floats of state a slot of zk_mlstm_scan needs: matrices [H, d, e + 1] and the running maxima.
+int zk_mlstm_state_floats(int H, int d, int e) { return H * d * (e + 1) + H * ((e + 1 + 31) / 32); }
+
+// Matrix memory with exponential gates (mLSTM): qkv float32 [n, >= 2*H*d + H*e] with rows `ld` floats apart, [q | k | v | ...] as the
+// projections gave them; zi, zf float32 [n, >= H] raw gates, rows ld_z apart, bi, bf [H]; state float32, a slot's
+// zk_mlstm_state_floats `state_stride` floats after the one before, zero when a sequence starts; o float32 [n, H * (e + 1)]: per head
+// the e sums S_t^T q_t and, last, the product of normaliser and query; m_out [n, H]: the running maximum after every token.
+int zk_mlstm_scan(const float* qkv, int ld, const float* zi, const float* zf, int ld_z, const float* bi, const float* bf, float cap,
+                  float* state, long long state_stride, float* o, float* m_out, const int* cu_q, const int* seq_slot, int n,
+                  int n_seqs, int H, int d, int e, cudaStream_t stream) {
+  if (n_seqs <= 0 || n <= 0) return 0;
+  if (H <= 0 || d <= 0 || e <= 0 || d > HG_MAX_D || !(cap > 0.f)) return ZK_EINVAL;
+  if (ld < 2 * H * d + H * e || ld_z < H || !zi || !zf || !bi || !bf || !m_out) return ZK_EINVAL;
+  const Capped cp{zi, zf, bi, bf, m_out, cap, ld_z, e, (long long)H * d * (e + 1)};
+  dim3 grid(n_seqs, H, (e + 1 + 31) / 32);
+#define ZK_ML(DP)                                                                                                    \
+  return zk_launch_dependent(hgrn2_scan_kernel<DP, (DP > 32 ? 4 : (DP > 16 ? 8 : 16)), REC_CAPPED>, grid, dim3(HG_R * 32), 0, stream, qkv, ld, \
+                             state, state_stride, o, cu_q, seq_slot, H, d, e + 1, (const float*)nullptr, Stepped{}, cp)
+  const int dpt = (d + HG_R - 1) / HG_R;
+  if (dpt <= 1) ZK_ML(1);
+  if (dpt <= 2) ZK_ML(2);
+  if (dpt <= 4) ZK_ML(4);
+  if (dpt <= 8) ZK_ML(8);
+  if (dpt <= 16) ZK_ML(16);
+  if (dpt <= 32) ZK_ML(32);
+  ZK_ML(64);
+#undef ZK_ML
 }
 
 }  // extern "C"

@@ -10,6 +10,10 @@
 // the contraction kernels with an activation epilogue want), down as [experts, D, F]; x and h are the run
 // dtype, y float32.
 //
+// Options of experts picked by a router: no gate (an expert is W_down act(W_up x), its stacked first matrix [experts, F, D]),
+// and weights that multiply what an expert READS instead of what it returns; W_up (w x) = w (W_up x), so the first kernel
+// multiplies its sums by the weight before the activation.
+//
 // For steps of many tokens there are two helper kernels instead: rows gathered in the order of their
 // experts (so that each expert's rows are one contiguous matrix for a tensor-core contraction) and the
 // weighted sum of a token's `top` result rows, added in the order of k.
@@ -97,11 +101,14 @@ __device__ __forceinline__ int moe_expert(const int* __restrict__ tokens, const 
   return e;
 }
 
-template <typename T, bool VEC>
+// act < 0: gated (silu(gate) * up), rows of w_gu as above; else ungated, act numbers the activation (zk_activate), w_gu
+// [experts, F, D].  in_w [n, top] (or null): the weight of each pair's input.
+template <typename T, bool VEC, bool GATED>
 __global__ void __launch_bounds__(MOE_WARPS * 32)
     moe_gate_up_kernel(const T* __restrict__ x, const int* __restrict__ tokens, const int* __restrict__ table,
                        const T* __restrict__ w_gu, int il, T* __restrict__ h, int D, int F,
-                       int top, int vocab, int n_experts, int units_per_block, int* status, int n_ident) {
+                       int top, int vocab, int n_experts, int units_per_block, int* status, int n_ident, int act,
+                       const float* __restrict__ in_w) {
   extern __shared__ float xs[];     // [D]
   zk_let_next_start();
   zk_wait_prior();
@@ -111,8 +118,25 @@ __global__ void __launch_bounds__(MOE_WARPS * 32)
   if (e >= n_experts) return;       // an identity expert has no hidden units
   for (int d = threadIdx.x; d < D; d += blockDim.x) xs[d] = to_f32(x[(size_t)t * D + d]);
   __syncthreads();
-  const T* w = w_gu + (size_t)e * 2 * F * D;
+  const T* w = w_gu + (size_t)e * (GATED ? 2 : 1) * F * D;
   const int f0 = blockIdx.y * units_per_block, f1 = min(F, f0 + units_per_block);
+  const float wi = in_w ? in_w[(size_t)t * top + k] : 1.0f;
+  if constexpr (!GATED) {
+    for (int fb = f0 + warp * MOE_UNITS; fb < f1; fb += MOE_WARPS * MOE_UNITS) {
+      const T* rows[MOE_UNITS];
+#pragma unroll
+      for (int u = 0; u < MOE_UNITS; ++u) rows[u] = w + (size_t)min(fb + u, f1 - 1) * D;
+      float dot[MOE_UNITS];
+      rows_dot<T, VEC, MOE_UNITS>(rows, xs, D, lane, dot);
+      if (lane < MOE_UNITS && fb + lane < f1) {
+        float z = 0.f;
+#pragma unroll
+        for (int i = 0; i < MOE_UNITS; ++i)
+          if (lane == i) z = dot[i];
+        h[((size_t)t * top + k) * F + fb + lane] = from_f32<T>(zk_activate(wi * z, act));
+      }
+    }
+  } else
   for (int fb = f0 + warp * MOE_UNITS; fb < f1; fb += MOE_WARPS * MOE_UNITS) {
     const T* rows[2 * MOE_UNITS];
 #pragma unroll
@@ -130,8 +154,8 @@ __global__ void __launch_bounds__(MOE_WARPS * 32)
 #pragma unroll
       for (int i = 0; i < MOE_UNITS; ++i)
         if (lane == i) {
-          g = dot[2 * i];
-          u = dot[2 * i + 1];
+          g = wi * dot[2 * i];
+          u = wi * dot[2 * i + 1];
         }
       h[((size_t)t * top + k) * F + fb + lane] = from_f32<T>(g / (1.0f + expf(-g)) * u);
     }
@@ -143,8 +167,8 @@ __global__ void __launch_bounds__(MOE_WARPS * 32)
     moe_down_kernel(const T* __restrict__ h, const int* __restrict__ tokens, const int* __restrict__ table,
                     const T* __restrict__ w_down, float* __restrict__ y, int D, int F, int top, int vocab,
                     int n_experts, int outs_per_block, int accumulate, int* status, const float* __restrict__ route_w,
-                    int n_ident, const T* __restrict__ x) {
-  // route_w [n, top]: the weight of each of the token's experts (null: 1/top each).  x [n, D]: the rows the experts
+                    int n_ident, const T* __restrict__ x, float weight) {
+  // route_w [n, top]: the weight of each of the token's experts (null: `weight` each).  x [n, D]: the rows the experts
   // read, which an identity expert (n_ident > 0) hands on as they are.
   extern __shared__ float hs[];     // [top][F]
   zk_let_next_start();
@@ -153,7 +177,6 @@ __global__ void __launch_bounds__(MOE_WARPS * 32)
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   for (int i = threadIdx.x; i < top * F; i += blockDim.x) hs[i] = to_f32(h[(size_t)t * top * F + i]);
   __syncthreads();
-  const float weight = 1.0f / (float)top;
   const int d0 = blockIdx.y * outs_per_block, d1 = min(D, d0 + outs_per_block);
   for (int db = d0 + warp * MOE_UNITS; db < d1; db += MOE_WARPS * MOE_UNITS) {
     float acc[MOE_UNITS];
@@ -189,20 +212,34 @@ __global__ void __launch_bounds__(MOE_WARPS * 32)
 }
 
 template <typename T>
-__global__ void moe_gather_kernel(const T* __restrict__ x, const int* __restrict__ row_token, T* __restrict__ xg, int D) {
+__global__ void moe_gather_kernel(const T* __restrict__ x, const int* __restrict__ row_token, T* __restrict__ xg, int D,
+                                  const float* __restrict__ pair_w, int top) {
+  // pair_w (or null): row_token then names the row's PAIR t * top + k, and the row is pair_w[pair] * x[t].
   zk_let_next_start();
   zk_wait_prior();
-  const int t = row_token[blockIdx.x];       // < 0: a padding row
+  int t = row_token[blockIdx.x];       // < 0: a padding row
+  float w = 1.0f;
+  if (pair_w && t >= 0) {
+    w = pair_w[t];
+    t /= top;
+  }
   const T* src = x + (size_t)(t < 0 ? 0 : t) * D;
   T* dst = xg + (size_t)blockIdx.x * D;
   constexpr int PER = 16 / (int)sizeof(T);
   if (D % PER == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(xg)) % 16) == 0) {   // rows in 16-byte pieces
     const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-    for (int d = threadIdx.x; d < D / PER; d += blockDim.x)
-      reinterpret_cast<uint4*>(dst)[d] = t < 0 ? zero : reinterpret_cast<const uint4*>(src)[d];
+    for (int d = threadIdx.x; d < D / PER; d += blockDim.x) {
+      uint4 v = t < 0 ? zero : reinterpret_cast<const uint4*>(src)[d];
+      if (pair_w) {
+        T* p = reinterpret_cast<T*>(&v);
+#pragma unroll
+        for (int j = 0; j < PER; ++j) p[j] = from_f32<T>(w * to_f32(p[j]));
+      }
+      reinterpret_cast<uint4*>(dst)[d] = v;
+    }
     return;
   }
-  for (int d = threadIdx.x; d < D; d += blockDim.x) dst[d] = t < 0 ? from_f32<T>(0.f) : src[d];
+  for (int d = threadIdx.x; d < D; d += blockDim.x) dst[d] = t < 0 ? from_f32<T>(0.f) : (pair_w ? from_f32<T>(w * to_f32(src[d])) : src[d]);
 }
 
 // The rows of a prompt step sorted by expert, made where the router left its choice (no trip to the host):
@@ -210,10 +247,11 @@ __global__ void moe_gather_kernel(const T* __restrict__ x, const int* __restrict
 // start_e a multiple of `tile` (every expert's rows are padded to whole tiles); row_token [cap] = the token of each
 // row, -1 for a padding row; pair_row [P] = the row of each pair; tile_group [cap / tile] = the expert of each tile
 // (0 for the tiles behind the last expert's, whose rows are all padding).  cap >= P rounded down to tiles plus one
-// tile per expert.  One block; the order of an expert's rows is not fixed, which no row's result depends on.
+// tile per expert.  With name_pairs row_token holds the row's pair i instead of its token.  One block; the order of an expert's rows is not fixed, which no row's result depends on.
 __global__ void __launch_bounds__(1024)
     moe_expert_rows_kernel(const int* __restrict__ ids, int P, int E, int top, int tile, int cap,
-                           int* __restrict__ row_token, int* __restrict__ pair_row, int* __restrict__ tile_group, int n_ident) {
+                           int* __restrict__ row_token, int* __restrict__ pair_row, int* __restrict__ tile_group, int n_ident,
+                           int name_pairs) {
   extern __shared__ int sh[];      // count [E], start [E]
   int* count = sh;
   int* start = sh + E;
@@ -246,7 +284,7 @@ __global__ void __launch_bounds__(1024)
     }
     const int e = min(max(ids[i], 0), E - 1);
     const int r = start[e] + atomicAdd(&count[e], 1);
-    row_token[r] = i / top;
+    row_token[r] = name_pairs ? i : i / top;
     pair_row[i] = r;
   }
 }
@@ -255,11 +293,10 @@ __global__ void __launch_bounds__(1024)
 // row x[t] (run dtype: float32 or, with x_bf16, bfloat16).
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pair_row, float* __restrict__ out,
                                    int D, int top, int accumulate, const float* __restrict__ route_w,
-                                   const void* __restrict__ x, int x_bf16) {
+                                   const void* __restrict__ x, int x_bf16, float weight) {
   zk_let_next_start();
   zk_wait_prior();
   const int t = blockIdx.x;
-  const float weight = 1.0f / (float)top;
   for (int d = threadIdx.x; d < D; d += blockDim.x) {
     float acc = 0.f;
     for (int k = 0; k < top; ++k) {
@@ -276,12 +313,13 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
 
 // Router of a mixture of experts, one block per token.  The logits are float32 dot products (a warp per expert,
 // lanes striding the row, sums in lane order then the warp's tree), the softmax runs over all E experts, and warp 0
-// then picks the `top` largest scores one after the other (of equal scores the lower index first).
+// then picks the `top` largest scores one after the other (of equal scores the lower index first).  `sigmoid`: a score is the
+// sigmoid of its own logit instead; `renorm` 0: the weights are the chosen scores as they are.
 #define MOE_ROUTER_MAX_EXPERTS 4096
 template <typename T>
 __global__ void __launch_bounds__(MOE_WARPS * 32)
     moe_router_kernel(const T* __restrict__ x, const float* __restrict__ w, int* __restrict__ ids, float* __restrict__ wts,
-                      int D, int E, int top, const float* __restrict__ correction) {
+                      int D, int E, int top, const float* __restrict__ correction, int sigmoid, int renorm) {
   // correction [E] (or null): the experts are CHOSEN by score + correction; the weights use the scores alone.
   extern __shared__ float rs[];     // [D] the token's row, [E] logits then scores, [E] what the choice looks at
   float* xs = rs;
@@ -318,11 +356,11 @@ __global__ void __launch_bounds__(MOE_WARPS * 32)
   m = warp_max(m);
   float sum = 0.f;
   for (int e = lane; e < E; e += 32) {
-    const float v = expf(z[e] - m);
+    const float v = sigmoid ? 1.0f / (1.0f + expf(-z[e])) : expf(z[e] - m);
     z[e] = v;
     sum += v;
   }
-  sum = warp_sum(sum);
+  sum = sigmoid ? 1.0f : warp_sum(sum);
   __syncwarp();
   for (int e = lane; e < E; e += 32) pick[e] = correction ? z[e] / sum + correction[e] : z[e];
   __syncwarp();
@@ -355,6 +393,7 @@ __global__ void __launch_bounds__(MOE_WARPS * 32)
     chosen_sum += score;
     __syncwarp();
   }
+  if (!renorm) return;
   const float inv = 1.0f / (chosen_sum + 1e-20f);
   __syncwarp();
   for (int k = lane; k < top; k += 32) wts[(size_t)t * top + k] *= inv;
@@ -365,7 +404,7 @@ namespace {
 template <typename T>
 int launch_moe(const void* x, const int* tokens, const int* table, const void* w_gu, int il,
                const void* w_down, void* h, float* y, int n, int D, int F, int top, int vocab, int n_experts,
-               int accumulate, int* status, const float* route_w, int n_ident, cudaStream_t stream) {
+               int accumulate, int* status, const float* route_w, int n_ident, int act, const float* in_w, cudaStream_t stream) {
   const int per = 16 / (int)sizeof(T);   // elements per 16 bytes
   auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
   const bool vec_gu = D % 8 == 0 && D % per == 0 && aligned(w_gu);
@@ -382,15 +421,16 @@ int launch_moe(const void* x, const int* tokens, const int* table, const void* w
   if (smem_gu > 200 * 1024 || smem_dn > 200 * 1024) return ZK_EINVAL;
   const dim3 grid_gu((unsigned)pairs, (F + units - 1) / units), grid_dn(n, (D + outs - 1) / outs);
   int rc;
-#define ZK_MOE_GU(V)                                                                                                  \
+#define ZK_MOE_GU(V, G)                                                                                                  \
   do {                                                                                                                \
-    auto kern = moe_gate_up_kernel<T, V>;                                                                             \
+    auto kern = moe_gate_up_kernel<T, V, G>;                                                                           \
     if (smem_gu > 48 * 1024) {                                                                                        \
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_gu);          \
       if (e != cudaSuccess) return (int)e;                                                                            \
     }                                                                                                                 \
     rc = zk_launch_dependent(kern, grid_gu, dim3(MOE_WARPS * 32), smem_gu, stream, (const T*)x, tokens, table,        \
-                             (const T*)w_gu, il, (T*)h, D, F, top, vocab, n_experts, units, status, n_ident);         \
+                             (const T*)w_gu, il, (T*)h, D, F, top, vocab, n_experts, units, status, n_ident, act,     \
+                             in_w);                                                                                   \
   } while (0)
 #define ZK_MOE_DN(V)                                                                                                  \
   do {                                                                                                                \
@@ -401,9 +441,13 @@ int launch_moe(const void* x, const int* tokens, const int* table, const void* w
     }                                                                                                                 \
     rc = zk_launch_dependent(kern, grid_dn, dim3(MOE_WARPS * 32), smem_dn, stream, (const T*)h, tokens, table,        \
                              (const T*)w_down, y, D, F, top, vocab, n_experts, outs, accumulate, status, route_w,     \
-                             n_ident, (const T*)x);                                                                   \
+                             n_ident, (const T*)x, in_w ? 1.0f : 1.0f / (float)top);                                  \
   } while (0)
-  if (vec_gu) ZK_MOE_GU(true); else ZK_MOE_GU(false);
+  if (act < 0) {
+    if (vec_gu) ZK_MOE_GU(true, true); else ZK_MOE_GU(false, true);
+  } else {
+    if (vec_gu) ZK_MOE_GU(true, false); else ZK_MOE_GU(false, false);
+  }
   if (rc != 0) return rc;
   if (vec_dn) ZK_MOE_DN(true); else ZK_MOE_DN(false);
   return rc;
@@ -423,24 +467,29 @@ int zk_moe_table(const void* x, const int* tokens, const int* table, const void*
   if (n <= 0) return 0;
   if (D <= 0 || F <= 0 || top <= 0 || vocab <= 0 || n_experts <= 0 || il < 0 || (il > 0 && F % il)) return ZK_EINVAL;
   if (dtype == ZK_F32)
-    return launch_moe<float>(x, tokens, table, w_gu, il, w_down, h, y, n, D, F, top, vocab, n_experts, accumulate, status, nullptr, 0, stream);
+    return launch_moe<float>(x, tokens, table, w_gu, il, w_down, h, y, n, D, F, top, vocab, n_experts, accumulate, status, nullptr, 0, -1, nullptr, stream);
   if (dtype == ZK_BF16)
-    return launch_moe<bf16>(x, tokens, table, w_gu, il, w_down, h, y, n, D, F, top, vocab, n_experts, accumulate, status, nullptr, 0, stream);
+    return launch_moe<bf16>(x, tokens, table, w_gu, il, w_down, h, y, n, D, F, top, vocab, n_experts, accumulate, status, nullptr, 0, -1, nullptr, stream);
   return ZK_EINVAL;
 }
 
 // The same with the experts a router chose: route_ids [n, top] int32 and route_w [n, top] float32 (the weight of
 // each), y_t = sum_k route_w[t, k] * Expert[route_ids[t, k]](x_t), added in the order of k.  Ids n_experts ..
-// n_experts + n_ident - 1 are identity experts: Expert(x_t) = x_t.
+// n_experts + n_ident - 1 are identity experts: Expert(x_t) = x_t.  act < 0: gated experts; else ungated, w_gu [experts, F, D].
+// weight_in != 0: the weights multiply the experts' inputs, y_t = sum_k Expert(route_w[t, k] * x_t) (no identity experts).
 int zk_moe_routed(const void* x, const int* route_ids, const float* route_w, const void* w_gu, int il, const void* w_down,
                   void* h, float* y, int n, int D, int F, int top, int n_experts, int accumulate, int dtype, int* status,
-                  int n_ident, cudaStream_t stream) {
+                  int n_ident, int act, int weight_in, cudaStream_t stream) {
   if (n <= 0) return 0;
+  if (act >= 0 && il) return ZK_EINVAL;
+  if (weight_in && n_ident) return ZK_EINVAL;
+  const float* in_w = weight_in ? route_w : nullptr;
+  const float* out_w = weight_in ? nullptr : route_w;
   if (D <= 0 || F <= 0 || top <= 0 || n_experts <= 0 || n_ident < 0 || il < 0 || (il > 0 && F % il) || !route_ids || !route_w) return ZK_EINVAL;
   if (dtype == ZK_F32)
-    return launch_moe<float>(x, nullptr, route_ids, w_gu, il, w_down, h, y, n, D, F, top, 1, n_experts, accumulate, status, route_w, n_ident, stream);
+    return launch_moe<float>(x, nullptr, route_ids, w_gu, il, w_down, h, y, n, D, F, top, 1, n_experts, accumulate, status, out_w, n_ident, act, in_w, stream);
   if (dtype == ZK_BF16)
-    return launch_moe<bf16>(x, nullptr, route_ids, w_gu, il, w_down, h, y, n, D, F, top, 1, n_experts, accumulate, status, route_w, n_ident, stream);
+    return launch_moe<bf16>(x, nullptr, route_ids, w_gu, il, w_down, h, y, n, D, F, top, 1, n_experts, accumulate, status, out_w, n_ident, act, in_w, stream);
   return ZK_EINVAL;
 }
 
@@ -448,7 +497,7 @@ int zk_moe_routed(const void* x, const int* route_ids, const float* route_w, con
 // largest s (ties: the lower index) are chosen and weighed s / (sum of the chosen + 1e-20).  With `correction` [E] the
 // choice goes by s + correction; the weights are made of s alone.
 int zk_moe_router(const void* x, const float* w_router, int* route_ids, float* route_w, int n, int D, int E, int top,
-                  int dtype, const float* correction, cudaStream_t stream) {
+                  int dtype, const float* correction, int sigmoid, int renorm, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (D <= 0 || E <= 0 || top <= 0 || top > E || E > MOE_ROUTER_MAX_EXPERTS) return ZK_EINVAL;
   const size_t smem = sizeof(float) * ((size_t)D + 2 * (size_t)E);
@@ -461,7 +510,7 @@ int zk_moe_router(const void* x, const float* w_router, int* route_ids, float* r
       if (e != cudaSuccess) return (int)e;                                                                           \
     }                                                                                                                \
     return zk_launch_dependent(kern, dim3(n), dim3(MOE_WARPS * 32), smem, stream, (const T*)x, w_router, route_ids,  \
-                               route_w, D, E, top, correction);                                                      \
+                               route_w, D, E, top, correction, sigmoid, renorm);                                     \
   } while (0)
   if (dtype == ZK_F32) ZK_ROUTER(float);
   if (dtype == ZK_BF16) ZK_ROUTER(bf16);
@@ -471,32 +520,35 @@ int zk_moe_router(const void* x, const float* w_router, int* route_ids, float* r
 
 // The device's own sort of (token, k) pairs by expert, as moe_expert_rows_kernel describes it.
 int zk_moe_expert_rows(const int* ids, int P, int E, int top, int tile, int cap, int* row_token, int* pair_row,
-                       int* tile_group, int n_ident, cudaStream_t stream) {
+                       int* tile_group, int n_ident, int name_pairs, cudaStream_t stream) {
   if (P <= 0) return 0;
   if (E <= 0 || E > 4096 || top <= 0 || tile <= 0 || cap % tile || cap < (P / tile + E) * tile) return ZK_EINVAL;
   return zk_launch_dependent(moe_expert_rows_kernel, dim3(1), dim3(1024), sizeof(int) * 2 * (size_t)E, stream, ids, P, E,
-                             top, tile, cap, row_token, pair_row, tile_group, n_ident);
+                             top, tile, cap, row_token, pair_row, tile_group, n_ident, name_pairs);
 }
 
-// xg[r, :] = x[row_token[r], :] for r < n_rows, zeros where row_token[r] < 0 (rows in the run dtype, D elements).
-int zk_moe_gather(const void* x, const int* row_token, void* xg, int n_rows, int D, int dtype, cudaStream_t stream) {
+// xg[r, :] = x[row_token[r], :] for r < n_rows, zeros where row_token[r] < 0 (rows in the run dtype, D elements).  With pair_w
+// row_token names pairs t * top + k and xg[r, :] = pair_w[pair] * x[t, :].
+int zk_moe_gather(const void* x, const int* row_token, void* xg, int n_rows, int D, int dtype, const float* pair_w, int top,
+                  cudaStream_t stream) {
   if (n_rows <= 0) return 0;
-  if (D <= 0) return ZK_EINVAL;
+  if (D <= 0 || (pair_w && top <= 0)) return ZK_EINVAL;
   const int threads = 128;
   if (dtype == ZK_F32)
-    return zk_launch_dependent(moe_gather_kernel<float>, dim3(n_rows), dim3(threads), 0, stream, (const float*)x, row_token, (float*)xg, D);
+    return zk_launch_dependent(moe_gather_kernel<float>, dim3(n_rows), dim3(threads), 0, stream, (const float*)x, row_token, (float*)xg, D, pair_w, top);
   if (dtype == ZK_BF16)
-    return zk_launch_dependent(moe_gather_kernel<bf16>, dim3(n_rows), dim3(threads), 0, stream, (const bf16*)x, row_token, (bf16*)xg, D);
+    return zk_launch_dependent(moe_gather_kernel<bf16>, dim3(n_rows), dim3(threads), 0, stream, (const bf16*)x, row_token, (bf16*)xg, D, pair_w, top);
   return ZK_EINVAL;
 }
 
-// out[t, :] (=|+=) (1/top) * sum_k y[pair_row[t * top + k], :], float32, added in the order of k.
+// out[t, :] (=|+=) sum_k weight * y[pair_row[t * top + k], :], float32, added in the order of k; the weight of a pair is
+// route_w's, or plain_weight without them.
 int zk_moe_combine(const float* y, const int* pair_row, float* out, int n, int D, int top, int accumulate,
-                   const float* route_w, const void* x_ident, int x_dtype, cudaStream_t stream) {
+                   const float* route_w, const void* x_ident, int x_dtype, float plain_weight, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (D <= 0 || top <= 0) return ZK_EINVAL;
   return zk_launch_dependent(moe_combine_kernel, dim3(n), dim3(128), 0, stream, y, pair_row, out, D, top, accumulate, route_w,
-                             x_ident, x_dtype == ZK_BF16 ? 1 : 0);
+                             x_ident, x_dtype == ZK_BF16 ? 1 : 0, plain_weight);
 }
 
 }  // extern "C"

@@ -42,8 +42,8 @@ _SIGNATURES = {
         "zk_clamped_glu": "ppiiiffip",
         "zk_head_gate": "ppiiiiip",
         "zk_layernorm": "pppppiifip",
-        "zk_value_gate": "ppiiiiiip",
-        "zk_unit_norm_gate": "ppipiiifip",
+        "zk_value_gate": "ppiiiiii" + "i" + "p",
+        "zk_unit_norm_gate": "ppipiiifi" + "piipf" + "p",
         "zk_gated_act": "ppiiiiip",
         "zk_gated_group_norm": "ppippiiifip",
     },
@@ -63,6 +63,13 @@ _SIGNATURES = {
         "zk_hgrn2_max_dim": "",
         "zk_retention_scan": "pippifpplpppiiiiip",
         "zk_ssd_scan": "pipipppplppp" + "iiiiii" + "p",
+        "zk_mlstm_state_floats": "iii",
+        "zk_mlstm_scan": "pippippf" + "plpppp" + "iiiii" + "p",
+    },
+    "delta": {
+        "zk_delta_max_dim": "",
+        "zk_delta_state_floats": "iii",
+        "zk_delta_scan": "pipipipp" + "plppp" + "iiiiii" + "fi" + "p",
     },
     "seqconv": {
         "zk_seqconv_forward": "ppppppp" + "iiiliii" + "ipi" + "p",
@@ -71,11 +78,11 @@ _SIGNATURES = {
     },
     "moe": {
         "zk_moe_table": "ppppippp" + "iiiiiiiipp",
-        "zk_moe_gather": "pppiiip",
-        "zk_moe_combine": "pppiiii" + "p" + "pi" + "p",
-        "zk_moe_routed": "ppppippp" + "iiiiiii" + "pip",
-        "zk_moe_router": "pppp" + "iiiii" + "pp",
-        "zk_moe_expert_rows": "piiiiippp" + "ip",
+        "zk_moe_gather": "pppiii" + "pi" + "p",
+        "zk_moe_combine": "pppiiii" + "p" + "pi" + "f" + "p",
+        "zk_moe_routed": "ppppippp" + "iiiiiii" + "pi" + "ii" + "p",
+        "zk_moe_router": "pppp" + "iiiii" + "p" + "ii" + "p",
+        "zk_moe_expert_rows": "piiiiippp" + "ii" + "p",
     },
     "gemm_simt": {
         "zk_gemm_simt": "ppppiiiiiiiiip",
@@ -91,7 +98,7 @@ _SIGNATURES = {
         "zk_gemm_tc": "ppppiiiiiiiiii" + "pifppp" + "p" + "pi" + "ff" + "p",
         "zk_gemm_tc_fuses_epilogue": "iiiii",
         "zk_gemm_tc_force_form": "i",
-        "zk_gemm_tc_grouped": "pppiiiiiiiippp",
+        "zk_gemm_tc_grouped": "pppiiiiiiii" + "pp" + "i" + "p",
     },
     "shortconv": {
         "zk_conv_forward": "ppppppppiiiliip",
@@ -135,8 +142,8 @@ _SIGNATURES = {
         "zk_sample": "piififfffip" + "lpp" + "pp",
     },
     "attention": {
-        "zk_qk_prepare": "pppppppppppp" + "iiiiiiifiiip" + "ii" + "fi" + "ipiiif" + "p",
-        "zk_qk_prepare_span": "pipppppppppiiiiiifiiip" + "pi" + "p",
+        "zk_qk_prepare": "pppppppppppp" + "iiiiiiifiiip" + "ii" + "fi" + "ipiiif" + "f" + "p",
+        "zk_qk_prepare_span": "pipppppppppiiiiiifiiip" + "pi" + "f" + "p",
         "zk_attn_fwd": "pppppp" + "pppppp" + "iiiiiiiifiiiii" + "ippi" + "ipi" + "f" + "piipi" + "p",
         "zk_attn_merge_talk": "ppppiiiiiip",
         "zk_attn_merge": "pppiiii" + "pi" + "pi" + "p",
@@ -505,6 +512,86 @@ def ssd_scan(xbc: torch.Tensor, z: torch.Tensor, dt_bias: torch.Tensor, a_log: t
     return o
 
 
+def mlstm_state_floats(n_heads: int, dim: int, value_dim: int) -> int:
+    """Floats of per-sequence state of `mlstm_scan` (what zk_mlstm_state_floats says; needed without a GPU)."""
+    return n_heads * dim * (value_dim + 1) + n_heads * -(-(value_dim + 1) // 32)
+
+
+def mlstm_scan(qkv: torch.Tensor, zi: torch.Tensor, zf: torch.Tensor, bias_i: torch.Tensor, bias_f: torch.Tensor, cap: float,
+               state: torch.Tensor, cu_q, seq_slot, n_seqs: int, n_heads: int, dim: int, value_dim: int):
+    """Matrix memory with exponential gates (mLSTM) per head over each sequence's tokens: i = cap tanh((zi + bias_i) / cap),
+    f = logsigmoid(cap tanh((zf + bias_f) / cap)), m_t = max(f + m_{t-1}, i) from m = 0, S_t = exp(f + m_{t-1} - m_t) S_{t-1} +
+    exp(i - m_t) k_t [v_t, 1]^T.  qkv float32 [n, >= 2*H*d + H*e] (row stride used), a row [q | k | v | ..]; zi, zf float32 [n, H] with
+    one row stride; state float32 [slots, mlstm_state_floats] (row stride used).  Returns (o float32 [n, H * (e + 1)]: the read-outs
+    S_t^T q_t with, last of a head, the normaliser's; m float32 [n, H])."""
+    H, d, e = n_heads, dim, value_dim
+    _need(qkv, "qkv", torch.float32, (None, None), contiguous=False)
+    n = qkv.shape[0]
+    if qkv.shape[1] < 2 * H * d + H * e or qkv.stride(1) != 1:
+        raise KernelError(f"mlstm_scan: rows of {qkv.shape[1]} values hold no q, k and v of {H} heads")
+    for z, nm in ((zi, "zi"), (zf, "zf")):
+        _need(z, nm, torch.float32, (n, H), contiguous=False)
+    if zi.stride() != zf.stride() or (H > 1 and zi.stride(1) != 1):
+        raise KernelError("mlstm_scan: the raw gates need one row stride, heads side by side")
+    for b, nm in ((bias_i, "bias_i"), (bias_f, "bias_f")):
+        _need(b, nm, torch.float32, (H,))
+    _need(state, "state", torch.float32, contiguous=False)
+    if state.dim() != 2 or state.shape[1] != mlstm_state_floats(H, d, e) or state.stride(1) != 1:
+        raise KernelError(f"mlstm_scan: state {tuple(state.shape)} must hold {mlstm_state_floats(H, d, e)} values per slot")
+    for t, nm in ((cu_q, "cu_q"), (seq_slot, "seq_slot")):
+        _need(t, nm, torch.int32)
+    o = torch.empty((n, H * (e + 1)), dtype=torch.float32, device=qkv.device)
+    m = torch.empty((n, H), dtype=torch.float32, device=qkv.device)
+    _check(_fn("hgrn2", "zk_mlstm_scan")(_ptr(qkv), qkv.stride(0), _ptr(zi), _ptr(zf), zi.stride(0), _ptr(bias_i), _ptr(bias_f),
+                                         float(cap), _ptr(state), state.stride(0), _ptr(o), _ptr(m), _ptr(cu_q), _ptr(seq_slot), n,
+                                         n_seqs, H, d, e, _stream()), "mlstm_scan")
+    return o, m
+
+
+# ------------------------------------------------------------------------------- gated delta rule
+
+def delta_max_dim() -> int:
+    return _constant("delta", "zk_delta_max_dim")
+
+
+def delta_state_floats(n_heads: int, dim: int, value_dim: int) -> int:
+    """Floats of per-sequence state of `delta_scan` (what zk_delta_state_floats says; needed without a GPU)."""
+    return n_heads * value_dim * (-(-dim // 4) * 4)
+
+
+def delta_scan(qkv: torch.Tensor, a: torch.Tensor, z_beta: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
+               state: torch.Tensor, cu_q, seq_slot, n_seqs: int, n_heads: int, groups: int, dim: int, value_dim: int,
+               single_token: bool = False) -> torch.Tensor:
+    """Gated delta rule per head over each sequence's tokens, from the state the step before left to the state this one leaves:
+    S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, with g = exp(-exp(a_log) softplus(a + dt_bias)) per head and key
+    channel, beta = sigmoid(z_beta), q and k unit vectors (x / sqrt(sum x^2 + 1e-6)), q also times d^-1/2.  qkv float32
+    [n, >= 2*G*d + H*e], a row [q | k | v | ..], q and k shared by the H / G heads of a group; a float32 [n, >= H*d]; z_beta float32
+    [n, H] (row strides used); a_log [H], dt_bias [H*d]; state float32 [slots, delta_state_floats], 16-byte aligned rows, ordered
+    [H, e, d up to a multiple of 4].  `single_token`: every sequence brings one token; otherwise q, k and a are overwritten by the unit
+    vectors and decays.  Returns o float32 [n, H*e]."""
+    H, G, d, e = n_heads, groups, dim, value_dim
+    _need(qkv, "qkv", torch.float32, (None, None), contiguous=False)
+    n = qkv.shape[0]
+    if qkv.shape[1] < 2 * G * d + H * e or qkv.stride(1) != 1:
+        raise KernelError(f"delta_scan: rows of {qkv.shape[1]} values hold no q, k and v of {H} heads")
+    _need(a, "a", torch.float32, (n, None), contiguous=False)
+    _need(z_beta, "z_beta", torch.float32, (n, H), contiguous=False)
+    if a.shape[1] < H * d or a.stride(1) != 1 or (H > 1 and z_beta.stride(1) != 1):
+        raise KernelError(f"delta_scan: decays {tuple(a.shape)} / betas {tuple(z_beta.shape)} do not fit {H} heads of {d}")
+    _need(a_log, "a_log", torch.float32, (H,))
+    _need(dt_bias, "dt_bias", torch.float32, (H * d,))
+    _need(state, "state", torch.float32, contiguous=False)
+    if state.dim() != 2 or state.shape[1] != delta_state_floats(H, d, e) or state.stride(1) != 1:
+        raise KernelError(f"delta_scan: state {tuple(state.shape)} must hold {delta_state_floats(H, d, e)} values per slot")
+    for t, nm in ((cu_q, "cu_q"), (seq_slot, "seq_slot")):
+        _need(t, nm, torch.int32)
+    o = torch.empty((n, H * e), dtype=torch.float32, device=qkv.device)
+    _check(_fn("delta", "zk_delta_scan")(_ptr(qkv), qkv.stride(0), _ptr(a), a.stride(0), _ptr(z_beta), z_beta.stride(0), _ptr(a_log),
+                                         _ptr(dt_bias), _ptr(state), state.stride(0), _ptr(o), _ptr(cu_q), _ptr(seq_slot), n, n_seqs, H, G,
+                                         d, e, float(d) ** -0.5, 1 if single_token else 0, _stream()), "delta_scan")
+    return o
+
+
 # ------------------------------------------------------------------------------- convolution over time on a mixer's input
 
 def seqconv_max_taps() -> int:
@@ -605,31 +692,48 @@ def layernorm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor
 
 def value_gate(rows: torch.Tensor, gate: torch.Tensor, n_heads: int, valid: int) -> torch.Tensor:
     """rows[t, h, j] *= sigmoid(gate[t, h * valid + j]) for j < valid, in place.  rows [n, H * width] contiguous (run
-    dtype; the values of a head behind `valid` are padding and left alone); gate float32 [n, >= H * valid] (a view of
+    dtype; the values of a head behind `valid` are padding and left alone); gate float32 or bfloat16 [n, >= H * valid] (a view of
     wider rows is fine: its row stride is used)."""
     _need(rows, "rows", (torch.float32, torch.bfloat16), (None, None))
     n, w = rows.shape
-    _need(gate, "gate", torch.float32, (n, None), contiguous=False)
+    _need(gate, "gate", (torch.float32, torch.bfloat16), (n, None), contiguous=False)
     if w % n_heads or valid > w // n_heads or gate.shape[1] < n_heads * valid or gate.stride(1) != 1:
         raise KernelError(f"value_gate: rows {tuple(rows.shape)} / gate {tuple(gate.shape)} do not fit {n_heads} heads "
                           f"of {valid} values")
     _check(_fn("elementwise", "zk_value_gate")(_ptr(rows), _ptr(gate), gate.stride(0), n, n_heads, w // n_heads, valid,
-                                               dtype_code(rows.dtype), _stream()), "value_gate")
+                                               dtype_code(rows.dtype), dtype_code(gate.dtype), _stream()), "value_gate")
     return rows
 
 
-def unit_norm_gate(o: torch.Tensor, gate: torch.Tensor, n_heads: int, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+def unit_norm_gate(o: torch.Tensor, gate: torch.Tensor, n_heads: int, eps: float, out_dtype: torch.dtype,
+                   weight: Optional[torch.Tensor] = None, sigmoid: bool = False, den_log: Optional[torch.Tensor] = None,
+                   out_scale: float = 1.0) -> torch.Tensor:
     """y[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * silu(gate[t, h, :]): every head over its root mean
     square (no weight), gated.  o float32 [n, H * e]; gate float32 [n, >= H * e] (may be a view of wider rows);
-    returns [n, H * e] in `out_dtype`."""
+    returns [n, H * e] in `out_dtype`.  `weight` float32 [e] (shared by the heads) or [H * e] multiplies behind the norm;
+    `sigmoid`: sigmoid(gate) in place of silu.  `den_log` float32 [n, H]: o is [n, H * (e + 1)], a head's last value the product of
+    normaliser and query of `mlstm_scan`, and the head that is normed is s * o / (max(|s * o_e|, exp(-den_log)) + 1e-6),
+    s = out_scale."""
     _need(o, "o", torch.float32, (None, None))
     n, w = o.shape
+    w -= n_heads if den_log is not None else 0
     _need(gate, "gate", torch.float32, (n, None), contiguous=False)
-    if w % n_heads or gate.shape[1] < w or gate.stride(1) != 1:
+    if weight is not None:
+        _need(weight, "weight", torch.float32)
+        if weight.numel() not in (w, w // n_heads):
+            raise KernelError(f"unit_norm_gate: a weight of {weight.numel()} values for {n_heads} heads of {w // n_heads}")
+    if den_log is not None:
+        _need(den_log, "den_log", torch.float32, (n, n_heads))
+    elif out_scale != 1.0:
+        raise KernelError("unit_norm_gate: the output scale goes with a denominator")
+    if w <= 0 or w % n_heads or gate.shape[1] < w or gate.stride(1) != 1:
         raise KernelError(f"unit_norm_gate: o {tuple(o.shape)} / gate {tuple(gate.shape)} do not fit {n_heads} heads")
     y = torch.empty((n, w), dtype=out_dtype, device=o.device)
     _check(_fn("elementwise", "zk_unit_norm_gate")(_ptr(o), _ptr(gate), gate.stride(0), _ptr(y), n, n_heads, w // n_heads,
-                                                   eps, dtype_code(out_dtype), _stream()), "unit_norm_gate")
+                                                   eps, dtype_code(out_dtype), _ptr(weight),
+                                                   0 if weight is None or weight.numel() != w or n_heads == 1 else w // n_heads,
+                                                   1 if sigmoid else 0, _ptr(den_log), float(out_scale), _stream()),
+           "unit_norm_gate")
     return y
 
 
@@ -895,10 +999,11 @@ def gemm_tc_grouped_takes(a: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def gemm_tc_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, swiglu: bool = False,
-                    out_dtype=torch.bfloat16) -> torch.Tensor:
+                    out_dtype=torch.bfloat16, act: Optional[str] = None) -> torch.Tensor:
     """out[rows of tile t] = a[rows of tile t] @ w[tile_group[t]].T on the tcgen05 kernel: a [M, K] bfloat16 in
     tiles of 128 rows, w [groups, N, K] bfloat16, tile_group int32 [M / 128] on the device.  With `swiglu`
-    every w[g] holds groups of 16 gate rows and their 16 up rows and the result is silu(gate) * up, [M, N/2]."""
+    every w[g] holds groups of 16 gate rows and their 16 up rows and the result is silu(gate) * up, [M, N/2].  `act` names an
+    activation of the result: the square of relu in the epilogue where N is a multiple of 256, any other by a kernel of its own."""
     if not gemm_tc_grouped_takes(a, w):
         raise KernelError(f"gemm_tc_grouped: a {tuple(a.shape)} / w {tuple(w.shape)} need bfloat16, whole tiles of "
                           f"{GEMM_TC_GROUP_ROWS} rows, K a multiple of 8")
@@ -907,19 +1012,27 @@ def gemm_tc_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, 
     _need(tile_group, "tile_group", torch.int32, (M // GEMM_TC_GROUP_ROWS,))
     if swiglu and N % 32:
         raise KernelError("gemm_tc_grouped: the SwiGLU epilogue needs N a multiple of 32")
+    if act is not None and (swiglu or act not in ACTIVATIONS):
+        raise KernelError(f"gemm_tc_grouped: no activation {act!r} here")
+    fused = act == "relu_squared" and N % 256 == 0 and _forced_form != 0
     out = torch.empty((M, N // 2 if swiglu else N), dtype=out_dtype, device=a.device)
     _need(out, "out", (torch.float32, torch.bfloat16))
     _check(_fn("gemm_tc", "zk_gemm_tc_grouped")(_ptr(a), _ptr(w), _ptr(out), M, N, K, G, a.stride(0), out.stride(0),
                                                 dtype_code(out.dtype), 1 if swiglu else 0, _ptr(tile_group),
-                                                _ptr(status_word(a.device)), _stream()), "gemm_tc_grouped")
-    return out
+                                                _ptr(status_word(a.device)), 1 if fused else 0, _stream()), "gemm_tc_grouped")
+    return activation(out, act, out=out) if act is not None and not fused else out
+
+
+_forced_form = -1
 
 
 def gemm_tc_force_form(form: int) -> None:
     """For measurements and tests: the form that products of more than 64 rows with N a multiple of
     256 take.  0 = one 128 x 128 tile per block, 256 = persistent blocks with 128 x 256 tiles, 512 =
     persistent pairs of blocks with 256 x 256 tiles (tcgen05.mma.cta_group::2); -1 = the library chooses."""
+    global _forced_form
     _check(_fn("gemm_tc", "zk_gemm_tc_force_form")(int(form)), "gemm_tc_force_form")
+    _forced_form = int(form)
 
 
 _constants: dict[str, int] = {}     # what the libraries say about themselves, asked once
@@ -1162,20 +1275,25 @@ def conv_decode(bcx, state, w, bias, seq_slot, interleave: int = 0) -> torch.Ten
     return y
 
 
-def moe_gather(x: torch.Tensor, row_token: torch.Tensor) -> torch.Tensor:
-    """xg[r] = x[row_token[r]] (zeros where row_token[r] < 0): rows in the order a grouped contraction wants them."""
+def moe_gather(x: torch.Tensor, row_token: torch.Tensor, pair_weights: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """xg[r] = x[row_token[r]] (zeros where row_token[r] < 0): rows in the order a grouped contraction wants them.  With
+    `pair_weights` float32 [n, top] row_token names pairs t * top + k and xg[r] = weight of the pair * x[t]."""
+    if pair_weights is not None:
+        _need(pair_weights, "pair_weights", torch.float32, (x.shape[0], None))
     _need(x, "x", (torch.float32, torch.bfloat16), (None, None))
     _need(row_token, "row_token", torch.int32)
     xg = torch.empty((row_token.numel(), x.shape[1]), dtype=x.dtype, device=x.device)
     _check(_fn("moe", "zk_moe_gather")(_ptr(x), _ptr(row_token), _ptr(xg), row_token.numel(), x.shape[1],
-                                       dtype_code(x.dtype), _stream()), "moe_gather")
+                                       dtype_code(x.dtype), _ptr(pair_weights),
+                                       pair_weights.shape[1] if pair_weights is not None else 1, _stream()), "moe_gather")
     return xg
 
 
 def moe_combine(y: torch.Tensor, pair_row: torch.Tensor, top: int, out: torch.Tensor, accumulate: bool = False,
-                weights: Optional[torch.Tensor] = None, identity_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out[t] (+)= sum_k weights[t, k] * y[pair_row[t * top + k]] (weights float32 [n, top]; without them 1/top
-    each), float32, added in the order of k.  A pair whose row is negative stands for an identity expert: its term is
+                weights: Optional[torch.Tensor] = None, identity_rows: Optional[torch.Tensor] = None,
+                plain_weight: Optional[float] = None) -> torch.Tensor:
+    """out[t] (+)= sum_k weights[t, k] * y[pair_row[t * top + k]] (weights float32 [n, top]; without them `plain_weight`,
+    default 1/top, each), float32, added in the order of k.  A pair whose row is negative stands for an identity expert: its term is
     identity_rows[t] (the rows the experts read, [n, D] in a run dtype)."""
     _need(y, "y", torch.float32, (None, None))
     _need(out, "out", torch.float32, (None, y.shape[1]))
@@ -1186,17 +1304,19 @@ def moe_combine(y: torch.Tensor, pair_row: torch.Tensor, top: int, out: torch.Te
         _need(identity_rows, "identity_rows", (torch.float32, torch.bfloat16), (out.shape[0], y.shape[1]))
     _check(_fn("moe", "zk_moe_combine")(_ptr(y), _ptr(pair_row), _ptr(out), out.shape[0], y.shape[1], top,
                                         1 if accumulate else 0, _ptr(weights), _ptr(identity_rows),
-                                        dtype_code(identity_rows.dtype) if identity_rows is not None else F32, _stream()),
+                                        dtype_code(identity_rows.dtype) if identity_rows is not None else F32,
+                                        1.0 / top if plain_weight is None else float(plain_weight), _stream()),
            "moe_combine")
     return out
 
 
-def moe_router(x: torch.Tensor, w_router: torch.Tensor, top: int,
-               correction: Optional[torch.Tensor] = None) -> tuple[torch.Tensor, torch.Tensor]:
+def moe_router(x: torch.Tensor, w_router: torch.Tensor, top: int, correction: Optional[torch.Tensor] = None,
+               sigmoid: bool = False, renormalize: bool = True) -> tuple[torch.Tensor, torch.Tensor]:
     """(experts int32 [n, top], weights float32 [n, top]) of every row of x [n, D] (run dtype): logits W x in
     float32 (w_router float32 [E, D]), softmax over all E experts, the `top` largest scores (of equal ones the
     lower index), each divided by the sum of the chosen (+ 1e-20).  `correction` float32 [E]: the choice goes by
-    score + correction, the weights are made of the scores alone."""
+    score + correction, the weights are made of the scores alone.  `sigmoid`: an expert's score is the sigmoid of its own
+    logit; `renormalize` False: the weights are the chosen scores as they are."""
     _need(x, "x", (torch.float32, torch.bfloat16), (None, None))
     n, D = x.shape
     _need(w_router, "w_router", torch.float32, (None, D))
@@ -1208,16 +1328,17 @@ def moe_router(x: torch.Tensor, w_router: torch.Tensor, top: int,
     ids = torch.empty((n, top), dtype=torch.int32, device=x.device)
     wts = torch.empty((n, top), dtype=torch.float32, device=x.device)
     _check(_fn("moe", "zk_moe_router")(_ptr(x), _ptr(w_router), _ptr(ids), _ptr(wts), n, D, E, top, dtype_code(x.dtype),
-                                       _ptr(correction), _stream()), "moe_router")
+                                       _ptr(correction), 1 if sigmoid else 0, 1 if renormalize else 0, _stream()), "moe_router")
     return ids, wts
 
 
 def moe_expert_rows(route_ids: torch.Tensor, n_experts: int, tile: int,
-                    n_identity: int = 0) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
+                    n_identity: int = 0, name_pairs: bool = False) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
     """The (token, k) pairs of route_ids [n, top] (int32, device) sorted by expert on the device, every expert's rows
     padded to whole tiles: (row_token [cap] with -1 for padding rows, pair_row [n * top], tile_group [cap / tile]),
     cap = the most rows any choice can need.  Tiles behind the last expert's hold padding rows only.  Ids n_experts ..
-    n_experts + n_identity - 1 name identity experts: such a pair gets no row (pair_row -1)."""
+    n_experts + n_identity - 1 name identity experts: such a pair gets no row (pair_row -1).  `name_pairs`: row_token holds the
+    row's pair t * top + k instead of its token."""
     _need(route_ids, "route_ids", torch.int32, (None, None))
     n, top = route_ids.shape
     P = n * top
@@ -1225,23 +1346,29 @@ def moe_expert_rows(route_ids: torch.Tensor, n_experts: int, tile: int,
     words = torch.empty(cap + P + cap // tile, dtype=torch.int32, device=route_ids.device)
     row_token, pair_row, tile_group = words[:cap], words[cap:cap + P], words[cap + P:]
     _check(_fn("moe", "zk_moe_expert_rows")(_ptr(route_ids), P, n_experts, top, tile, cap, _ptr(row_token), _ptr(pair_row),
-                                            _ptr(tile_group), int(n_identity), _stream()), "moe_expert_rows")
+                                            _ptr(tile_group), int(n_identity), 1 if name_pairs else 0, _stream()), "moe_expert_rows")
     return row_token, pair_row, tile_group
 
 
 def moe_routed(x: torch.Tensor, route_ids: torch.Tensor, route_w: torch.Tensor, w_gate_up: torch.Tensor, interleave: int,
                w_down: torch.Tensor, status: torch.Tensor, out: Optional[torch.Tensor] = None,
-               accumulate: bool = False, n_identity: int = 0) -> torch.Tensor:
+               accumulate: bool = False, n_identity: int = 0, act: Optional[str] = None,
+               weight_input: bool = False) -> torch.Tensor:
     """y[t] = sum_k route_w[t, k] * W_down[e] (silu(W_gate[e] x_t) * (W_up[e] x_t)), e = route_ids[t, k], added in
     the order of k.  Tensors as in `moe_table`.  Ids E .. E + n_identity - 1 name identity experts, whose term is
-    route_w[t, k] * x_t."""
+    route_w[t, k] * x_t.  `act` names an activation (`ACTIVATIONS`): the experts are ungated, W_down[e] act(W_up[e] x_t), and
+    w_gate_up is [E, F, D].  `weight_input`: a weight multiplies what its expert reads, not what it returns."""
+    if act is not None and act not in ACTIVATIONS:
+        raise KernelError(f"moe_routed: unknown activation {act!r}")
+    if weight_input and n_identity:
+        raise KernelError("moe_routed: weights on the inputs do not go with identity experts")
     _need(x, "x", (torch.float32, torch.bfloat16), (None, None))
     n, D = x.shape
     _need(route_ids, "route_ids", torch.int32, (n, None))
     top = route_ids.shape[1]
     _need(route_w, "route_w", torch.float32, (n, top))
     _need(w_gate_up, "w_gate_up", x.dtype, (None, None, D))
-    E, F = w_gate_up.shape[0], w_gate_up.shape[1] // 2
+    E, F = w_gate_up.shape[0], w_gate_up.shape[1] // (2 if act is None else 1)
     _need(w_down, "w_down", x.dtype, (E, D, F))
     if out is None:
         if accumulate:
@@ -1251,7 +1378,8 @@ def moe_routed(x: torch.Tensor, route_ids: torch.Tensor, route_w: torch.Tensor, 
     h = torch.empty((n, top, F), dtype=x.dtype, device=x.device)
     _check(_fn("moe", "zk_moe_routed")(_ptr(x), _ptr(route_ids), _ptr(route_w), _ptr(w_gate_up), int(interleave), _ptr(w_down),
                                        _ptr(h), _ptr(out), n, D, F, top, E, 1 if accumulate else 0, dtype_code(x.dtype),
-                                       _ptr(status), int(n_identity), _stream()), "moe_routed")
+                                       _ptr(status), int(n_identity), -1 if act is None else ACTIVATIONS[act],
+                                       1 if weight_input else 0, _stream()), "moe_routed")
     return out
 
 
@@ -1381,7 +1509,7 @@ def attn_max_head_dim() -> int:
 def qk_prepare(qkv, k_cache, v_cache, q_w, k_w, inv_freq, tok_seq, tok_pos, seq_slot, page_table, n_heads: int,
                n_kv: int, head_dim: int, n_rot: int, interleaved: bool, eps: float, status, write_kv: bool = True,
                value_dim: Optional[int] = None, unit_norm_after: bool = False,
-               query_temperature: Optional[tuple] = None, mix_values: Optional[tuple] = None):
+               query_temperature: Optional[tuple] = None, mix_values: Optional[tuple] = None, rot_amp: float = 1.0):
     """Per-head RMSNorm of q and k (if weights are given), rotary encoding (if `inv_freq` is
     given), then with `unit_norm_after` q and k heads divided by their root mean square (no weight);
     q out as [n, H*hd], and k, v written to their pages.  k_cache is one layer's
@@ -1390,7 +1518,7 @@ def qk_prepare(qkv, k_cache, v_cache, q_w, k_w, inv_freq, tok_seq, tok_pos, seq_
     1 + coef * ln(floor((p + 1) / every) + 1).
     A row of qkv may hold more behind its values (row stride used).  `mix_values` = (first, share): value heads of the same
     tokens, a tensor [n, Hkv, width <= value_dim] in qkv's dtype (strides used), mixed in before a value is cached,
-    v <- (1 - share) v + share first, in float32."""
+    v <- (1 - share) v + share first, in float32.  `rot_amp` multiplies the rotation's cosines and sines."""
     qt_coef, qt_every = (float(query_temperature[0]), int(query_temperature[1])) if query_temperature else (0.0, 0)
     vd = head_dim if value_dim is None else int(value_dim)
     _need(qkv, "qkv", (torch.float32, torch.bfloat16), (None, None), contiguous=False)
@@ -1422,20 +1550,23 @@ def qk_prepare(qkv, k_cache, v_cache, q_w, k_w, inv_freq, tok_seq, tok_pos, seq_
         _ptr(tok_pos), _ptr(seq_slot), _ptr(page_table), page_table.stride(0), n, n_heads, n_kv, head_dim, n_rot,
         1 if interleaved else 0, eps, page_size, 1 if write_kv else 0, dtype_code(qkv.dtype), _ptr(status), vd,
         1 if unit_norm_after else 0, qt_coef, qt_every, qkv.stride(0), _ptr(first), first_ld, first_hs, first_vd, float(share),
-        _stream()),
+        float(rot_amp), _stream()),
         "qk_prepare")
     return q
 
 
 def qk_prepare_span(qkv, k_cache, v_cache, q_w, k_w, tok_seq, tok_pos, seq_slot, page_table, n_heads: int, n_kv: int,
                     head_dim: int, value_dim: int, eps: float, status, write_kv: bool = True,
-                    inv_freq: Optional[torch.Tensor] = None, n_rot: int = 0) -> torch.Tensor:
+                    inv_freq: Optional[torch.Tensor] = None, n_rot: int = 0, rot_amp: float = 1.0) -> torch.Tensor:
     """RMSNorm of q over all its heads at once (weight [H*hd], or None) and of k likewise ([Hkv*hd]); with
     `inv_freq` [n_rot / 2] the first n_rot entries of every q and k head are then rotated by the token's position
-    (entry i paired with entry i + n_rot/2); q out as [n, H*hd]; k and v (value_dim wide) written to their pages.
-    A row of qkv holds [q | k | v], or q alone with write_kv False (the caches are then only needed for their sizes)."""
+    (entry i paired with entry i + n_rot/2, cosines and sines times `rot_amp`); q out as [n, H*hd]; k and v (value_dim wide) written to their pages.
+    A row of qkv holds [q | k | v] (and may hold more behind them), or q alone with write_kv False (the caches are then only
+    needed for their sizes)."""
     qd, kd, vd = n_heads * head_dim, n_kv * head_dim, n_kv * value_dim
-    _need(qkv, "qkv", (torch.float32, torch.bfloat16), (None, qd + (kd + vd if write_kv else 0)))
+    _need(qkv, "qkv", (torch.float32, torch.bfloat16), (None, None))
+    if qkv.shape[1] < qd + (kd + vd if write_kv else 0):
+        raise KernelError(f"qk_prepare_span: rows of {qkv.shape[1]} values hold no q, k and v of these heads")
     n = qkv.shape[0]
     _need(k_cache, "k_cache", qkv.dtype, (None, n_kv, None, head_dim))
     _need(v_cache, "v_cache", qkv.dtype, (None, n_kv, None, value_dim))
@@ -1453,7 +1584,7 @@ def qk_prepare_span(qkv, k_cache, v_cache, q_w, k_w, tok_seq, tok_pos, seq_slot,
         _ptr(qkv), qkv.stride(0), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(q_w), _ptr(k_w), _ptr(tok_seq),
         _ptr(tok_pos), _ptr(seq_slot), _ptr(page_table), page_table.stride(0), n, n_heads, n_kv, head_dim, value_dim,
         eps, k_cache.shape[2], 1 if write_kv else 0, dtype_code(qkv.dtype), _ptr(status), _ptr(inv_freq), int(n_rot),
-        _stream()), "qk_prepare_span")
+        float(rot_amp), _stream()), "qk_prepare_span")
     return q
 
 

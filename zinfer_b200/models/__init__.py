@@ -6,3 +6,4 @@ from . import zosurax  # noqa: F401  (registers Zosurax)
 from . import kerotar  # noqa: F401  (registers Kerotar)
 from . import pirisun  # noqa: F401  (registers Pirisun)
 from . import varolorn  # noqa: F401  (registers Varolorn)
+from . import nipizen  # noqa: F401  (registers Nipizen)

@@ -3,6 +3,7 @@ from .base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, POSITION_ENCODINGS, Blo
                    Norm, Part, PositionEncoding, Registry, RotaryParams, StateRequest, WeightSpec, walk_parts)
 from .attention import GqaAttention
 from .block import ParallelBlock, PreNormBlock, SublayerNormBlock
+from .delta import GatedDelta
 from .depth import DepthAverage
 from .embedding import LMHead, TokenEmbedding
 from .feedforward import ActMlp, ClampedGLU, ReluGLU, SwiGLU
@@ -11,6 +12,7 @@ from .latent import LatentAttention
 from .linear import linear
 from .loop import PassInput
 from .mamba2 import Mamba2
+from .mlstm import MLstm
 from .moe import RoutedMoE, TableMoE
 from .norm import LayerNorm, RMSNorm
 from .pair import MixerPair

@@ -25,7 +25,7 @@ one more term of head h's softmax denominator, with no key and no value, and is 
 `query_temperature` = (coef, every): the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)
 (positions enter through that factor alone when there is no position encoding).  `softcap`: a scaled score s becomes
 softcap * tanh(s / softcap) before the softmax.
-`bias_names` = (q, k, v, out): vectors added in the four projections.
+`bias_names` = (q, k, v, out): vectors added in the four projections (out None: not in that one).
 `distance_rows` = (name, most): a learned number per (distance bucket, head), a tensor [buckets, heads] added to the scaled
 score of query position i and key position j in row `distance_buckets(...)[i - j]`: one row per distance up to half the
 buckets, then rows whose edges grow geometrically up to the distance `most`.  The number of buckets is the tensor's.
@@ -33,14 +33,17 @@ buckets, then rows whose edges grow geometrically up to the distance `most`.  Th
 gives the pages of earlier stretches back.
 `head_gate_name`: a matrix [heads, hidden]; head h's output is multiplied by sigmoid of row h's product with the mixer's
 input before the output projection.  Its rows are part of the one q/k/v contraction.
+`value_gate_name`: a matrix [heads * value_dim, hidden]; every value of the concatenated heads is multiplied by sigmoid of its row's
+product with the mixer's input before the output projection.  Its rows are part of the one q/k/v contraction too.
 `value_mix` = (name, is_first): layers that share their first layer's values.  The layer with is_first leaves the values of
 the step's tokens for the others (its own number of that name is loaded and unused); in every other layer a value becomes
 (1 - lambda) v + lambda v_first before it is cached, lambda the layer's number of that name.
 `pad_heads`: in a bfloat16 run, heads whose keys and values are not both 64 or both 128 wide (and at most 128) are
 padded at load to the next of those widths, with zero rows in W_q, W_k and W_v and zero columns in W_o, so that the
 tensor-core kernels take them; a padded entry adds nothing to a score and meets a zero column of W_o, the cache holds
-the padded rows.  Per-head q/k norms count the padding; their weights and eps are scaled so that the result is the same
-(with P the padded width and d the head's: x / sqrt(ssq/P + eps d/P) * w sqrt(d/P) = x / sqrt(ssq/d + eps) * w).
+the padded rows.  q/k norms count the padding; their weights and eps are scaled so that the result is the same
+(with P the padded width and d the head's: x / sqrt(ssq/P + eps d/P) * w sqrt(d/P) = x / sqrt(ssq/d + eps) * w; norms over the whole projection have the
+same ratio).
 
 How the kernels are launched is decided here, not by the engine: the table of query tiles of a
 step, and for single-token steps the cut of a sequence's keys into chunks that separate blocks
@@ -142,8 +145,9 @@ class GqaAttention(Mixer):
                  unit_norm_after_rotation: bool = False, talk_name: Optional[str] = None, keep_first: int = 0,
                  sink_name: Optional[str] = None, query_temperature: Optional[tuple[float, int]] = None,
                  softcap: Optional[float] = None, pad_heads: bool = False,
-                 bias_names: Optional[tuple[str, str, str, str]] = None, distance_rows: Optional[tuple[str, float]] = None,
-                 chunk: int = 0, head_gate_name: Optional[str] = None, value_mix: Optional[tuple[str, bool]] = None):
+                 bias_names: Optional[tuple[str, str, str, Optional[str]]] = None, distance_rows: Optional[tuple[str, float]] = None,
+                 chunk: int = 0, head_gate_name: Optional[str] = None, value_mix: Optional[tuple[str, bool]] = None,
+                 value_gate_name: Optional[str] = None):
         """split_keys: keys per chunk of single-token attention, a multiple of 64 (0 = chosen per
         step from the batch and the GPU's size)."""
         if n_heads % n_kv_heads:
@@ -170,20 +174,24 @@ class GqaAttention(Mixer):
         if softcap is not None and (not softcap > 0 or talk_name is not None):
             raise ValueError("attention: a score cap must be positive and does not go with weights mixed across heads")
         self.softcap = 0.0 if softcap is None else float(softcap)
-        if pad_heads and (unit_norm_after_rotation or not own_kv or qk_norm_span == "all"
-                          or (position is not None and (q_norm_name or k_norm_name))):
-            raise ValueError("attention: padded heads go with key/value weights of the mixer's own and no norms but per-head ones "
-                             "without a position encoding")
-        newer = any(o is not None for o in (bias_names, distance_rows, head_gate_name, value_mix)) or chunk > 0
-        if newer and (self.span_prepare or talk_name is not None or not own_kv):
-            raise ValueError("attention: projection biases, distance buckets, chunks, a gate per head and mixed values go with "
-                             "per-head preparation, key/value weights of the mixer's own and weights not mixed across heads")
+        if pad_heads and (unit_norm_after_rotation or not own_kv):
+            raise ValueError("attention: padded heads go with key/value weights of the mixer's own and no norm behind the position "
+                             "encoding")
+        per_head_only = any(o is not None for o in (distance_rows, head_gate_name, value_mix)) or chunk > 0
+        newer = per_head_only or bias_names is not None or value_gate_name is not None
+        if newer and (talk_name is not None or not own_kv):
+            raise ValueError("attention: projection biases, distance buckets, chunks, gates and mixed values go with "
+                             "key/value weights of the mixer's own and weights not mixed across heads")
+        if per_head_only and self.span_prepare:
+            raise ValueError("attention: distance buckets, chunks, a gate per head and mixed values go with per-head preparation")
+        if head_gate_name is not None and value_gate_name is not None:
+            raise ValueError("attention: one gate, per head or per value")
         if chunk < 0 or (chunk > 0 and window > 0):
             raise ValueError("attention: a mask in stretches and a window exclude each other")
         if position is not None and newer and not hasattr(position, "rotary"):
             raise ValueError("attention: these options take a rotation table or no position encoding")
         self.bias_names, self.distance_rows, self.chunk = bias_names, distance_rows, int(chunk)
-        self.head_gate_name, self.value_mix = head_gate_name, value_mix
+        self.head_gate_name, self.value_mix, self.value_gate_name = head_gate_name, value_mix, value_gate_name
         self.b_qkv = self.b_out = self.distance_table = None
         self.value_share = 0.0
         self._plain_only = distance_rows is not None or chunk > 0 or head_gate_name is not None
@@ -242,11 +250,13 @@ class GqaAttention(Mixer):
             specs.append(WeightSpec(self.sink_name, (self.n_heads,), role="vector"))
         if self.bias_names is not None:
             specs += [WeightSpec(n, (w,), role="vector") for n, w in
-                      zip(self.bias_names, (self.q_dim, self.kv_dim, self.v_dim, self.hidden))]
+                      zip(self.bias_names, (self.q_dim, self.kv_dim, self.v_dim, self.hidden)) if n is not None]
         if self.distance_rows is not None:
             specs.append(WeightSpec(self.distance_rows[0], (ANY_SIZE, self.n_heads), role="vector", free_size=32))
         if self.head_gate_name is not None:
             specs.append(WeightSpec(self.head_gate_name, (self.n_heads, self.hidden)))
+        if self.value_gate_name is not None:
+            specs.append(WeightSpec(self.value_gate_name, (self.out_dim, self.hidden)))
         if self.value_mix is not None:
             specs.append(WeightSpec(self.value_mix[0], (), role="vector", init="unit_interval"))
         return specs
@@ -255,7 +265,7 @@ class GqaAttention(Mixer):
         self.run_head_dim, self.run_value_dim = self.head_dim, self.value_dim
         hd, vd = self.head_dim, self.value_dim
         self.run_eps, norm_scale = self.eps, 1.0
-        bq, bk, bv, self.b_out = (weights[n] for n in self.bias_names) if self.bias_names is not None else (None,) * 4
+        bq, bk, bv, self.b_out = (weights[n] if n is not None else None for n in self.bias_names) if self.bias_names is not None else (None,) * 4
         if (self.pad_heads and dtype == torch.bfloat16 and max(hd, vd) <= 128 and not (hd == vd and hd in (64, 128))
                 and (self.position is None or hasattr(self.position, "inv_freq_host"))):
             P = 64 if max(hd, vd) <= 64 else 128
@@ -284,14 +294,16 @@ class GqaAttention(Mixer):
         self.q_norm = weights[self.q_norm_name] if self.q_norm_name else None
         self.k_norm = weights[self.k_norm_name] if self.k_norm_name and self.own_kv else None
         if self.run_head_dim != hd:          # see `pad_heads`: the norms' weights behind the padding meet zeros
-            self.q_norm, self.k_norm = (None if w is None else torch.nn.functional.pad(w * norm_scale, (0, self.run_head_dim - hd))
+            pad = (0, self.run_head_dim - hd)      # a norm over the whole projection has a weight per head and entry
+            self.q_norm, self.k_norm = (None if w is None else torch.nn.functional.pad((w * norm_scale).reshape(-1, hd), pad).reshape(-1)
                                         for w in (self.q_norm, self.k_norm))
-        if self.head_gate_name is not None:  # the gates' logits are further columns of the same contraction
-            self.w_qkv = torch.cat([self.w_qkv, weights[self.head_gate_name]], dim=0)
+        gate_name = self.head_gate_name or self.value_gate_name
+        if gate_name is not None:            # the gates' logits are further columns of the same contraction
+            self.w_qkv = torch.cat([self.w_qkv, weights[gate_name]], dim=0)
         if self.bias_names is not None:
             b = torch.cat([bq, bk, bv])
             self.b_qkv = torch.nn.functional.pad(b, (0, self.w_qkv.shape[0] - b.shape[0]))
-        if self.head_gate_name is not None:
+        if gate_name is not None:
             self.w_qkv = pad_rows(self.w_qkv)
             if self.b_qkv is not None:
                 self.b_qkv = torch.nn.functional.pad(self.b_qkv, (0, self.w_qkv.shape[0] - self.b_qkv.shape[0]))
@@ -334,6 +346,8 @@ class GqaAttention(Mixer):
         if not self.own_kv and call.writes_kv:
             raise ValueError("attention: a mixer without key and value weights must read another call's cache")
         # a call that reads another call's cache needs its queries only (the stacked rows start with q)
+        if self.value_gate_name is not None and not call.writes_kv:
+            raise ValueError("attention: a gate per value goes with a call that writes its own cache")
         w_qkv = self.w_qkv[:self.q_dim] if self.span_prepare and self.own_kv and not call.writes_kv else self.w_qkv
         qkv = linear(xn, w_qkv, bias=self.b_qkv)
         rot = self.position.rotary() if self.position is not None else None
@@ -347,17 +361,18 @@ class GqaAttention(Mixer):
                 raise ValueError("attention: norms over the whole projection take the half-split pairing only")
             q = kernels.qk_prepare_span(qkv, kv.k, kv.v, self.q_norm, self.k_norm, value_dim=vd,
                                         write_kv=call.writes_kv, inv_freq=rot.inv_freq if rot else None,
-                                        n_rot=rot.n_rot if rot else 0, **common)
+                                        n_rot=rot.n_rot if rot else 0, rot_amp=rot.amplitude if rot else 1.0, **common)
         elif fused:
             mix = self._values_to_mix(ctx, qkv) if self.value_mix is not None else None
             q = kernels.qk_prepare(qkv, kv.k, kv.v, self.q_norm, self.k_norm, rot.inv_freq if rot else None, mix_values=mix,
                                    n_rot=rot.n_rot if rot else 0, interleaved=rot.interleaved if rot else False,
                                    write_kv=call.writes_kv, value_dim=vd,
-                                   unit_norm_after=self.unit_norm_after, query_temperature=self.query_temperature, **common)
+                                   unit_norm_after=self.unit_norm_after, query_temperature=self.query_temperature,
+                                   rot_amp=rot.amplitude if rot else 1.0, **common)
         else:
             # A position encoding that is not a rotation table runs between the norm and the
             # cache write: norm in place of a copy of qkv, the encoding's own step, then the write.
-            if self.value_dim != self.head_dim or self.query_temperature is not None or self.value_mix or self.head_gate_name:
+            if self.value_dim != self.head_dim or self.query_temperature is not None or self.value_mix or self.head_gate_name or self.value_gate_name:
                 raise ValueError("attention: a position encoding of its own needs values as wide as the keys and takes "
                                  "no query temperature, no mixed values and no gate")
             normed = kernels.qk_normed(qkv, self.q_norm, self.k_norm, self.n_heads, self.n_kv, self.head_dim, self.eps,
@@ -380,6 +395,9 @@ class GqaAttention(Mixer):
                                 bias=(self.bias_r1, self.bias_r2) if self.distance_bias is not None else None,
                                 talk=self.talk, keep_first=self.keep_first, sink=self.sink, softcap=self.softcap,
                                 distance_table=self.distance_table, chunk=self.chunk, gate=self._gate_logits(qkv))
+        if self.value_gate_name is not None:
+            at = (self.n_heads + self.n_kv) * hd + self.n_kv * vd
+            kernels.value_gate(att, qkv[:, at:at + self.out_dim], self.n_heads, self.value_dim)
         linear(att, self.w_out, out=out, accumulate=accumulate, bias=self.b_out)
 
     def _gate_logits(self, qkv):

@@ -112,6 +112,7 @@ class RotaryParams:
     inv_freq: torch.Tensor          # [n_rot / 2] float32 on the device
     n_rot: int
     interleaved: bool = False
+    amplitude: float = 1.0          # factor on the cosines and sines
 
 
 class Part:

@@ -27,7 +27,7 @@ import torch
 
 from .. import kernels
 from .base import FEED_FORWARDS, FeedForward, WeightSpec
-from .feedforward import SwiGLU
+from .feedforward import ActMlp, SwiGLU
 from .linear import FUSION_GROUP, interleave_rows
 
 # From this many tokens on a step whose ids the host knows runs expert by expert.  Below it the streaming
@@ -70,6 +70,7 @@ def _expert_rows(experts: np.ndarray, tokens: np.ndarray, n_experts: int, tile: 
 
 class TableMoE(FeedForward):
     takes_residual_rows = True       # the shared expert's gate reads the float32 rows
+    gated = True                     # the experts are gated units
 
     def __init__(self, hidden: int, ffn_dim: int, n_experts: int, top: int, vocab: int, table_name: str,
                  expert_names, shared: Optional[FeedForward] = None, shared_gate_name: Optional[str] = None):
@@ -169,11 +170,11 @@ class TableMoE(FeedForward):
         self._staged.record()
         return dev
 
-    def _expert_by_expert(self, ctx, rows, host_tokens, out, accumulate, chosen=None, weights=None):
-        """`chosen` (host, flat [n * top]) names the experts when a router picked them, `weights` (device, float32
+    def _expert_by_expert(self, ctx, rows, host_tokens, out, accumulate, chosen=None, weights=None, weight_input=False):
+        """`weight_input`: the weights multiply the gathered rows instead of the experts' results.  `chosen` (host, flat [n * top]) names the experts when a router picked them, `weights` (device, float32
         [n, top]) their weights; without them the table decides and every expert weighs 1/top."""
         tile = kernels.GEMM_TC_GROUP_ROWS
-        grouped = (self.interleave and rows.dtype == torch.bfloat16 and self.hidden % 8 == 0 and self.ffn_dim % 8 == 0
+        grouped = (self.interleave and self.gated and rows.dtype == torch.bfloat16 and self.hidden % 8 == 0 and self.ffn_dim % 8 == 0
                    and rows.is_contiguous())
 
         def make():
@@ -181,6 +182,8 @@ class TableMoE(FeedForward):
                 row_token, pair_row, bounds = self.routing(host_tokens, tile if grouped else 1)
             else:
                 row_token, pair_row, bounds = expert_rows(chosen, self.n_experts, self.top, tile if grouped else 1)
+            if weight_input:             # a padding row stays -1; the others name their pair instead of their token
+                row_token[pair_row] = np.arange(pair_row.size, dtype=np.int32)
             tile_group = np.repeat(np.arange(self.n_experts), np.diff(bounds) // tile).astype(np.int32) if grouped \
                 else np.zeros(0, dtype=np.int32)
             sizes = np.cumsum([row_token.size, pair_row.size, tile_group.size])
@@ -189,7 +192,7 @@ class TableMoE(FeedForward):
 
         # a table's rows depend on the step's ids alone; a router's on what this very call read
         row_token, pair_row, tile_group, bounds = ctx.memo(("expert rows", id(self)), make) if chosen is None else make()
-        xg = kernels.moe_gather(rows, row_token)
+        xg = kernels.moe_gather(rows, row_token, weights if weight_input else None)
         if grouped:
             h = kernels.gemm_tc_grouped(xg, self.w_gate_up, tile_group, swiglu=True)
             y = kernels.gemm_tc_grouped(h, self.w_down, tile_group, out_dtype=torch.float32)
@@ -199,8 +202,9 @@ class TableMoE(FeedForward):
                 r0, r1 = int(bounds[e]), int(bounds[e + 1])
                 if r1 > r0:
                     ff.forward(ctx, xg[r0:r1], y[r0:r1], False)
-        kernels.moe_combine(y, pair_row, self.top, out, accumulate, weights,
-                            identity_rows=rows if getattr(self, "n_identity", 0) else None)
+        kernels.moe_combine(y, pair_row, self.top, out, accumulate, None if weight_input else weights,
+                            identity_rows=rows if getattr(self, "n_identity", 0) else None,
+                            plain_weight=1.0 if weight_input else None)
 
 
 class RoutedMoE(TableMoE):
@@ -219,17 +223,32 @@ class RoutedMoE(TableMoE):
     only; the weights are made of the scores alone.  `n_identity`: the router has that many outputs more than there are
     experts with weights, and its last `n_identity` outputs stand for identity experts, whose result is the row they
     read (times the weight); `top` may then exceed nothing but the router's outputs.  `shared`: a feed-forward every
-    token takes, added with weight 1."""
+    token takes, added with weight 1.  `score` "sigmoid": an expert's score is the sigmoid of its own logit instead of the
+    softmax; `renormalize` False: the weights are the chosen scores as they are.  `weight_input`: a weight multiplies what its
+    expert READS, y_t = sum_k Expert[e_k](s_k x_t).  `act`: the experts are ungated, W_down[e] act(W_up[e] x), act one of
+    `kernels.ACTIVATIONS`; `expert_names(e)` then gives (up name, down name)."""
+
 
     takes_residual_rows = False
     takes_pending_norm = True
 
     def __init__(self, hidden: int, ffn_dim: int, n_experts: int, top: int, router_name: str, expert_names,
-                 correction_name: Optional[str] = None, n_identity: int = 0, shared: Optional[FeedForward] = None):
+                 correction_name: Optional[str] = None, n_identity: int = 0, shared: Optional[FeedForward] = None,
+                 score: str = "softmax", renormalize: bool = True, weight_input: bool = False, act: Optional[str] = None):
+        if score not in ("softmax", "sigmoid"):
+            raise ValueError(f"router scores {score!r}: 'softmax' or 'sigmoid'")
+        if weight_input and n_identity:
+            raise ValueError("weights on the experts' inputs do not go with identity experts")
+        if act is not None and act not in kernels.ACTIVATIONS:
+            raise ValueError(f"activation {act!r}; known: {sorted(kernels.ACTIVATIONS)}")
         if n_identity < 0 or not 0 < top <= n_experts + n_identity:
             raise ValueError(f"{top} experts per token out of {n_experts} and {n_identity} identity experts")
         super().__init__(hidden, ffn_dim, n_experts, min(top, n_experts), 1, "", expert_names, shared=shared)
         self.top = top
+        self.score, self.renormalize, self.weight_input = score, bool(renormalize), bool(weight_input)
+        self.act, self.gated = act, act is None
+        if not self.gated:
+            self.interleave = 0
         self.router_name, self.w_router = router_name, None
         self.correction_name, self.correction, self.n_identity = correction_name, None, int(n_identity)
 
@@ -242,17 +261,24 @@ class RoutedMoE(TableMoE):
         specs = [WeightSpec(self.router_name, (self.n_router, D), role="vector")]      # kept in float32
         if self.correction_name is not None:
             specs.append(WeightSpec(self.correction_name, (self.n_router,), role="vector"))
-        for g, u, d in self.names:
-            specs += [WeightSpec(g, (F, D)), WeightSpec(u, (F, D)), WeightSpec(d, (D, F))]
+        for *ups, d in self.names:           # gate and up, or up alone
+            specs += [WeightSpec(u, (F, D)) for u in ups] + [WeightSpec(d, (D, F))]
         return specs
 
     def load(self, weights, dtype, device):
         self.w_router = weights[self.router_name].contiguous()
         self.correction = weights[self.correction_name].contiguous() if self.correction_name is not None else None
+        self.w_down = torch.stack([weights[n[-1]] for n in self.names]).contiguous()
+        self.experts = []
+        if not self.gated:
+            self.w_gate_up = torch.stack([weights[u] for u, _ in self.names]).contiguous()
+            for e in range(self.n_experts):
+                ff = ActMlp(self.hidden, self.ffn_dim, "", "", self.act)
+                ff.w_up, ff.w_down = self.w_gate_up[e], self.w_down[e]
+                self.experts.append(ff)
+            return
         stack = (lambda g, u: interleave_rows([g, u])) if self.interleave else (lambda g, u: torch.cat([g, u], dim=0))
         self.w_gate_up = torch.stack([stack(weights[g], weights[u]) for g, u, _ in self.names]).contiguous()
-        self.w_down = torch.stack([weights[d] for _, _, d in self.names]).contiguous()
-        self.experts = []
         for e in range(self.n_experts):
             ff = SwiGLU(self.hidden, self.ffn_dim, "", "", "")
             ff.w_gate_up, ff.w_down = self.w_gate_up[e], self.w_down[e]
@@ -268,23 +294,27 @@ class RoutedMoE(TableMoE):
             self.shared.forward(ctx, rows, out, True)
 
     def _experts(self, ctx, rows, out, accumulate):
-        ids, wts = kernels.moe_router(rows, self.w_router, self.top, self.correction)
+        ids, wts = kernels.moe_router(rows, self.w_router, self.top, self.correction, sigmoid=self.score == "sigmoid",
+                                      renormalize=self.renormalize)
         if ctx.is_decode or rows.shape[0] < GROUPED_MIN_TOKENS:
             kernels.moe_routed(rows, ids, wts, self.w_gate_up, self.interleave, self.w_down, ctx.status, out=out,
-                               accumulate=accumulate, n_identity=self.n_identity)
+                               accumulate=accumulate, n_identity=self.n_identity, act=self.act, weight_input=self.weight_input)
             return
         tile = kernels.GEMM_TC_GROUP_ROWS
-        if (self.interleave and rows.dtype == torch.bfloat16 and self.hidden % 8 == 0 and self.ffn_dim % 8 == 0
+        if ((self.interleave or not self.gated) and rows.dtype == torch.bfloat16 and self.hidden % 8 == 0 and self.ffn_dim % 8 == 0
                 and rows.is_contiguous() and self.n_experts <= 4096):
             # the rows are sorted by expert where the router left its choice: the step never waits for the host
-            row_token, pair_row, tile_group = kernels.moe_expert_rows(ids, self.n_experts, tile, self.n_identity)
-            xg = kernels.moe_gather(rows, row_token)
-            h = kernels.gemm_tc_grouped(xg, self.w_gate_up, tile_group, swiglu=True)
+            row_token, pair_row, tile_group = kernels.moe_expert_rows(ids, self.n_experts, tile, self.n_identity,
+                                                                       name_pairs=self.weight_input)
+            xg = kernels.moe_gather(rows, row_token, wts if self.weight_input else None)
+            h = kernels.gemm_tc_grouped(xg, self.w_gate_up, tile_group, swiglu=self.gated, act=self.act)
             y = kernels.gemm_tc_grouped(h, self.w_down, tile_group, out_dtype=torch.float32)
-            kernels.moe_combine(y, pair_row, self.top, out, accumulate, wts, identity_rows=rows if self.n_identity else None)
+            kernels.moe_combine(y, pair_row, self.top, out, accumulate, None if self.weight_input else wts,
+                                identity_rows=rows if self.n_identity else None, plain_weight=1.0 if self.weight_input else None)
             return
         chosen = ids.cpu().numpy().reshape(-1).astype(np.int64)
-        self._expert_by_expert(ctx, rows, None, out, accumulate, chosen=np.clip(chosen, 0, self.n_router - 1), weights=wts)
+        self._expert_by_expert(ctx, rows, None, out, accumulate, chosen=np.clip(chosen, 0, self.n_router - 1), weights=wts,
+                               weight_input=self.weight_input)
 
 
 FEED_FORWARDS.register("table_moe", TableMoE)

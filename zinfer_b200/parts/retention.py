@@ -37,8 +37,8 @@ class Retention(Mixer):
                  key_scale: Optional[float] = None, norm_eps: float = 1e-5):
         if len(decay) != n_heads:
             raise ValueError(f"retention: {len(decay)} decays for {n_heads} heads")
-        if position is not None and position.interleaved:
-            raise ValueError("retention: the recurrence kernel rotates half-split pairs only")
+        if position is not None and (position.interleaved or position.amplitude != 1.0):
+            raise ValueError("retention: the recurrence kernel rotates half-split pairs, without a factor on cosines and sines")
         self.hidden, self.n_heads, self.dim, self.value_dim, self.eps = hidden, n_heads, dim, value_dim, float(norm_eps)
         self.decay_host = [float(g) for g in decay]
         self.key_scale = float(dim) ** -0.5 if key_scale is None else float(key_scale)
