@@ -439,17 +439,63 @@ def zosurax_like_varolorn(sz: dict) -> dict:
             "norm": {"eps": 1e-5}, "layers": layers}
 
 
+# Nipizen beside the closest existing architecture at equal size, Pirisun (attention beside a recurrence, routed experts): width,
+# layers, vocabulary, the attention heads, the recurrence's heads and sizes and the number of experts are the same, and the
+# experts have the same parameters (two matrices of one and a half times the hidden units here, three there).  Every Pirisun layer is
+# its pair of mixers, without identity and shared experts and with no temperature or cap; every fourth Nipizen layer is an mLSTM in
+# place of the pair.
+NIPIZEN_SIZES = {
+    "w1024": dict(width=1024, layers=8, heads=16, kv=4, dim=64, rec_heads=8, rec_dim=128, conv=4, mem_heads=4, mem_dim=128, mem_vdim=256,
+                  experts=16, top=2, ff=1024, vocab=32768),
+    "w2048": dict(width=2048, layers=8, heads=32, kv=8, dim=64, rec_heads=16, rec_dim=128, conv=4, mem_heads=8, mem_dim=128, mem_vdim=256,
+                  experts=16, top=2, ff=2048, vocab=65536),
+}
+
+
+def nipizen_config(sz: dict) -> dict:
+    layers = []
+    for i in range(sz["layers"]):
+        if i % 4 == 3:
+            kind, mixer = "mlstm", {"heads": sz["mem_heads"], "dim": sz["mem_dim"], "vdim": sz["mem_vdim"], "gate_cap": 15.0}
+        else:
+            kind = "parallel"
+            mixer = {"left": {"heads": sz["heads"], "kv_heads": sz["kv"], "dim": sz["dim"], "vdim": sz["dim"], "scale": sz["dim"] ** -0.5,
+                              "rot": {"base": 10000.0, "dims": sz["dim"],
+                                      "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
+                     "right": {"heads": sz["rec_heads"], "kv_heads": sz["rec_heads"], "dim": sz["rec_dim"],
+                               "vdim": sz["width"] // sz["rec_heads"], "conv": sz["conv"]},
+                     "left_scale": 0.5, "right_scale": 0.5}
+        mlp = {"kind": "moe", "expert": {"ff": sz["ff"] * 3 // 2}, "router": {"experts": sz["experts"], "top": sz["top"]}}
+        layers.append({"type": kind, "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Nipizen", "vocab": sz["vocab"], "width": sz["width"], "max_positions": CONTEXT,
+            "norm": {"eps": 1e-5}, "layers": layers}
+
+
+def pirisun_like_nipizen(sz: dict) -> dict:
+    layers = []
+    for i in range(sz["layers"]):
+        mixer = {"left": {"heads": sz["heads"], "kv_heads": sz["kv"], "dim": sz["dim"], "vdim": sz["dim"], "scale": sz["dim"] ** -0.5},
+                 "right": {"heads": sz["rec_heads"], "dim": sz["rec_dim"], "vdim": sz["width"] // sz["rec_heads"],
+                           "decay": [1.0 - 1.0 / (24.0 * (h + 1)) for h in range(sz["rec_heads"])],
+                           "rot": {"base": 10000.0, "dims": sz["rec_dim"]}}}
+        mlp = {"kind": "moe", "expert": {"ff": sz["ff"]}, "router": {"experts": sz["experts"], "top": sz["top"]}}
+        layers.append({"type": "parallel", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Pirisun", "vocab": sz["vocab"], "width": sz["width"], "max_positions": CONTEXT,
+            "norm": {"eps": 1e-5}, "logit_scale": 1.0, "layers": layers}
+
+
 # new architecture -> (sizes, its configuration, the configuration of the architecture beside it, that one's name)
 COMPARISONS = {"ponusun": (PONUSUN_SIZES, ponusun_config, lfm2_like, "lfm2"),
                "zosurax": (ZOSURAX_SIZES, zosurax_config, lfm2_like_zosurax, "lfm2"),
                "kerotar": (KEROTAR_SIZES, kerotar_config, ponusun_like_kerotar, "ponusun"),
                "pirisun": (PIRISUN_SIZES, pirisun_config, kerotar_like_pirisun, "kerotar"),
-               "varolorn": (VAROLORN_SIZES, varolorn_config, zosurax_like_varolorn, "zosurax")}
+               "varolorn": (VAROLORN_SIZES, varolorn_config, zosurax_like_varolorn, "zosurax"),
+               "nipizen": (NIPIZEN_SIZES, nipizen_config, pirisun_like_nipizen, "pirisun")}
 
 
 def ponusun_arm(args) -> dict:
-    """Prompt and single-token throughput of Ponusun (or Zosurax, Kerotar, Pirisun, Varolorn: `--model`) and of the closest earlier
-    architecture (LFM2; for Kerotar, Ponusun; for Pirisun, Kerotar; for Varolorn, Zosurax) at equal size, random
+    """Prompt and single-token throughput of Ponusun (or Zosurax, Kerotar, Pirisun, Varolorn, Nipizen: `--model`) and of the closest earlier
+    architecture (LFM2; for Kerotar, Ponusun; for Pirisun, Kerotar; for Varolorn, Zosurax; for Nipizen, Pirisun) at equal size, random
     weights, bfloat16: one prompt of --prefill-tokens tokens in one step (median of 5), then --steps single-token
     steps of --batch sequences replayed from CUDA graphs (prompts of 512..2,048 tokens)."""
     import numpy as np
@@ -613,10 +659,10 @@ def main() -> int:
                     help="with --only prefill: the prompt's length (the headline line always uses 2,048)")
     ap.add_argument("--model", default="1.2b", choices=["1.2b"] + list(COMPARISONS) + sorted(SECONDARY),
                     help="1.2b: the headline benchmark; 2.6b, 350m: the secondary workloads (decode only); ponusun, zosurax, "
-                         "kerotar, pirisun, varolorn: that architecture beside the closest earlier one at equal size, prompt and single-token steps")
-    ap.add_argument("--size", default="", choices=[""] + sorted(PONUSUN_SIZES), help="with --model ponusun, zosurax, kerotar, pirisun or varolorn: one size only")
+                         "kerotar, pirisun, varolorn, nipizen: that architecture beside the closest earlier one at equal size, prompt and single-token steps")
+    ap.add_argument("--size", default="", choices=[""] + sorted(PONUSUN_SIZES), help="with --model ponusun, zosurax, kerotar, pirisun, varolorn or nipizen: one size only")
     ap.add_argument("--arch", default="", choices=["", "lfm2"] + list(COMPARISONS),
-                    help="with --model ponusun, zosurax, kerotar, pirisun or varolorn: one architecture of the two only")
+                    help="with --model ponusun, zosurax, kerotar, pirisun, varolorn or nipizen: one architecture of the two only")
     args = ap.parse_args()
     args.warmup = max(3, args.warmup)
     if args.impl == "reference":

@@ -3,78 +3,135 @@
 //     S <- diag(g_t) S        u_t = beta_t (v_t - S^T k_t)        S <- S + k_t u_t^T        o_t = S^T q_t
 //
 // g_t in (0, 1] per head and channel, beta_t in (0, 1) per head; q and k (unit vectors) may be shared by the heads of a group.
-// Everything here is float32.
+// Everything here is float32.  State in memory: [H, e, d4], d4 = d rounded up to a multiple of 4, channels side by side.
 //
-// delta_scan_kernel serves prompt steps and single-token steps.  What a token writes depends on what its key reads of the state
-// before it, so the tokens are a chain; its length per token is what the kernel's layout is made for.  A column of S (one value
-// channel) is owned by L neighbouring lanes, each of which keeps CH of the d key channels in registers; columns never meet.  The
-// read S^T k is a sum in registers and log2(L) shuffles, the write needs nothing of another lane, and the read-out S^T q of one
-// token overlaps the next token's read.  The decay is folded into the key for the read (sum (g k) S), so the chain is: read, shuffles,
-// one multiplication by beta, one fused multiply-add.  A block owns (sequence, head, COLS columns); q, k, g of the next TT tokens reach
-// shared memory with cp.async while the current TT are worked on.  State in memory: [H, e, d4], d4 = d rounded up to a multiple of 4,
-// channels side by side, so that a column's lanes read whole lines.  The order of every sum is fixed by the layout alone: a
-// sequence cut into steps gives the same bits as the whole.
+// What a token writes depends on what its key reads of the state before it, so the tokens are a chain.  Prompt steps walk it four
+// tokens (a chunk, counted from the sequence's first token of the step) at a time.  With S0 the state before a chunk, c_i the product
+// of the decays of its tokens 0..i and p_ij that of tokens j+1..i (per channel):
 //
-// delta_prepare_kernel comes before it in prompt steps: unit vectors and decays, once for all the blocks that read them.  In
-// single-token steps (RAW) the scan does both itself on the one token it has.
+//     read of token i        S^T k_i = S0^T (c_i k_i) + sum_{j<i} A_ij u_j        A_ij = sum_channels k_i p_ij k_j
+//     output of token i      o_i = S0^T (c_i q_i) + sum_{j<=i} B_ij u_j           B_ij = sum_channels q_i p_ij k_j
+//     state after the chunk  c_3 S0 + sum_j (p_3j k_j) u_j^T
+//
+// so the four reads and the four outputs of a chunk are sums over S0 that do not wait for one another, and only the four u, a
+// small triangular system per column, are a chain.  Products of decays are never divided by, so nothing overflows.
+// delta_chunk_prepare_kernel makes the vectors and the numbers A, B once per (chunk, head), with unit vectors, decays and beta on
+// the way; delta_chunk_kernel owns (sequence, head, some columns of S) per block and walks the chunks: a column lies in L
+// neighbouring lanes, CH channels each, in registers; the vectors of the next chunks reach shared memory with cp.async meanwhile.
+//
+// delta_single_kernel is the single-token step: the recurrence as it stands, unit vectors and decays made on the spot.
 #include "common.cuh"
 #include <math.h>
 
 #define DL_THREADS 128
 #define DL_MAX_D 512
+#define DL_CHUNK 4
 #define DL_UNIT_EPS 1e-6f     // inside the root of the unit vectors' length
 
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
-// In place.  Rows of qkv [q (G*d) | k (G*d) | ...]: every q and k head is divided by sqrt(sum of squares + 1e-6), q then multiplied by
-// q_scale.  Rows of a [H*d]: a <- exp(-exp(a_log_h) softplus(a + dt_bias)).  One warp per (token, head slot): G queries, G keys, H decays.
-__global__ void __launch_bounds__(256)
-    delta_prepare_kernel(float* __restrict__ qkv, int ld, float* __restrict__ a, int ld_a, const float* __restrict__ a_log,
-                         const float* __restrict__ dt_bias, long long items, int G, int H, int d, float q_scale) {
-  zk_let_next_start();
-  zk_wait_prior();
-  const int lane = threadIdx.x & 31;
-  const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (item >= items) return;
-  const int slots = 2 * G + H;
-  const long long t = item / slots;
-  const int s = (int)(item - t * slots);
-  if (s < 2 * G) {
-    float* head = qkv + (size_t)t * ld + (size_t)s * d;
-    float ss = 0.f;
-    if (d <= 128) {             // the head stays in registers between the sum and the scaling
-      float v[4];
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        v[j] = lane + 32 * j < d ? head[lane + 32 * j] : 0.f;
-        ss = fmaf(v[j], v[j], ss);
-      }
-      const float mul = (s < G ? q_scale : 1.0f) / sqrtf(warp_sum(ss) + DL_UNIT_EPS);
-#pragma unroll
-      for (int j = 0; j < 4; ++j)
-        if (lane + 32 * j < d) head[lane + 32 * j] = v[j] * mul;
-      return;
-    }
-    for (int i = lane; i < d; i += 32) ss = fmaf(head[i], head[i], ss);
-    const float mul = (s < G ? q_scale : 1.0f) / sqrtf(warp_sum(ss) + DL_UNIT_EPS);
-    for (int i = lane; i < d; i += 32) head[i] *= mul;
-    return;
-  }
-  const int h = s - 2 * G;
-  float* row = a + (size_t)t * ld_a + (size_t)h * d;
-  const float* b = dt_bias + (size_t)h * d;
-  const float rate = -expf(a_log[h]);
-  for (int i = lane; i < d; i += 32) row[i] = expf(rate * softplus_f(row[i] + b[i]));
-}
-
 struct DeltaArgs {
-  const float *qkv, *g, *zb, *a_log, *dt_bias;      // zb: raw beta logits [n, H], rows ld_b apart; a_log, dt_bias: RAW only
+  const float *qkv, *a, *zb, *a_log, *dt_bias;      // as zk_delta_scan takes them
+  float *vec, *total, *num;                         // prompt steps: [n, H, 3, d4], [chunks, H, d4], [n, H, 8]
   float *state, *o;
-  const int *cu_q, *seq_slot;
+  const int *cu_q, *seq_slot, *tok_seq;
   long long state_stride;
-  int ld, ld_g, ld_b, H, G, d, e, d4, vec;          // vec: heads start on 16-byte boundaries
+  int ld, ld_a, ld_b, H, G, d, e, d4;
   float q_scale;
 };
+
+// Chunks of all sequences have distinct numbers below n / 4 + n_seqs: that of the chunk of sequence b that starts at row t.
+__device__ __forceinline__ int chunk_number(int t0, int t, int b) { return t0 / DL_CHUNK + (t - t0) / DL_CHUNK + b; }
+
+// One warp per (token that starts a chunk, head); the warps of other tokens end at once.  vec: c_i k_i, c_i q_i, p_3i k_i per token;
+// total: c_3; num, per token i: A_i0 A_i1 A_i2 beta_i B_i0 B_i1 B_i2 B_i3 (zeros where j is too large).  NJ: channels per lane.
+template <int NJ>
+__global__ void __launch_bounds__(128) delta_chunk_prepare_kernel(const DeltaArgs p) {
+  zk_wait_prior();      // and no early start of the kernel behind: its few long blocks would crowd onto the SMs that have room first
+  const int t = blockIdx.x, lane = threadIdx.x & 31, h = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int b = p.tok_seq[t], t0 = p.cu_q[b];
+  if (((t - t0) & (DL_CHUNK - 1)) != 0 || h >= p.H) return;
+  const int nt = min(DL_CHUNK, p.cu_q[b + 1] - t);
+  const int hk = h / (p.H / p.G);
+  const float rate = -expf(p.a_log[h]);
+  float q[DL_CHUNK][NJ], k[DL_CHUNK][NJ], g[DL_CHUNK][NJ];
+#pragma unroll
+  for (int i = 0; i < DL_CHUNK; ++i) {
+    const float* row = p.qkv + (size_t)(t + (i < nt ? i : 0)) * p.ld;
+    const float* ar = p.a + (size_t)(t + (i < nt ? i : 0)) * p.ld_a + (size_t)h * p.d;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int c = lane + 32 * j;
+      const bool ok = i < nt && c < p.d;
+      q[i][j] = ok ? row[hk * p.d + c] : 0.f;
+      k[i][j] = ok ? row[(p.G + hk) * p.d + c] : 0.f;
+      g[i][j] = ok ? expf(rate * softplus_f(ar[c] + p.dt_bias[(size_t)h * p.d + c])) : 1.f;
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < DL_CHUNK; ++i) {
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      sq = fmaf(q[i][j], q[i][j], sq);
+      sk = fmaf(k[i][j], k[i][j], sk);
+    }
+    const float mq = p.q_scale / sqrtf(warp_sum(sq) + DL_UNIT_EPS), mk = 1.0f / sqrtf(warp_sum(sk) + DL_UNIT_EPS);
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      q[i][j] *= mq;
+      k[i][j] *= mk;
+    }
+  }
+  // the sixteen numbers: A_ij at i*i + j, B_ij at i*i + i + j
+  float v[16];
+#pragma unroll
+  for (int x = 0; x < 16; ++x) v[x] = 0.f;
+  const size_t vec_row = (size_t)3 * p.d4;
+#pragma unroll
+  for (int j = 0; j < NJ; ++j) {
+    const int c = lane + 32 * j;
+    float cum = 1.f;
+#pragma unroll
+    for (int i = 0; i < DL_CHUNK; ++i) {
+      cum *= g[i][j];
+      float w = k[i][j];                       // p_li k_i for growing l
+      v[i * i + i + i] = fmaf(q[i][j], w, v[i * i + i + i]);
+#pragma unroll
+      for (int l = i + 1; l < DL_CHUNK; ++l) {
+        w *= g[l][j];
+        v[l * l + i] = fmaf(k[l][j], w, v[l * l + i]);
+        v[l * l + l + i] = fmaf(q[l][j], w, v[l * l + l + i]);
+      }
+      if (i < nt && c < p.d4) {
+        float* dst = p.vec + ((size_t)(t + i) * p.H + h) * vec_row + c;
+        dst[0] = cum * k[i][j];
+        dst[p.d4] = cum * q[i][j];
+        dst[2 * p.d4] = w;
+      }
+    }
+    if (c < p.d4) p.total[((size_t)chunk_number(t0, t, b) * p.H + h) * p.d4 + c] = cum;
+  }
+  // sum all sixteen over the lanes: each exchange halves what a lane holds; lanes 2x and 2x + 1 end with number x
+#pragma unroll
+  for (int off = 16, n = 8; n >= 1; off >>= 1, n >>= 1) {
+    const bool up = lane & off;
+#pragma unroll
+    for (int x = 0; x < n; ++x) {
+      const float send = up ? v[x] : v[x + n], keep = up ? v[x + n] : v[x];
+      v[x] = keep + __shfl_xor_sync(0xffffffffu, send, off);
+    }
+  }
+  v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
+  const int i = lane >> 3, s = lane & 7, j = s < 4 ? s : s - 4;
+  const bool is_a = s < 3 && j < i, is_b = s >= 4 && j <= i;
+  const float got = __shfl_sync(0xffffffffu, v[0], 2 * (is_a ? i * i + j : (is_b ? i * i + i + j : 0)));
+  if (i < nt) {
+    float out = is_a || is_b ? got : 0.f;
+    if (s == 3) out = 1.0f / (1.0f + expf(-p.zb[(size_t)(t + i) * p.ld_b + h]));
+    p.num[((size_t)(t + i) * p.H + h) * 8 + s] = out;
+  }
+}
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
@@ -82,69 +139,67 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
 __device__ __forceinline__ void cp_async4(void* dst, const void* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
+__device__ __forceinline__ float dot4(const float4& a, const float4& b, float acc) {
+  return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, acc))));
+}
 
-// L lanes per column, CH channels per lane (a multiple of 4, quads l, l + L, ...), TT tokens staged at once.
-template <int L, int CH, int TT, bool RAW>
-__global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(const DeltaArgs p) {
-  constexpr int DP = L * CH, NQ = CH / 4, COLS = DL_THREADS / L, WCOLS = 32 / L;
-  __shared__ __align__(16) float ks[2][TT][DP], qs[2][TT][DP], gs[2][TT][DP];
-  __shared__ float vs[2][TT][COLS], os[TT][COLS], zs[2][TT];
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+// Shared memory of a block of the chunk kernel: two buffers of NC chunks, and the outputs of one.
+template <int L, int CH, int X, int NC>
+struct ChunkSmem {
+  static constexpr int DP = L * CH, TT = NC * DL_CHUNK, COLS = DL_THREADS / L * X;
+  static constexpr int VEC = TT * 3 * DP, TOTAL = NC * DP, NUM = TT * 8, VAL = TT * COLS;       // floats
+  static constexpr int BUF = VEC + TOTAL + NUM + VAL;
+  static constexpr size_t BYTES = sizeof(float) * (2 * BUF + VAL);
+};
+
+// L lanes per column, CH channels per lane (a multiple of 4, quads l, l + L, ...), X columns per lane, NC chunks staged at once.
+template <int L, int CH, int X, int NC>
+__global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs p) {
+  using M = ChunkSmem<L, CH, X, NC>;
+  constexpr int DP = M::DP, TT = M::TT, NQ = CH / 4, COLS = M::COLS, GROUPS = DL_THREADS / L;
+  extern __shared__ __align__(16) float sm[];
+  float* os = sm + 2 * M::BUF;                       // [TT][COLS]
+  const int tid = threadIdx.x, l = tid % L, grp = tid / L;
   const int b = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * COLS;
-  const int l = lane % L, wc = warp * WCOLS + lane / L;      // this lane's part of its column, the column within the block
-  const int c = c0 + wc;
-  const bool col = c < p.e;
-  const int hk = h / (p.H / p.G);
-  if (p.d < DP) {          // channels beyond d are zero for good
-    for (int i = tid; i < 2 * TT * DP; i += DL_THREADS) {
-      (&ks[0][0][0])[i] = 0.f;
-      (&qs[0][0][0])[i] = 0.f;
-      (&gs[0][0][0])[i] = 0.f;
-    }
-    __syncthreads();
-  }
+  const int cols_here = min(COLS, p.e - c0);
+  for (int i = tid; i < 2 * M::BUF; i += DL_THREADS) sm[i] = 0.f;      // channels and columns that are not there stay zero
+  __syncthreads();
   zk_wait_prior();
   const int t0 = p.cu_q[b], t1 = p.cu_q[b + 1];
-  float* st = p.state + (size_t)p.seq_slot[b] * p.state_stride + ((size_t)h * p.e + (col ? c : 0)) * p.d4;
-  float4 S[NQ];
+  float* st = p.state + (size_t)p.seq_slot[b] * p.state_stride + (size_t)h * p.e * p.d4;
+  float4 S[X][NQ];
 #pragma unroll
-  for (int j = 0; j < NQ; ++j) {
-    const int i = 4 * (l + L * j);
-    S[j] = col && i < p.d4 ? *reinterpret_cast<const float4*>(st + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int x = 0; x < X; ++x) {
+    const int c = c0 + grp + x * GROUPS;             // this lane's columns of the block: grp, grp + GROUPS, ...
+#pragma unroll
+    for (int j = 0; j < NQ; ++j) {
+      const int i = 4 * (l + L * j);
+      S[x][j] = c < p.e && i < p.d4 ? *reinterpret_cast<const float4*>(st + (size_t)c * p.d4 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
   }
-  const int off_q = hk * p.d, off_k = (p.G + hk) * p.d, off_v = 2 * p.G * p.d + h * p.e + c0;
-  const int cols_here = min(COLS, p.e - c0);
+  const int nq = p.d4 >> 2, off_v = 2 * p.G * p.d + h * p.e + c0;
   auto fetch = [&](int buf, int tb) {
+    float* s = sm + buf * M::BUF;
     const int nt = min(TT, t1 - tb);
-    if (p.vec) {
-      const int nq = p.d >> 2;
-      for (int i = tid; i < nt * nq; i += DL_THREADS) {
-        const int tt = i / nq, x = 4 * (i - tt * nq);
-        const float* row = p.qkv + (size_t)(tb + tt) * p.ld;
-        cp_async16(&ks[buf][tt][x], row + off_k + x);
-        cp_async16(&qs[buf][tt][x], row + off_q + x);
-        cp_async16(&gs[buf][tt][x], p.g + (size_t)(tb + tt) * p.ld_g + (size_t)h * p.d + x);
-      }
-    } else {
-      for (int i = tid; i < nt * p.d; i += DL_THREADS) {
-        const int tt = i / p.d, x = i - tt * p.d;
-        const float* row = p.qkv + (size_t)(tb + tt) * p.ld;
-        cp_async4(&ks[buf][tt][x], row + off_k + x);
-        cp_async4(&qs[buf][tt][x], row + off_q + x);
-        cp_async4(&gs[buf][tt][x], p.g + (size_t)(tb + tt) * p.ld_g + (size_t)h * p.d + x);
-      }
+    for (int r = grp; r < nt * 3; r += GROUPS) {                       // a group of L lanes copies a vector
+      const float* src = p.vec + ((size_t)(tb + r / 3) * p.H + h) * 3 * p.d4 + (size_t)(r % 3) * p.d4;
+      for (int x = l; x < nq; x += L) cp_async16(s + (size_t)r * DP + 4 * x, src + 4 * x);
     }
-    for (int i = tid; i < nt * cols_here; i += DL_THREADS) {
-      const int tt = i / cols_here, x = i - tt * cols_here;
-      cp_async4(&vs[buf][tt][x], p.qkv + (size_t)(tb + tt) * p.ld + off_v + x);
+    for (int r = grp; r * DL_CHUNK < nt; r += GROUPS) {
+      const float* src = p.total + ((size_t)chunk_number(t0, tb + r * DL_CHUNK, b) * p.H + h) * p.d4;
+      for (int x = l; x < nq; x += L) cp_async16(s + M::VEC + (size_t)r * DP + 4 * x, src + 4 * x);
     }
-    if (tid < nt) cp_async4(&zs[buf][tid], p.zb + (size_t)(tb + tid) * p.ld_b + h);
+    float* num = s + M::VEC + M::TOTAL;
+    for (int x = tid; x < TT * 2; x += DL_THREADS) {
+      if (x < nt * 2) cp_async16(num + 4 * x, p.num + ((size_t)(tb + x / 2) * p.H + h) * 8 + 4 * (x & 1));
+      else *reinterpret_cast<float4*>(num + 4 * x) = make_float4(0.f, 0.f, 0.f, 0.f);        // no token: beta 0, nothing is written
+    }
+    float* val = num + M::NUM;
+    for (int x = tid; x < nt * COLS; x += DL_THREADS) {
+      const int tt = x / COLS, c = x % COLS;
+      if (c < cols_here) cp_async4(val + x, p.qkv + (size_t)(tb + tt) * p.ld + off_v + c);
+    }
     asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  auto reduce = [&](float v) {
-#pragma unroll
-    for (int o = L / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
   };
 
   if (t0 < t1) fetch(0, t0);
@@ -152,95 +207,205 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(const DeltaArgs 
   for (int tb = t0; tb < t1; tb += TT, buf ^= 1) {
     const int nt = min(TT, t1 - tb);
     asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                  // this group has arrived, and everyone is done with the other buffer
+    __syncthreads();                  // these chunks have arrived, and everyone is done with the other buffer
     if (tb + TT < t1) fetch(buf ^ 1, tb + TT);
-    const float my_beta = lane < nt ? 1.0f / (1.0f + expf(-zs[buf][lane])) : 0.f;
-    if constexpr (RAW) {              // one token as the projections and the convolution gave it
-      const float rate = -expf(p.a_log[h]);
-      for (int i = tid; i < nt * p.d; i += DL_THREADS) {
-        const int tt = i / p.d, x = i - tt * p.d;
-        gs[buf][tt][x] = expf(rate * softplus_f(gs[buf][tt][x] + p.dt_bias[(size_t)h * p.d + x]));
-      }
-      __syncthreads();
-    }
-    auto token = [&](int tt) {
-      float4 k[NQ], q[NQ], g[NQ];
+    const float* s = sm + buf * M::BUF;
+#pragma unroll 1
+    for (int ch = 0; ch < NC && ch * DL_CHUNK < nt; ++ch) {
+      const float* vec = s + (size_t)ch * DL_CHUNK * 3 * DP;
+      const float* num = s + M::VEC + M::TOTAL + ch * DL_CHUNK * 8;
+      const float* val = s + M::VEC + M::TOTAL + M::NUM + ch * DL_CHUNK * COLS;
+      const float* at = vec + 4 * l;                 // this lane's first quad of the chunk's vectors; the next lies 4 * L further on
+      auto load = [&](float4 (&kk)[DL_CHUNK], float4 (&qq)[DL_CHUNK], int j) {
 #pragma unroll
-      for (int j = 0; j < NQ; ++j) {
-        k[j] = *reinterpret_cast<const float4*>(&ks[buf][tt][4 * (l + L * j)]);
-        q[j] = *reinterpret_cast<const float4*>(&qs[buf][tt][4 * (l + L * j)]);
-        g[j] = *reinterpret_cast<const float4*>(&gs[buf][tt][4 * (l + L * j)]);
-      }
-      if constexpr (RAW) {
-        float sk = 0.f, sq = 0.f;
-#pragma unroll
-        for (int j = 0; j < NQ; ++j) {
-          sk = fmaf(k[j].x, k[j].x, fmaf(k[j].y, k[j].y, fmaf(k[j].z, k[j].z, fmaf(k[j].w, k[j].w, sk))));
-          sq = fmaf(q[j].x, q[j].x, fmaf(q[j].y, q[j].y, fmaf(q[j].z, q[j].z, fmaf(q[j].w, q[j].w, sq))));
+        for (int i = 0; i < DL_CHUNK; ++i) {
+          kk[i] = *reinterpret_cast<const float4*>(at + (3 * i) * DP + 4 * L * j);
+          qq[i] = *reinterpret_cast<const float4*>(at + (3 * i + 1) * DP + 4 * L * j);
         }
-        const float mk = 1.0f / sqrtf(reduce(sk) + DL_UNIT_EPS), mq = p.q_scale / sqrtf(reduce(sq) + DL_UNIT_EPS);
+      };
+      auto load_write = [&](float4 (&kk)[DL_CHUNK], float4& T, int j) {
 #pragma unroll
-        for (int j = 0; j < NQ; ++j) {
-          k[j].x *= mk, k[j].y *= mk, k[j].z *= mk, k[j].w *= mk;
-          q[j].x *= mq, q[j].y *= mq, q[j].z *= mq, q[j].w *= mq;
+        for (int i = 0; i < DL_CHUNK; ++i) kk[i] = *reinterpret_cast<const float4*>(at + (3 * i + 2) * DP + 4 * L * j);
+        T = *reinterpret_cast<const float4*>(s + M::VEC + (size_t)ch * DP + 4 * l + 4 * L * j);
+      };
+      // reads and outputs over S0: the next quad's vectors are under way while one quad is worked on, eight sums at a time
+      float4 kk[2][DL_CHUNK], qq[2][DL_CHUNK], T[2];
+      float r[X][DL_CHUNK], y[X][DL_CHUNK], w[X][DL_CHUNK];
+      load(kk[0], qq[0], 0);
+      float4 A[DL_CHUNK];                            // A_i0 A_i1 A_i2 beta_i
+#pragma unroll
+      for (int i = 0; i < DL_CHUNK; ++i) {
+        A[i] = *reinterpret_cast<const float4*>(num + 8 * i);
+#pragma unroll
+        for (int x = 0; x < X; ++x) {
+          r[x][i] = y[x][i] = 0.f;
+          w[x][i] = val[i * COLS + grp + x * GROUPS];
         }
       }
-      float4 r = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
       for (int j = 0; j < NQ; ++j) {
-        r.x = fmaf(S[j].x, g[j].x * k[j].x, r.x);
-        r.y = fmaf(S[j].y, g[j].y * k[j].y, r.y);
-        r.z = fmaf(S[j].z, g[j].z * k[j].z, r.z);
-        r.w = fmaf(S[j].w, g[j].w * k[j].w, r.w);
+        if (j + 1 < NQ) load(kk[(j + 1) & 1], qq[(j + 1) & 1], j + 1);
+#pragma unroll
+        for (int x = 0; x < X; ++x)
+#pragma unroll
+          for (int i = 0; i < DL_CHUNK; ++i) {
+            r[x][i] = dot4(S[x][j], kk[j & 1][i], r[x][i]);
+            y[x][i] = dot4(S[x][j], qq[j & 1][i], y[x][i]);
+          }
       }
-      const float read = reduce((r.x + r.y) + (r.z + r.w));
-      const float u = __shfl_sync(0xffffffffu, my_beta, tt) * ((col ? vs[buf][tt][wc] : 0.f) - read);
-      float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+      load_write(kk[0], T[0], 0);                    // for the state's update, under way during the exchanges
+#pragma unroll
+      for (int o = L / 2; o > 0; o >>= 1)
+#pragma unroll
+        for (int x = 0; x < X; ++x)
+#pragma unroll
+          for (int i = 0; i < DL_CHUNK; ++i) r[x][i] += __shfl_xor_sync(0xffffffffu, r[x][i], o);
+      // the outputs: the four sums of a column need not end in every lane, so two exchanges leave a lane one token's
+      float a[X];
+#pragma unroll
+      for (int x = 0; x < X; ++x) {
+        const bool hi = l & (L / 2), lo = l & (L / 4);
+        const float a0 = (hi ? y[x][2] : y[x][0]) + __shfl_xor_sync(0xffffffffu, hi ? y[x][0] : y[x][2], L / 2);
+        const float a1 = (hi ? y[x][3] : y[x][1]) + __shfl_xor_sync(0xffffffffu, hi ? y[x][1] : y[x][3], L / 2);
+        a[x] = (lo ? a1 : a0) + __shfl_xor_sync(0xffffffffu, lo ? a0 : a1, L / 4);
+#pragma unroll
+        for (int o = L / 8; o > 0; o >>= 1) a[x] += __shfl_xor_sync(0xffffffffu, a[x], o);
+      }
+      float u[X][DL_CHUNK];
+#pragma unroll
+      for (int i = 0; i < DL_CHUNK; ++i)
+#pragma unroll
+        for (int x = 0; x < X; ++x) {
+          float z = w[x][i] - r[x][i];
+          if (i > 0) z = fmaf(-A[i].x, u[x][0], z);
+          if (i > 1) z = fmaf(-A[i].y, u[x][1], z);
+          if (i > 2) z = fmaf(-A[i].z, u[x][2], z);
+          u[x][i] = A[i].w * z;
+        }
 #pragma unroll
       for (int j = 0; j < NQ; ++j) {
-        S[j].x = fmaf(k[j].x, u, g[j].x * S[j].x);
-        S[j].y = fmaf(k[j].y, u, g[j].y * S[j].y);
-        S[j].z = fmaf(k[j].z, u, g[j].z * S[j].z);
-        S[j].w = fmaf(k[j].w, u, g[j].w * S[j].w);
-        y.x = fmaf(S[j].x, q[j].x, y.x);
-        y.y = fmaf(S[j].y, q[j].y, y.y);
-        y.z = fmaf(S[j].z, q[j].z, y.z);
-        y.w = fmaf(S[j].w, q[j].w, y.w);
-      }
-      const float out = reduce((y.x + y.y) + (y.z + y.w));
-      if (l == 0) os[tt][wc] = out;
-    };
-    if (nt == TT) {
+        if (j + 1 < NQ) load_write(kk[(j + 1) & 1], T[(j + 1) & 1], j + 1);
+        const float4 t4 = T[j & 1];
 #pragma unroll
-      for (int tt = 0; tt < TT; ++tt) token(tt);
-    } else {
-      for (int tt = 0; tt < nt; ++tt) token(tt);
+        for (int x = 0; x < X; ++x) S[x][j].x *= t4.x, S[x][j].y *= t4.y, S[x][j].z *= t4.z, S[x][j].w *= t4.w;
+#pragma unroll
+        for (int i = 0; i < DL_CHUNK; ++i)
+#pragma unroll
+          for (int x = 0; x < X; ++x) {
+            S[x][j].x = fmaf(kk[j & 1][i].x, u[x][i], S[x][j].x);
+            S[x][j].y = fmaf(kk[j & 1][i].y, u[x][i], S[x][j].y);
+            S[x][j].z = fmaf(kk[j & 1][i].z, u[x][i], S[x][j].z);
+            S[x][j].w = fmaf(kk[j & 1][i].w, u[x][i], S[x][j].w);
+          }
+      }
+      const int mine = l / (L / 4);                  // the token whose output this lane ended with
+      const float4 B = *reinterpret_cast<const float4*>(num + 8 * mine + 4);
+#pragma unroll
+      for (int x = 0; x < X; ++x) {
+        a[x] = fmaf(B.x, u[x][0], fmaf(B.y, u[x][1], fmaf(B.z, u[x][2], fmaf(B.w, u[x][3], a[x]))));
+        if (l % (L / 4) == 0) os[(ch * DL_CHUNK + mine) * COLS + grp + x * GROUPS] = a[x];
+      }
     }
     __syncthreads();
-    for (int i = tid; i < nt * cols_here; i += DL_THREADS) {
-      const int tt = i / cols_here, x = i - tt * cols_here;
-      p.o[(size_t)(tb + tt) * p.H * p.e + (size_t)h * p.e + c0 + x] = os[tt][x];
+    for (int x = tid; x < nt * COLS; x += DL_THREADS) {
+      const int tt = x / COLS, c = x % COLS;
+      if (c < cols_here) p.o[(size_t)(tb + tt) * p.H * p.e + (size_t)h * p.e + c0 + c] = os[x];
     }
   }
   zk_let_next_start();      // only now: a block that waits for this long kernel would hold an SM's issue slots against it
-  if (col) {
+#pragma unroll
+  for (int x = 0; x < X; ++x) {
+    const int c = c0 + grp + x * GROUPS;
 #pragma unroll
     for (int j = 0; j < NQ; ++j) {
       const int i = 4 * (l + L * j);
-      if (i < p.d4) *reinterpret_cast<float4*>(st + i) = S[j];
+      if (c < p.e && i < p.d4) *reinterpret_cast<float4*>(st + (size_t)c * p.d4 + i) = S[x][j];
     }
   }
+}
+
+// One token per sequence: row b is sequence b's.  Block (sequence, head, columns); its threads make the decays once, every column's
+// lanes read them, and the raw q and k, from shared memory.
+template <int L, int CH>
+__global__ void __launch_bounds__(DL_THREADS) delta_single_kernel(const DeltaArgs p) {
+  constexpr int DP = L * CH, NQ = CH / 4, COLS = DL_THREADS / L;
+  __shared__ __align__(16) float ks[DP], qs[DP], gs[DP];
+  const int tid = threadIdx.x, l = tid % L, c = blockIdx.z * COLS + tid / L;
+  const int b = blockIdx.x, h = blockIdx.y, hk = h / (p.H / p.G);
+  const bool col = c < p.e;
+  zk_let_next_start();
+  zk_wait_prior();
+  float* st = p.state + (size_t)p.seq_slot[b] * p.state_stride + ((size_t)h * p.e + (col ? c : 0)) * p.d4;
+  float4 S[NQ];
+#pragma unroll
+  for (int j = 0; j < NQ; ++j) {
+    const int i = 4 * (l + L * j);
+    S[j] = col && i < p.d4 ? *reinterpret_cast<const float4*>(st + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const float* row = p.qkv + (size_t)b * p.ld;
+  const float v = col ? row[2 * p.G * p.d + h * p.e + c] : 0.f;
+  const float beta = 1.0f / (1.0f + expf(-p.zb[(size_t)b * p.ld_b + h]));
+  const float rate = -expf(p.a_log[h]);
+  for (int i = tid; i < DP; i += DL_THREADS) {
+    const bool ok = i < p.d;
+    qs[i] = ok ? row[hk * p.d + i] : 0.f;
+    ks[i] = ok ? row[(p.G + hk) * p.d + i] : 0.f;
+    gs[i] = ok ? expf(rate * softplus_f(p.a[(size_t)b * p.ld_a + (size_t)h * p.d + i] + p.dt_bias[(size_t)h * p.d + i])) : 0.f;
+  }
+  __syncthreads();
+  auto reduce = [&](float x) {
+#pragma unroll
+    for (int o = L / 2; o > 0; o >>= 1) x += __shfl_xor_sync(0xffffffffu, x, o);
+    return x;
+  };
+  float sk = 0.f, sq = 0.f, r = 0.f;
+#pragma unroll
+  for (int j = 0; j < NQ; ++j) {
+    const float4 k = *reinterpret_cast<const float4*>(ks + 4 * (l + L * j)), q = *reinterpret_cast<const float4*>(qs + 4 * (l + L * j));
+    const float4 g = *reinterpret_cast<const float4*>(gs + 4 * (l + L * j));
+    sk = dot4(k, k, sk);
+    sq = dot4(q, q, sq);
+    S[j].x *= g.x, S[j].y *= g.y, S[j].z *= g.z, S[j].w *= g.w;
+    r = dot4(S[j], k, r);
+  }
+  const float mk = 1.0f / sqrtf(reduce(sk) + DL_UNIT_EPS), mq = p.q_scale / sqrtf(reduce(sq) + DL_UNIT_EPS);
+  const float uk = beta * (v - mk * reduce(r)) * mk;      // times the raw key
+  float y = 0.f;
+#pragma unroll
+  for (int j = 0; j < NQ; ++j) {
+    const float4 k = *reinterpret_cast<const float4*>(ks + 4 * (l + L * j)), q = *reinterpret_cast<const float4*>(qs + 4 * (l + L * j));
+    S[j].x = fmaf(k.x, uk, S[j].x);
+    S[j].y = fmaf(k.y, uk, S[j].y);
+    S[j].z = fmaf(k.z, uk, S[j].z);
+    S[j].w = fmaf(k.w, uk, S[j].w);
+    y = dot4(S[j], q, y);
+    const int i = 4 * (l + L * j);
+    if (col && i < p.d4) *reinterpret_cast<float4*>(st + i) = S[j];
+  }
+  y = mq * reduce(y);
+  if (col && l == 0) p.o[(size_t)b * p.H * p.e + (size_t)h * p.e + c] = y;
 }
 
 namespace {
 
-template <int L, int CH, int TT>
-int launch_scan(const DeltaArgs& p, int n_seqs, int raw, cudaStream_t stream) {
-  constexpr int COLS = DL_THREADS / L;
-  const dim3 grid(n_seqs, p.H, (p.e + COLS - 1) / COLS);
-  if (raw) return zk_launch_dependent(delta_scan_kernel<L, CH, 1, true>, grid, dim3(DL_THREADS), 0, stream, p);
-  return zk_launch_dependent(delta_scan_kernel<L, CH, TT, false>, grid, dim3(DL_THREADS), 0, stream, p);
+template <int L, int CH, int X, int NC>
+int launch_chunks(const DeltaArgs& p, int n_seqs, cudaStream_t stream) {
+  using M = ChunkSmem<L, CH, X, NC>;
+  auto kern = delta_chunk_kernel<L, CH, X, NC>;
+  if (M::BYTES > 48 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)M::BYTES);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return zk_launch_dependent(kern, dim3(n_seqs, p.H, (p.e + M::COLS - 1) / M::COLS), dim3(DL_THREADS), M::BYTES, stream, p);
 }
+
+template <int L, int CH>
+int launch_single(const DeltaArgs& p, int n_seqs, cudaStream_t stream) {
+  constexpr int COLS = DL_THREADS / L;
+  return zk_launch_dependent(delta_single_kernel<L, CH>, dim3(n_seqs, p.H, (p.e + COLS - 1) / COLS), dim3(DL_THREADS), 0, stream, p);
+}
+
+int forced_layout = 0;      // lanes per column of the chunk kernel at d of 65..128 (8 or 16); 0 = the library chooses
 
 }  // namespace
 
@@ -251,34 +416,59 @@ int zk_delta_max_dim() { return DL_MAX_D; }
 // Floats of state a slot needs: [H, e, d rounded up to a multiple of 4].
 int zk_delta_state_floats(int H, int d, int e) { return H * e * ((d + 3) / 4 * 4); }
 
+// Floats of scratch a prompt step of n tokens and n_seqs sequences needs.
+long long zk_delta_scratch_floats(int n, int n_seqs, int H, int d) {
+  const long long d4 = (d + 3) / 4 * 4;
+  return (long long)n * H * (3 * d4 + 8) + (long long)(n / DL_CHUNK + n_seqs) * H * d4;
+}
+
+// For measurements: lanes per column (8 or 16) of prompt steps with 65..128 key channels; 0 gives the choice back.
+int zk_delta_force_lanes(int lanes) {
+  if (lanes != 0 && lanes != 8 && lanes != 16) return ZK_EINVAL;
+  forced_layout = lanes;
+  return 0;
+}
+
 // qkv float32 [n, >= 2*G*d + H*e], rows `ld` apart, [q | k | v | ...] behind their convolutions; a float32 [n, >= H*d], rows ld_a
 // apart: the raw decays; zb float32 [n, >= H], rows ld_b apart: beta's logits; a_log [H], dt_bias [H*d].  state: 16-byte aligned slots
-// of zk_delta_state_floats, `state_stride` floats apart (a multiple of 4).  o float32 [n, H*e].  single != 0: every sequence has one
-// token, and qkv and a are left as they are; otherwise q, k and a are REPLACED by unit vectors and decays first.
-int zk_delta_scan(float* qkv, int ld, float* a, int ld_a, const float* zb, int ld_b, const float* a_log, const float* dt_bias,
-                  float* state, long long state_stride, float* o, const int* cu_q, const int* seq_slot, int n, int n_seqs, int H,
-                  int G, int d, int e, float q_scale, int single, cudaStream_t stream) {
+// of zk_delta_state_floats, `state_stride` floats apart (a multiple of 4).  o float32 [n, H*e].  scratch: 16-byte aligned, of
+// zk_delta_scratch_floats, or null: then every sequence has one token (n = n_seqs, row b sequence b's).
+int zk_delta_scan(const float* qkv, int ld, const float* a, int ld_a, const float* zb, int ld_b, const float* a_log,
+                  const float* dt_bias, float* state, long long state_stride, float* o, const int* cu_q, const int* seq_slot,
+                  const int* tok_seq, int n, int n_seqs, int H, int G, int d, int e, float q_scale, float* scratch,
+                  cudaStream_t stream) {
   if (n_seqs <= 0 || n <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || d <= 0 || e <= 0 || d > DL_MAX_D) return ZK_EINVAL;
   if (ld < 2 * G * d + H * e || ld_a < H * d || ld_b < H || !a_log || !dt_bias || !zb) return ZK_EINVAL;
-  if (state_stride % 4 || (uintptr_t)state % 16 || (single && n != n_seqs)) return ZK_EINVAL;
-  if (!single) {
-    const long long items = (long long)n * (2 * G + H);
-    const int rc = zk_launch_dependent(delta_prepare_kernel, dim3((unsigned)((items + 7) / 8)), dim3(256), 0, stream, qkv, ld, a, ld_a,
-                                       a_log, dt_bias, items, G, H, d, q_scale);
-    if (rc != 0) return rc;
-  }
+  if (state_stride % 4 || (uintptr_t)state % 16 || (uintptr_t)scratch % 16 || (!scratch && n != n_seqs)) return ZK_EINVAL;
   DeltaArgs p{};
-  p.qkv = qkv; p.g = a; p.zb = zb; p.a_log = a_log; p.dt_bias = dt_bias;
-  p.state = state; p.o = o; p.cu_q = cu_q; p.seq_slot = seq_slot; p.state_stride = state_stride;
-  p.ld = ld; p.ld_g = ld_a; p.ld_b = ld_b; p.H = H; p.G = G; p.d = d; p.e = e; p.d4 = (d + 3) / 4 * 4;
-  p.vec = d % 4 == 0 && ld % 4 == 0 && ld_a % 4 == 0 && ((uintptr_t)qkv | (uintptr_t)a) % 16 == 0;
+  p.qkv = qkv; p.a = a; p.zb = zb; p.a_log = a_log; p.dt_bias = dt_bias;
+  p.state = state; p.o = o; p.cu_q = cu_q; p.seq_slot = seq_slot; p.tok_seq = tok_seq; p.state_stride = state_stride;
+  p.ld = ld; p.ld_a = ld_a; p.ld_b = ld_b; p.H = H; p.G = G; p.d = d; p.e = e; p.d4 = (d + 3) / 4 * 4;
   p.q_scale = q_scale;
-  if (d <= 32) return launch_scan<8, 4, 8>(p, n_seqs, single, stream);
-  if (d <= 64) return launch_scan<8, 8, 8>(p, n_seqs, single, stream);
-  if (d <= 128) return launch_scan<8, 16, 8>(p, n_seqs, single, stream);
-  if (d <= 256) return launch_scan<16, 16, 4>(p, n_seqs, single, stream);
-  return launch_scan<32, 16, 2>(p, n_seqs, single, stream);
+  if (!scratch) {
+    if (d <= 32) return launch_single<8, 4>(p, n_seqs, stream);
+    if (d <= 64) return launch_single<8, 8>(p, n_seqs, stream);
+    if (d <= 128) return launch_single<8, 16>(p, n_seqs, stream);
+    if (d <= 256) return launch_single<16, 16>(p, n_seqs, stream);
+    return launch_single<32, 16>(p, n_seqs, stream);
+  }
+  p.vec = scratch;
+  p.num = p.vec + (size_t)n * H * 3 * p.d4;
+  p.total = p.num + (size_t)n * H * 8;
+  const dim3 grid(n, (H + 3) / 4), block(128);
+  int rc;
+  if (d <= 32) rc = zk_launch_dependent(delta_chunk_prepare_kernel<1>, grid, block, 0, stream, p);
+  else if (d <= 64) rc = zk_launch_dependent(delta_chunk_prepare_kernel<2>, grid, block, 0, stream, p);
+  else if (d <= 128) rc = zk_launch_dependent(delta_chunk_prepare_kernel<4>, grid, block, 0, stream, p);
+  else if (d <= 256) rc = zk_launch_dependent(delta_chunk_prepare_kernel<8>, grid, block, 0, stream, p);
+  else rc = zk_launch_dependent(delta_chunk_prepare_kernel<16>, grid, block, 0, stream, p);
+  if (rc != 0) return rc;
+  if (d <= 32) return launch_chunks<8, 4, 1, 2>(p, n_seqs, stream);
+  if (d <= 64) return launch_chunks<16, 4, 2, 2>(p, n_seqs, stream);
+  if (d <= 128) return forced_layout == 8 ? launch_chunks<8, 16, 1, 2>(p, n_seqs, stream) : launch_chunks<16, 8, 2, 2>(p, n_seqs, stream);
+  if (d <= 256) return launch_chunks<16, 16, 2, 1>(p, n_seqs, stream);
+  return launch_chunks<32, 16, 2, 1>(p, n_seqs, stream);
 }
 
 }  // extern "C"

@@ -631,21 +631,27 @@ __global__ void activation_kernel(const T* __restrict__ in, T* __restrict__ out,
 
 // Float32 rows in the run dtype (the input of a contraction that reads the residual rows as they are).
 template <typename T>
-__global__ void cast_rows_kernel(const float* __restrict__ in, T* __restrict__ out, size_t total) {
+__global__ void cast_rows_kernel(const float* __restrict__ in, T* __restrict__ out, size_t rows, size_t width, size_t ld) {
+  // rows of `width` values, `ld` apart in `in`, packed in `out`
   zk_let_next_start();
   zk_wait_prior();
+  const size_t total = rows * width;
   if constexpr (sizeof(T) == 2) {
-    if (total % 4 == 0 && ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out)) % 16) == 0) {
+    if (width % 4 == 0 && ld % 4 == 0 && ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out)) % 16) == 0) {
+      const size_t w4 = width / 4;
       for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total / 4; i += (size_t)gridDim.x * blockDim.x) {
-        const float4 v = reinterpret_cast<const float4*>(in)[i];
+        const size_t r = rows == 1 ? 0 : i / w4;
+        const float4 v = *reinterpret_cast<const float4*>(in + r * ld + 4 * (i - r * w4));
         __nv_bfloat162 pk[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
         reinterpret_cast<uint2*>(out)[i] = *reinterpret_cast<const uint2*>(pk);
       }
       return;
     }
   }
-  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
-    out[i] = from_f32<T>(in[i]);
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = rows == 1 ? 0 : i / width;
+    out[i] = from_f32<T>(in[r * ld + (i - r * width)]);
+  }
 }
 
 // logits <- cap * tanh(logits / cap), in place, float32.
@@ -1027,13 +1033,15 @@ int zk_activation(const void* in, void* out, long long total, int kind, int dtyp
   return ZK_EINVAL;
 }
 
-int zk_cast_rows(const float* in, void* out, long long total, int dtype, cudaStream_t stream) {
-  if (total <= 0) return 0;
-  const int threads = 256, blocks = grid_for_total((size_t)total, threads);
+// rows of `width` float32 values, `ld` apart, as packed rows of the run dtype.
+int zk_cast_rows(const float* in, void* out, long long rows, long long width, long long ld, int dtype, cudaStream_t stream) {
+  if (rows <= 0 || width <= 0) return 0;
+  if (ld < width) return ZK_EINVAL;
+  const int threads = 256, blocks = grid_for_total((size_t)(rows * width), threads);
   if (dtype == ZK_F32)
-    return zk_launch_dependent(cast_rows_kernel<float>, dim3(blocks), dim3(threads), 0, stream, in, (float*)out, (size_t)total);
+    return zk_launch_dependent(cast_rows_kernel<float>, dim3(blocks), dim3(threads), 0, stream, in, (float*)out, (size_t)rows, (size_t)width, (size_t)ld);
   if (dtype == ZK_BF16)
-    return zk_launch_dependent(cast_rows_kernel<bf16>, dim3(blocks), dim3(threads), 0, stream, in, (bf16*)out, (size_t)total);
+    return zk_launch_dependent(cast_rows_kernel<bf16>, dim3(blocks), dim3(threads), 0, stream, in, (bf16*)out, (size_t)rows, (size_t)width, (size_t)ld);
   return ZK_EINVAL;
 }
 

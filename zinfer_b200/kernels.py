@@ -31,7 +31,7 @@ _SIGNATURES = {
         "zk_rmsnorm_add": "pppiiffp",
         "zk_rmsnorm_pair_add": "pppppiiffp",
         "zk_activation": "ppliip",
-        "zk_cast_rows": "pplip",
+        "zk_cast_rows": "pp" + "llli" + "p",
         "zk_softcap": "plfp",
         "zk_scale": "plfp",
         "zk_weighted_sum": "ppilpp",
@@ -69,7 +69,9 @@ _SIGNATURES = {
     "delta": {
         "zk_delta_max_dim": "",
         "zk_delta_state_floats": "iii",
-        "zk_delta_scan": "pipipipp" + "plppp" + "iiiiii" + "fi" + "p",
+        "zk_delta_scratch_floats": "iiii",
+        "zk_delta_force_lanes": "i",
+        "zk_delta_scan": "pipipipp" + "plpppp" + "iiiiii" + "fp" + "p",
     },
     "seqconv": {
         "zk_seqconv_forward": "ppppppp" + "iiiliii" + "ipi" + "p",
@@ -153,7 +155,7 @@ _SIGNATURES = {
 }
 
 
-_RESTYPES = {"zk_attn_decode_noalloc_bytes": ctypes.c_longlong}
+_RESTYPES = {"zk_attn_decode_noalloc_bytes": ctypes.c_longlong, "zk_delta_scratch_floats": ctypes.c_longlong}
 
 
 class KernelError(RuntimeError):
@@ -336,12 +338,17 @@ def activation(z: torch.Tensor, kind: str, out: Optional[torch.Tensor] = None) -
 
 
 def cast_rows(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
-    """Float32 rows in the run dtype (the rows themselves when that is float32)."""
-    _need(x, "x", torch.float32)
+    """Float32 rows (row stride used) in the run dtype (the rows themselves when that is float32)."""
+    strided = x.dim() == 2 and not x.is_contiguous()
+    _need(x, "x", torch.float32, contiguous=not strided)
+    if strided and x.stride(1) != 1:
+        raise KernelError("cast_rows: the values of a row must lie side by side")
     if dtype == torch.float32:
         return x
+    rows, width, ld = (x.shape[0], x.shape[1], x.stride(0)) if strided else (1, x.numel(), x.numel())
     y = torch.empty(x.shape, dtype=dtype, device=x.device)
-    _check(_fn("elementwise", "zk_cast_rows")(_ptr(x), _ptr(y), x.numel(), dtype_code(dtype), _stream()), "cast_rows")
+    _check(_fn("elementwise", "zk_cast_rows")(_ptr(x), _ptr(y), rows, width, ld, dtype_code(dtype), _stream()),
+           "cast_rows")
     return y
 
 
@@ -560,15 +567,15 @@ def delta_state_floats(n_heads: int, dim: int, value_dim: int) -> int:
 
 
 def delta_scan(qkv: torch.Tensor, a: torch.Tensor, z_beta: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
-               state: torch.Tensor, cu_q, seq_slot, n_seqs: int, n_heads: int, groups: int, dim: int, value_dim: int,
+               state: torch.Tensor, tok_seq, cu_q, seq_slot, n_seqs: int, n_heads: int, groups: int, dim: int, value_dim: int,
                single_token: bool = False) -> torch.Tensor:
     """Gated delta rule per head over each sequence's tokens, from the state the step before left to the state this one leaves:
     S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, with g = exp(-exp(a_log) softplus(a + dt_bias)) per head and key
     channel, beta = sigmoid(z_beta), q and k unit vectors (x / sqrt(sum x^2 + 1e-6)), q also times d^-1/2.  qkv float32
     [n, >= 2*G*d + H*e], a row [q | k | v | ..], q and k shared by the H / G heads of a group; a float32 [n, >= H*d]; z_beta float32
     [n, H] (row strides used); a_log [H], dt_bias [H*d]; state float32 [slots, delta_state_floats], 16-byte aligned rows, ordered
-    [H, e, d up to a multiple of 4].  `single_token`: every sequence brings one token; otherwise q, k and a are overwritten by the unit
-    vectors and decays.  Returns o float32 [n, H*e]."""
+    [H, e, d up to a multiple of 4].  `single_token`: every sequence brings one token (one kernel); otherwise chunks of four tokens
+    are prepared by a kernel of their own.  Returns o float32 [n, H*e]."""
     H, G, d, e = n_heads, groups, dim, value_dim
     _need(qkv, "qkv", torch.float32, (None, None), contiguous=False)
     n = qkv.shape[0]
@@ -583,13 +590,22 @@ def delta_scan(qkv: torch.Tensor, a: torch.Tensor, z_beta: torch.Tensor, a_log: 
     _need(state, "state", torch.float32, contiguous=False)
     if state.dim() != 2 or state.shape[1] != delta_state_floats(H, d, e) or state.stride(1) != 1:
         raise KernelError(f"delta_scan: state {tuple(state.shape)} must hold {delta_state_floats(H, d, e)} values per slot")
-    for t, nm in ((cu_q, "cu_q"), (seq_slot, "seq_slot")):
+    for t, nm in ((cu_q, "cu_q"), (seq_slot, "seq_slot"), (tok_seq, "tok_seq")):
         _need(t, nm, torch.int32)
     o = torch.empty((n, H * e), dtype=torch.float32, device=qkv.device)
+    scratch = None
+    if not single_token:
+        scratch = torch.empty(_fn("delta", "zk_delta_scratch_floats")(n, n_seqs, H, d), dtype=torch.float32, device=qkv.device)
     _check(_fn("delta", "zk_delta_scan")(_ptr(qkv), qkv.stride(0), _ptr(a), a.stride(0), _ptr(z_beta), z_beta.stride(0), _ptr(a_log),
-                                         _ptr(dt_bias), _ptr(state), state.stride(0), _ptr(o), _ptr(cu_q), _ptr(seq_slot), n, n_seqs, H, G,
-                                         d, e, float(d) ** -0.5, 1 if single_token else 0, _stream()), "delta_scan")
+                                         _ptr(dt_bias), _ptr(state), state.stride(0), _ptr(o), _ptr(cu_q), _ptr(seq_slot), _ptr(tok_seq),
+                                         n, n_seqs, H, G, d, e, float(d) ** -0.5, _ptr(scratch), _stream()), "delta_scan")
     return o
+
+
+def delta_force_lanes(lanes: int) -> None:
+    """For measurements and tests: lanes per column of the state (8 or 16) in prompt steps with 65..128 key channels; 0 = the library
+    chooses."""
+    _check(_fn("delta", "zk_delta_force_lanes")(int(lanes)), "delta_force_lanes")
 
 
 # ------------------------------------------------------------------------------- convolution over time on a mixer's input
@@ -859,8 +875,10 @@ def fill_normal(out: torch.Tensor, seed: int, mean: float = 0.0, std: float = 1.
 def gemm_simt(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, out_dtype=None,
               accumulate: bool = False, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out (+)= a @ w.T (+ bias) with float32 FMA on the CUDA cores.  a [M, K], w [N, K] share a
-    dtype; out is that dtype or float32; accumulate needs a float32 or same-dtype `out`."""
-    _need(a, "a", (torch.float32, torch.bfloat16), (None, None))
+    dtype; out is that dtype or float32; accumulate needs a float32 or same-dtype `out`.  Rows of a may lie in wider ones."""
+    _need(a, "a", (torch.float32, torch.bfloat16), (None, None), contiguous=False)
+    if a.stride(1) != 1:
+        raise KernelError("gemm: the values of a row must lie side by side")
     _need(w, "w", a.dtype, (None, a.shape[1]))
     M, K = a.shape
     N = w.shape[0]

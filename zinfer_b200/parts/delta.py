@@ -14,8 +14,8 @@ Each head's o_t is divided by its root mean square, multiplied by one weight vec
 sigmoid(W_g2 W_g1 x); the concatenated heads are projected by W_o.  The two inner widths (rows of W_a1 and W_g1) are the
 tensors' own.
 
-q, k, v and beta's logits are one contraction with a float32 result, the two low-rank maps are one contraction into both inner
-widths and one block-diagonal contraction out of them (float32 result).  Convolution, unit vectors, decays, beta, state, sums,
+q, k, v, both inner widths of the low-rank maps and beta's logits are one contraction with a float32 result; one block-diagonal
+contraction (float32 result) leads out of both inner widths.  Convolution, unit vectors, decays, beta, state, sums,
 norm and gate are float32 in both run dtypes (`kernels.seqconv`, `kernels.delta_scan`, `kernels.unit_norm_gate`).  The call's
 per-sequence state holds the convolution's last K - 1 inputs followed by the matrices.  Prompt steps and single-token steps run
 the same recurrence kernel from the state the step before left."""
@@ -25,9 +25,9 @@ import torch
 
 from .. import kernels
 from .base import ANY_SIZE, MIXERS, Mixer, StateRequest, WeightSpec
-from .linear import as_tensor, linear, pad_rows
+from .linear import linear, pad_rows
 
-LOW_RANK_ALIGN = 64      # the inner widths together, brought up to whole contraction steps with zeros
+LOW_RANK_ALIGN = 8       # the inner widths together, brought up to what the tensor-core contractions take with zeros
 
 
 class GatedDelta(Mixer):
@@ -49,7 +49,7 @@ class GatedDelta(Mixer):
         self.a_log_name, self.dt_bias_name = a_log_name, dt_bias_name
         self.a1_name, self.a2_name, self.g1_name, self.g2_name = a1_name, a2_name, g1_name, g2_name
         self.norm_name, self.out_name = norm_name, out_name
-        self.w_in = self.w_low = self.w_high = self.w_out = self.conv = self.a_log = self.dt_bias = self.norm = None
+        self.w_in = self.w_high = self.w_out = self.conv = self.a_log = self.dt_bias = self.norm = None
 
     @property
     def key_dim(self):
@@ -92,10 +92,11 @@ class GatedDelta(Mixer):
         for inner, outer, name in ((a1, a2, self.a1_name), (g1, g2, self.g1_name)):
             if inner.shape[0] != outer.shape[1]:
                 raise ValueError(f"tensor '{name}' has {inner.shape[0]} rows, the matrix behind it {outer.shape[1]} columns")
-        self.w_in = pad_rows(torch.cat([weights[n] for n in self.proj_names], dim=0).contiguous())
         ra, rg = a1.shape[0], g1.shape[0]
         r = -(-(ra + rg) // LOW_RANK_ALIGN) * LOW_RANK_ALIGN
-        self.w_low = torch.cat([a1, g1, a1.new_zeros((r - ra - rg, self.hidden))], dim=0).contiguous()
+        q, k, v, beta = (weights[n] for n in self.proj_names)
+        self.rank = r
+        self.w_in = pad_rows(torch.cat([q, k, v, a1, g1, a1.new_zeros((r - ra - rg, self.hidden)), beta], dim=0).contiguous())
         self.w_high = a2.new_zeros((self.decay_dim + self.out_dim, r))
         self.w_high[:self.decay_dim, :ra] = a2
         self.w_high[self.decay_dim:, ra:ra + rg] = g2
@@ -116,14 +117,14 @@ class GatedDelta(Mixer):
 
     def forward(self, ctx, call, xn, out, accumulate):
         H, G, d, e, ch = self.n_heads, self.n_kv, self.dim, self.value_dim, self.channels
-        x = as_tensor(xn)
-        p = linear(x, self.w_in, out_dtype=torch.float32)                    # [q | k | v | beta (| padding)]
-        ag = linear(linear(x, self.w_low), self.w_high, out_dtype=torch.float32)      # [decays | gate (| padding)]
+        r = self.rank
+        p = linear(xn, self.w_in, out_dtype=torch.float32)                   # [q | k | v | inner widths | beta (| padding)]
+        ag = linear(kernels.cast_rows(p[:, ch:ch + r], ctx.dtype), self.w_high, out_dtype=torch.float32)   # [decays | gate (| padding)]
         conv = call.state[:, :(self.taps - 1) * ch].unflatten(1, (self.taps - 1, ch))
         rec = call.state[:, self.conv_floats:self.conv_floats + kernels.delta_state_floats(H, d, e)]
         qkv = kernels.seqconv(p[:, :ch], conv, self.conv, ctx.tok_seq, ctx.cu_q, ctx.seq_slot, ctx.n_seqs, torch.float32,
                               residual=False, single_token=ctx.is_decode, silu=True)
-        o = kernels.delta_scan(qkv, ag, p[:, ch:ch + H], self.a_log, self.dt_bias, rec, ctx.cu_q, ctx.seq_slot, ctx.n_seqs, H, G, d, e,
+        o = kernels.delta_scan(qkv, ag, p[:, ch + r:ch + r + H], self.a_log, self.dt_bias, rec, ctx.tok_seq, ctx.cu_q, ctx.seq_slot, ctx.n_seqs, H, G, d, e,
                                single_token=ctx.is_decode)
         on = kernels.unit_norm_gate(o, ag[:, self.decay_dim:], H, self.eps, ctx.dtype, weight=self.norm, sigmoid=True)
         linear(on, self.w_out, out=out, accumulate=accumulate)
