@@ -107,7 +107,7 @@ def make_weights(cfg: dict, seed: int, ranks=(8, 8)) -> dict[str, np.ndarray]:
         elif name == "embed":
             W[name] = bf16_round(rng.normal(0, 1.0, shape))
         elif name.endswith((".router", ".mix.i", ".mix.f")):
-            W[name] = bf16_round(rng.normal(0, 3.0 * shape[-1] ** -0.5, shape))
+            W[name] = bf16_round(rng.normal(0, (3.0 if name.endswith(".router") else 1.5) * shape[-1] ** -0.5, shape))
         else:
             W[name] = bf16_round(rng.normal(0, shape[-1] ** -0.5, shape))
     return W

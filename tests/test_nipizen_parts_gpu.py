@@ -371,7 +371,9 @@ def test_mlstm_keeps_the_first_token_for_hundreds_of_steps(k, dtype, prompt):
     other = x.clone()
     other[0, 1:] = rnd((D - 1,), 42, dtype)
     assert np.abs(ref[-1] - plain_mem(other, t, H, d, e, cap)[-1]).max() > 0.1 * np.abs(ref).max()
-    close(run_mixer(k, make_mem(D, H, d, e, cap, t, dtype), dtype, [x], [prompt], page=16)[0], ref, dtype, f"prompt of {prompt}")
+    got = run_mixer(k, make_mem(D, H, d, e, cap, t, dtype), dtype, [x], [prompt], page=16)[0]
+    # where a query all but misses the first key its two products are small differences of larger terms: 1e-4 in 32-bit
+    assert np.abs(f64(got) - ref).max() <= (1e-4 if dtype == torch.float32 else 1.5e-2) * np.abs(ref).max()
 
 
 # ------------------------------------------------------------------------------- the pair

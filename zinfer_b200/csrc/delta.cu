@@ -16,11 +16,12 @@
 // so the four reads and the four outputs of a chunk are sums over S0 that do not wait for one another, and only the four u, a
 // small triangular system per column, are a chain.  Products of decays are never divided by, so nothing overflows.
 // delta_chunk_prepare_kernel makes the vectors and the numbers A, B once per (chunk, head), with unit vectors, decays and beta on
-// the way; delta_chunk_kernel owns (sequence, head, some columns of S) per block and walks the chunks: a column lies in L
-// neighbouring lanes, CH channels each, in registers; the vectors of the next chunks reach shared memory with cp.async meanwhile.
+// the way, as one contiguous record.  delta_chunk_kernel owns (sequence, head, some columns of S) per block and walks the chunks: a
+// column lies in L neighbouring lanes, CH channels each, in registers; the records of the next chunks arrive in a ring in shared
+// memory, one bulk copy each, counted on an mbarrier.
 //
 // delta_single_kernel is the single-token step: the recurrence as it stands, unit vectors and decays made on the spot.
-#include "common.cuh"
+#include "tcgen05.cuh"
 #include <math.h>
 
 #define DL_THREADS 128
@@ -32,8 +33,9 @@ __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + lo
 
 struct DeltaArgs {
   const float *qkv, *a, *zb, *a_log, *dt_bias;      // as zk_delta_scan takes them
-  float *vec, *total, *num;                         // prompt steps: [n, H, 3, d4], [chunks, H, d4], [n, H, 8]
+  float* rec;                                       // prompt steps: the records of all chunks, [chunks, H, record_floats(DP, e)]
   float *state, *o;
+  int* status;
   const int *cu_q, *seq_slot, *tok_seq;
   long long state_stride;
   int ld, ld_a, ld_b, H, G, d, e, d4;
@@ -43,8 +45,14 @@ struct DeltaArgs {
 // Chunks of all sequences have distinct numbers below n / 4 + n_seqs: that of the chunk of sequence b that starts at row t.
 __device__ __forceinline__ int chunk_number(int t0, int t, int b) { return t0 / DL_CHUNK + (t - t0) / DL_CHUNK + b; }
 
-// One warp per (token that starts a chunk, head); the warps of other tokens end at once.  vec: c_i k_i, c_i q_i, p_3i k_i per token;
-// total: c_3; num, per token i: A_i0 A_i1 A_i2 beta_i B_i0 B_i1 B_i2 B_i3 (zeros where j is too large).  NJ: channels per lane.
+// A record: for each of the four tokens the vectors c_i k_i, c_i q_i, p_3i k_i; then c_3; then, for each token,
+// A_i0 A_i1 A_i2 beta_i B_i0 B_i1 B_i2 B_i3 (zeros where j is too large).  Vectors are padded with zeros to DP channels; a token
+// that the chunk has not (its sequence ends) is all zeros: it writes nothing.  Behind that lie the chunk's values, column by column:
+// [e up to a multiple of 16][4 tokens], of which a block of the chunk kernel takes its own columns.
+__host__ __device__ constexpr int vector_floats(int DP) { return 13 * DP + 8 * DL_CHUNK; }
+__host__ __device__ __forceinline__ int record_floats(int DP, int e) { return vector_floats(DP) + (e + 15) / 16 * 16 * DL_CHUNK; }
+
+// One warp per (token that starts a chunk, head); the warps of other tokens end at once.  NJ: channels per lane, DP = 32 NJ.
 template <int NJ>
 __global__ void __launch_bounds__(128) delta_chunk_prepare_kernel(const DeltaArgs p) {
   zk_wait_prior();      // and no early start of the kernel behind: its few long blocks would crowd onto the SMs that have room first
@@ -87,7 +95,8 @@ __global__ void __launch_bounds__(128) delta_chunk_prepare_kernel(const DeltaArg
   float v[16];
 #pragma unroll
   for (int x = 0; x < 16; ++x) v[x] = 0.f;
-  const size_t vec_row = (size_t)3 * p.d4;
+  constexpr int DP = 32 * NJ;
+  float* rec = p.rec + ((size_t)chunk_number(t0, t, b) * p.H + h) * record_floats(DP, p.e);
 #pragma unroll
   for (int j = 0; j < NJ; ++j) {
     const int c = lane + 32 * j;
@@ -103,14 +112,11 @@ __global__ void __launch_bounds__(128) delta_chunk_prepare_kernel(const DeltaArg
         v[l * l + i] = fmaf(k[l][j], w, v[l * l + i]);
         v[l * l + l + i] = fmaf(q[l][j], w, v[l * l + l + i]);
       }
-      if (i < nt && c < p.d4) {
-        float* dst = p.vec + ((size_t)(t + i) * p.H + h) * vec_row + c;
-        dst[0] = cum * k[i][j];
-        dst[p.d4] = cum * q[i][j];
-        dst[2 * p.d4] = w;
-      }
+      rec[(3 * i) * DP + c] = cum * k[i][j];
+      rec[(3 * i + 1) * DP + c] = cum * q[i][j];
+      rec[(3 * i + 2) * DP + c] = w;
     }
-    if (c < p.d4) p.total[((size_t)chunk_number(t0, t, b) * p.H + h) * p.d4 + c] = cum;
+    rec[12 * DP + c] = cum;
   }
   // sum all sixteen over the lanes: each exchange halves what a lane holds; lanes 2x and 2x + 1 end with number x
 #pragma unroll
@@ -126,96 +132,79 @@ __global__ void __launch_bounds__(128) delta_chunk_prepare_kernel(const DeltaArg
   const int i = lane >> 3, s = lane & 7, j = s < 4 ? s : s - 4;
   const bool is_a = s < 3 && j < i, is_b = s >= 4 && j <= i;
   const float got = __shfl_sync(0xffffffffu, v[0], 2 * (is_a ? i * i + j : (is_b ? i * i + i + j : 0)));
-  if (i < nt) {
-    float out = is_a || is_b ? got : 0.f;
-    if (s == 3) out = 1.0f / (1.0f + expf(-p.zb[(size_t)(t + i) * p.ld_b + h]));
-    p.num[((size_t)(t + i) * p.H + h) * 8 + s] = out;
+  float out = is_a || is_b ? got : 0.f;
+  if (s == 3 && i < nt) out = 1.0f / (1.0f + expf(-p.zb[(size_t)(t + i) * p.ld_b + h]));
+  rec[13 * DP + lane] = out;
+  const float* values = p.qkv + (size_t)t * p.ld + 2 * p.G * p.d + h * p.e;
+  for (int c = lane; c < (p.e + 15) / 16 * 16; c += 32) {
+    float x[DL_CHUNK];
+#pragma unroll
+    for (int i = 0; i < DL_CHUNK; ++i) x[i] = i < nt && c < p.e ? values[(size_t)i * p.ld + c] : 0.f;
+    *reinterpret_cast<float4*>(rec + vector_floats(DP) + 4 * c) = make_float4(x[0], x[1], x[2], x[3]);
   }
 }
 
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async4(void* dst, const void* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+// `bytes` (a multiple of 16, both addresses 16-byte aligned) from global to this block's shared memory, counted on `bar`.
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, unsigned bytes, unsigned long long* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(tc5::smem_u32(dst)),
+               "l"(src), "r"(bytes), "r"(tc5::smem_u32(bar))
+               : "memory");
 }
 __device__ __forceinline__ float dot4(const float4& a, const float4& b, float acc) {
   return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, acc))));
 }
 
-// Shared memory of a block of the chunk kernel: two buffers of NC chunks, and the outputs of one.
-template <int L, int CH, int X, int NC>
-struct ChunkSmem {
-  static constexpr int DP = L * CH, TT = NC * DL_CHUNK, COLS = DL_THREADS / L * X;
-  static constexpr int VEC = TT * 3 * DP, TOTAL = NC * DP, NUM = TT * 8, VAL = TT * COLS;       // floats
-  static constexpr int BUF = VEC + TOTAL + NUM + VAL;
-  static constexpr size_t BYTES = sizeof(float) * (2 * BUF + VAL);
-};
-
-// L lanes per column, CH channels per lane (a multiple of 4, quads l, l + L, ...), X columns per lane, NC chunks staged at once.
-template <int L, int CH, int X, int NC>
-__global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs p) {
-  using M = ChunkSmem<L, CH, X, NC>;
-  constexpr int DP = M::DP, TT = M::TT, NQ = CH / 4, COLS = M::COLS, GROUPS = DL_THREADS / L;
-  extern __shared__ __align__(16) float sm[];
-  float* os = sm + 2 * M::BUF;                       // [TT][COLS]
+// L lanes per column, CH channels per lane (a multiple of 4, quads l, l + L, ...), X neighbouring columns per lane, a ring of ST records.
+template <int L, int CH, int X, int ST>
+__global__ void __launch_bounds__(DL_THREADS, 1) delta_chunk_kernel(const DeltaArgs p) {
+  constexpr int DP = L * CH, NQ = CH / 4, COLS = DL_THREADS / L * X;
+  constexpr int VEC = vector_floats(DP), REC = VEC + COLS * DL_CHUNK;      // what a block takes of a record
+  extern __shared__ __align__(128) float sm[];       // [ST][REC]
+  __shared__ __align__(8) unsigned long long full[ST];
   const int tid = threadIdx.x, l = tid % L, grp = tid / L;
-  const int b = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * COLS;
-  const int cols_here = min(COLS, p.e - c0);
-  for (int i = tid; i < 2 * M::BUF; i += DL_THREADS) sm[i] = 0.f;      // channels and columns that are not there stay zero
+  const int b = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * COLS + grp * X;      // this lane's first column
+  if (tid == 0) {
+    for (int s = 0; s < ST; ++s) tc5::mbar_init(&full[s], 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+  }
   __syncthreads();
   zk_wait_prior();
   const int t0 = p.cu_q[b], t1 = p.cu_q[b + 1];
+  const int n_chunks = (t1 - t0 + DL_CHUNK - 1) / DL_CHUNK;
+  const int rec_floats = record_floats(DP, p.e);
+  const float* records = p.rec + ((size_t)chunk_number(t0, t0, b) * p.H + h) * rec_floats;      // chunk ch: ch * H records further on
+  const size_t rec_step = (size_t)p.H * rec_floats;
+  const int col0 = blockIdx.z * COLS;
+  const unsigned val_bytes = 4u * DL_CHUNK * min(COLS, (p.e + 15) / 16 * 16 - col0);
+  auto fetch = [&](int ch) {
+    unsigned long long* bar = &full[ch % ST];
+    tc5::mbar_expect_tx(bar, VEC * 4 + val_bytes);
+    bulk_load(sm + (size_t)(ch % ST) * REC, records + ch * rec_step, VEC * 4, bar);
+    bulk_load(sm + (size_t)(ch % ST) * REC + VEC, records + ch * rec_step + VEC + col0 * DL_CHUNK, val_bytes, bar);
+  };
+  if (tid == 0)
+    for (int ch = 0; ch < ST && ch < n_chunks; ++ch) fetch(ch);
   float* st = p.state + (size_t)p.seq_slot[b] * p.state_stride + (size_t)h * p.e * p.d4;
   float4 S[X][NQ];
 #pragma unroll
   for (int x = 0; x < X; ++x) {
-    const int c = c0 + grp + x * GROUPS;             // this lane's columns of the block: grp, grp + GROUPS, ...
 #pragma unroll
     for (int j = 0; j < NQ; ++j) {
       const int i = 4 * (l + L * j);
-      S[x][j] = c < p.e && i < p.d4 ? *reinterpret_cast<const float4*>(st + (size_t)c * p.d4 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      S[x][j] = c0 + x < p.e && i < p.d4 ? *reinterpret_cast<const float4*>(st + (size_t)(c0 + x) * p.d4 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
   }
-  const int nq = p.d4 >> 2, off_v = 2 * p.G * p.d + h * p.e + c0;
-  auto fetch = [&](int buf, int tb) {
-    float* s = sm + buf * M::BUF;
-    const int nt = min(TT, t1 - tb);
-    for (int r = grp; r < nt * 3; r += GROUPS) {                       // a group of L lanes copies a vector
-      const float* src = p.vec + ((size_t)(tb + r / 3) * p.H + h) * 3 * p.d4 + (size_t)(r % 3) * p.d4;
-      for (int x = l; x < nq; x += L) cp_async16(s + (size_t)r * DP + 4 * x, src + 4 * x);
-    }
-    for (int r = grp; r * DL_CHUNK < nt; r += GROUPS) {
-      const float* src = p.total + ((size_t)chunk_number(t0, tb + r * DL_CHUNK, b) * p.H + h) * p.d4;
-      for (int x = l; x < nq; x += L) cp_async16(s + M::VEC + (size_t)r * DP + 4 * x, src + 4 * x);
-    }
-    float* num = s + M::VEC + M::TOTAL;
-    for (int x = tid; x < TT * 2; x += DL_THREADS) {
-      if (x < nt * 2) cp_async16(num + 4 * x, p.num + ((size_t)(tb + x / 2) * p.H + h) * 8 + 4 * (x & 1));
-      else *reinterpret_cast<float4*>(num + 4 * x) = make_float4(0.f, 0.f, 0.f, 0.f);        // no token: beta 0, nothing is written
-    }
-    float* val = num + M::NUM;
-    for (int x = tid; x < nt * COLS; x += DL_THREADS) {
-      const int tt = x / COLS, c = x % COLS;
-      if (c < cols_here) cp_async4(val + x, p.qkv + (size_t)(tb + tt) * p.ld + off_v + c);
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-
-  if (t0 < t1) fetch(0, t0);
-  int buf = 0;
-  for (int tb = t0; tb < t1; tb += TT, buf ^= 1) {
-    const int nt = min(TT, t1 - tb);
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                  // these chunks have arrived, and everyone is done with the other buffer
-    if (tb + TT < t1) fetch(buf ^ 1, tb + TT);
-    const float* s = sm + buf * M::BUF;
-#pragma unroll 1
-    for (int ch = 0; ch < NC && ch * DL_CHUNK < nt; ++ch) {
-      const float* vec = s + (size_t)ch * DL_CHUNK * 3 * DP;
-      const float* num = s + M::VEC + M::TOTAL + ch * DL_CHUNK * 8;
-      const float* val = s + M::VEC + M::TOTAL + M::NUM + ch * DL_CHUNK * COLS;
-      const float* at = vec + 4 * l;                 // this lane's first quad of the chunk's vectors; the next lies 4 * L further on
+  float* out = p.o + (size_t)t0 * p.H * p.e + (size_t)h * p.e + c0;
+  const int mine = l / (L / 4);                      // the token of a chunk whose outputs this lane ends with
+  int ch = 0;
+  bool lost = false;
+  for (; ch < n_chunks; ++ch) {
+    const float* s = sm + (size_t)(ch % ST) * REC;
+    const bool here = tc5::mbar_wait(&full[ch % ST], (ch / ST) & 1);
+    {
+      const float* at = s + 4 * l;                   // this lane's first quad of the chunk's vectors; the next lies 4 * L further on
+      const float* num = s + 13 * DP;
       auto load = [&](float4 (&kk)[DL_CHUNK], float4 (&qq)[DL_CHUNK], int j) {
 #pragma unroll
         for (int i = 0; i < DL_CHUNK; ++i) {
@@ -226,22 +215,22 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs
       auto load_write = [&](float4 (&kk)[DL_CHUNK], float4& T, int j) {
 #pragma unroll
         for (int i = 0; i < DL_CHUNK; ++i) kk[i] = *reinterpret_cast<const float4*>(at + (3 * i + 2) * DP + 4 * L * j);
-        T = *reinterpret_cast<const float4*>(s + M::VEC + (size_t)ch * DP + 4 * l + 4 * L * j);
+        T = *reinterpret_cast<const float4*>(at + 12 * DP + 4 * L * j);
       };
       // reads and outputs over S0: the next quad's vectors are under way while one quad is worked on, eight sums at a time
       float4 kk[2][DL_CHUNK], qq[2][DL_CHUNK], T[2];
-      float r[X][DL_CHUNK], y[X][DL_CHUNK], w[X][DL_CHUNK];
+      float r[X][DL_CHUNK], y[X][DL_CHUNK];
+      float4 w[X];                                   // the four tokens' values of each column
       load(kk[0], qq[0], 0);
       float4 A[DL_CHUNK];                            // A_i0 A_i1 A_i2 beta_i
 #pragma unroll
       for (int i = 0; i < DL_CHUNK; ++i) {
         A[i] = *reinterpret_cast<const float4*>(num + 8 * i);
 #pragma unroll
-        for (int x = 0; x < X; ++x) {
-          r[x][i] = y[x][i] = 0.f;
-          w[x][i] = val[i * COLS + grp + x * GROUPS];
-        }
+        for (int x = 0; x < X; ++x) r[x][i] = y[x][i] = 0.f;
       }
+#pragma unroll
+      for (int x = 0; x < X; ++x) w[x] = *reinterpret_cast<const float4*>(s + VEC + 4 * (grp * X + x));
 #pragma unroll
       for (int j = 0; j < NQ; ++j) {
         if (j + 1 < NQ) load(kk[(j + 1) & 1], qq[(j + 1) & 1], j + 1);
@@ -276,7 +265,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs
       for (int i = 0; i < DL_CHUNK; ++i)
 #pragma unroll
         for (int x = 0; x < X; ++x) {
-          float z = w[x][i] - r[x][i];
+          float z = (i == 0 ? w[x].x : (i == 1 ? w[x].y : (i == 2 ? w[x].z : w[x].w))) - r[x][i];
           if (i > 0) z = fmaf(-A[i].x, u[x][0], z);
           if (i > 1) z = fmaf(-A[i].y, u[x][1], z);
           if (i > 2) z = fmaf(-A[i].z, u[x][2], z);
@@ -298,28 +287,34 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs
             S[x][j].w = fmaf(kk[j & 1][i].w, u[x][i], S[x][j].w);
           }
       }
-      const int mine = l / (L / 4);                  // the token whose output this lane ended with
       const float4 B = *reinterpret_cast<const float4*>(num + 8 * mine + 4);
+      const int t = ch * DL_CHUNK + mine;
 #pragma unroll
       for (int x = 0; x < X; ++x) {
         a[x] = fmaf(B.x, u[x][0], fmaf(B.y, u[x][1], fmaf(B.z, u[x][2], fmaf(B.w, u[x][3], a[x]))));
-        if (l % (L / 4) == 0) os[(ch * DL_CHUNK + mine) * COLS + grp + x * GROUPS] = a[x];
+        if (l % (L / 4) == 0 && t < t1 - t0 && c0 + x < p.e) out[(size_t)t * p.H * p.e + x] = a[x];
       }
     }
-    __syncthreads();
-    for (int x = tid; x < nt * COLS; x += DL_THREADS) {
-      const int tt = x / COLS, c = x % COLS;
-      if (c < cols_here) p.o[(size_t)(tb + tt) * p.H * p.e + (size_t)h * p.e + c0 + c] = os[x];
+    if (__syncthreads_or(!here)) {                   // everyone is done with this record, or one never came
+      lost = true;
+      break;
     }
+    if (tid == 0 && ch + ST < n_chunks) fetch(ch + ST);
   }
   zk_let_next_start();      // only now: a block that waits for this long kernel would hold an SM's issue slots against it
+  if (lost) {
+    if (tid == 0) {
+      atomicExch(p.status, 19);
+      for (int k = ch + 1; k < n_chunks && k < ch + ST; ++k) tc5::mbar_wait(&full[k % ST], (k / ST) & 1);      // the copies under way
+    }
+    return;
+  }
 #pragma unroll
   for (int x = 0; x < X; ++x) {
-    const int c = c0 + grp + x * GROUPS;
 #pragma unroll
     for (int j = 0; j < NQ; ++j) {
       const int i = 4 * (l + L * j);
-      if (c < p.e && i < p.d4) *reinterpret_cast<float4*>(st + (size_t)c * p.d4 + i) = S[x][j];
+      if (c0 + x < p.e && i < p.d4) *reinterpret_cast<float4*>(st + (size_t)(c0 + x) * p.d4 + i) = S[x][j];
     }
   }
 }
@@ -388,16 +383,19 @@ __global__ void __launch_bounds__(DL_THREADS) delta_single_kernel(const DeltaArg
 
 namespace {
 
-template <int L, int CH, int X, int NC>
+template <int L, int CH, int X, int ST>
 int launch_chunks(const DeltaArgs& p, int n_seqs, cudaStream_t stream) {
-  using M = ChunkSmem<L, CH, X, NC>;
-  auto kern = delta_chunk_kernel<L, CH, X, NC>;
-  if (M::BYTES > 48 * 1024) {
-    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)M::BYTES);
+  auto kern = delta_chunk_kernel<L, CH, X, ST>;
+  constexpr int COLS = DL_THREADS / L * X;
+  constexpr size_t smem = sizeof(float) * ST * (vector_floats(L * CH) + COLS * DL_CHUNK);
+  if (smem > 40 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  return zk_launch_dependent(kern, dim3(n_seqs, p.H, (p.e + M::COLS - 1) / M::COLS), dim3(DL_THREADS), M::BYTES, stream, p);
+  return zk_launch_dependent(kern, dim3(n_seqs, p.H, (p.e + COLS - 1) / COLS), dim3(DL_THREADS), smem, stream, p);
 }
+
+int padded_channels(int d) { return d <= 32 ? 32 : (d <= 64 ? 64 : (d <= 128 ? 128 : (d <= 256 ? 256 : 512))); }
 
 template <int L, int CH>
 int launch_single(const DeltaArgs& p, int n_seqs, cudaStream_t stream) {
@@ -417,9 +415,8 @@ int zk_delta_max_dim() { return DL_MAX_D; }
 int zk_delta_state_floats(int H, int d, int e) { return H * e * ((d + 3) / 4 * 4); }
 
 // Floats of scratch a prompt step of n tokens and n_seqs sequences needs.
-long long zk_delta_scratch_floats(int n, int n_seqs, int H, int d) {
-  const long long d4 = (d + 3) / 4 * 4;
-  return (long long)n * H * (3 * d4 + 8) + (long long)(n / DL_CHUNK + n_seqs) * H * d4;
+long long zk_delta_scratch_floats(int n, int n_seqs, int H, int d, int e) {
+  return (long long)(n / DL_CHUNK + n_seqs) * H * record_floats(padded_channels(d), e);
 }
 
 // For measurements: lanes per column (8 or 16) of prompt steps with 65..128 key channels; 0 gives the choice back.
@@ -436,16 +433,16 @@ int zk_delta_force_lanes(int lanes) {
 int zk_delta_scan(const float* qkv, int ld, const float* a, int ld_a, const float* zb, int ld_b, const float* a_log,
                   const float* dt_bias, float* state, long long state_stride, float* o, const int* cu_q, const int* seq_slot,
                   const int* tok_seq, int n, int n_seqs, int H, int G, int d, int e, float q_scale, float* scratch,
-                  cudaStream_t stream) {
+                  int* status, cudaStream_t stream) {
   if (n_seqs <= 0 || n <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || d <= 0 || e <= 0 || d > DL_MAX_D) return ZK_EINVAL;
-  if (ld < 2 * G * d + H * e || ld_a < H * d || ld_b < H || !a_log || !dt_bias || !zb) return ZK_EINVAL;
+  if (ld < 2 * G * d + H * e || ld_a < H * d || ld_b < H || !a_log || !dt_bias || !zb || !status) return ZK_EINVAL;
   if (state_stride % 4 || (uintptr_t)state % 16 || (uintptr_t)scratch % 16 || (!scratch && n != n_seqs)) return ZK_EINVAL;
   DeltaArgs p{};
   p.qkv = qkv; p.a = a; p.zb = zb; p.a_log = a_log; p.dt_bias = dt_bias;
   p.state = state; p.o = o; p.cu_q = cu_q; p.seq_slot = seq_slot; p.tok_seq = tok_seq; p.state_stride = state_stride;
   p.ld = ld; p.ld_a = ld_a; p.ld_b = ld_b; p.H = H; p.G = G; p.d = d; p.e = e; p.d4 = (d + 3) / 4 * 4;
-  p.q_scale = q_scale;
+  p.q_scale = q_scale; p.status = status;
   if (!scratch) {
     if (d <= 32) return launch_single<8, 4>(p, n_seqs, stream);
     if (d <= 64) return launch_single<8, 8>(p, n_seqs, stream);
@@ -453,9 +450,7 @@ int zk_delta_scan(const float* qkv, int ld, const float* a, int ld_a, const floa
     if (d <= 256) return launch_single<16, 16>(p, n_seqs, stream);
     return launch_single<32, 16>(p, n_seqs, stream);
   }
-  p.vec = scratch;
-  p.num = p.vec + (size_t)n * H * 3 * p.d4;
-  p.total = p.num + (size_t)n * H * 8;
+  p.rec = scratch;
   const dim3 grid(n, (H + 3) / 4), block(128);
   int rc;
   if (d <= 32) rc = zk_launch_dependent(delta_chunk_prepare_kernel<1>, grid, block, 0, stream, p);
@@ -464,11 +459,11 @@ int zk_delta_scan(const float* qkv, int ld, const float* a, int ld_a, const floa
   else if (d <= 256) rc = zk_launch_dependent(delta_chunk_prepare_kernel<8>, grid, block, 0, stream, p);
   else rc = zk_launch_dependent(delta_chunk_prepare_kernel<16>, grid, block, 0, stream, p);
   if (rc != 0) return rc;
-  if (d <= 32) return launch_chunks<8, 4, 1, 2>(p, n_seqs, stream);
-  if (d <= 64) return launch_chunks<16, 4, 2, 2>(p, n_seqs, stream);
-  if (d <= 128) return forced_layout == 8 ? launch_chunks<8, 16, 1, 2>(p, n_seqs, stream) : launch_chunks<16, 8, 2, 2>(p, n_seqs, stream);
-  if (d <= 256) return launch_chunks<16, 16, 2, 1>(p, n_seqs, stream);
-  return launch_chunks<32, 16, 2, 1>(p, n_seqs, stream);
+  if (d <= 32) return launch_chunks<8, 4, 1, 8>(p, n_seqs, stream);
+  if (d <= 64) return launch_chunks<16, 4, 2, 8>(p, n_seqs, stream);
+  if (d <= 128) return forced_layout == 8 ? launch_chunks<8, 16, 1, 6>(p, n_seqs, stream) : launch_chunks<16, 8, 2, 6>(p, n_seqs, stream);
+  if (d <= 256) return launch_chunks<16, 16, 2, 4>(p, n_seqs, stream);
+  return launch_chunks<32, 16, 2, 4>(p, n_seqs, stream);
 }
 
 }  // extern "C"

@@ -211,7 +211,7 @@ __global__ void __launch_bounds__(HG_R * 32)
       const float m = fmaxf(A + m_run, B);
       float before = __shfl_up_sync(0xffffffffu, m, 1);
       if (lane == 0) before = m_run;
-      lane_decay = expf(gf + before - m);
+      lane_decay = expf(gf - (m - before));      // in this order what m was rounded by is not lost
       lane_dt = expf(gi - m);
       if (warp == 0 && blockIdx.z == 0 && lane < nt) cp.m_out[(size_t)(tb + lane) * H + h] = m;
       m_run = __shfl_sync(0xffffffffu, m, nt - 1);

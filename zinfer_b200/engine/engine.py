@@ -36,7 +36,8 @@ _STATUS_TEXT = {1: "a token id lies outside the vocabulary", 2: "a token's posit
                 15: "the tcgen05 prompt attention gave up waiting for its query or K/V tiles",
                 16: "the tcgen05 prompt attention gave up waiting for the probabilities",
                 17: "the tcgen05 prompt attention gave up waiting for the scores",
-                18: "the tcgen05 prompt attention gave up waiting for P V"}
+                18: "the tcgen05 prompt attention gave up waiting for P V",
+                19: "the gated delta rule gave up waiting for a chunk's vectors"}
 
 
 class _DecodeBatch:

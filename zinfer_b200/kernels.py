@@ -69,9 +69,9 @@ _SIGNATURES = {
     "delta": {
         "zk_delta_max_dim": "",
         "zk_delta_state_floats": "iii",
-        "zk_delta_scratch_floats": "iiii",
+        "zk_delta_scratch_floats": "iiiii",
         "zk_delta_force_lanes": "i",
-        "zk_delta_scan": "pipipipp" + "plpppp" + "iiiiii" + "fp" + "p",
+        "zk_delta_scan": "pipipipp" + "plpppp" + "iiiiii" + "fpp" + "p",
     },
     "seqconv": {
         "zk_seqconv_forward": "ppppppp" + "iiiliii" + "ipi" + "p",
@@ -595,10 +595,11 @@ def delta_scan(qkv: torch.Tensor, a: torch.Tensor, z_beta: torch.Tensor, a_log: 
     o = torch.empty((n, H * e), dtype=torch.float32, device=qkv.device)
     scratch = None
     if not single_token:
-        scratch = torch.empty(_fn("delta", "zk_delta_scratch_floats")(n, n_seqs, H, d), dtype=torch.float32, device=qkv.device)
+        scratch = torch.empty(_fn("delta", "zk_delta_scratch_floats")(n, n_seqs, H, d, e), dtype=torch.float32, device=qkv.device)
     _check(_fn("delta", "zk_delta_scan")(_ptr(qkv), qkv.stride(0), _ptr(a), a.stride(0), _ptr(z_beta), z_beta.stride(0), _ptr(a_log),
                                          _ptr(dt_bias), _ptr(state), state.stride(0), _ptr(o), _ptr(cu_q), _ptr(seq_slot), _ptr(tok_seq),
-                                         n, n_seqs, H, G, d, e, float(d) ** -0.5, _ptr(scratch), _stream()), "delta_scan")
+                                         n, n_seqs, H, G, d, e, float(d) ** -0.5, _ptr(scratch),
+                                         _ptr(status_word(qkv.device)), _stream()), "delta_scan")
     return o
 
 
