@@ -1620,7 +1620,7 @@ def qk_normed(qkv, q_w, k_w, n_heads: int, n_kv: int, head_dim: int, eps: float,
     _check(_fn("attention", "zk_qk_prepare")(
         _ptr(qkv), None, _ptr(dense), None, None, _ptr(q_w), _ptr(k_w), None, None, _ptr(tok_pos), None, None, 0,
         qkv.shape[0], n_heads, n_kv, head_dim, 0, 0, eps, 1, 0, dtype_code(qkv.dtype), _ptr(status), head_dim, 0, 0.0, 0,
-        qkv.shape[1], None, 0, 0, 0, 0.0, _stream()),
+        qkv.shape[1], None, 0, 0, 0, 0.0, 1.0, _stream()),
         "qk_normed")
     return dense
 
